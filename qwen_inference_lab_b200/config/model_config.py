@@ -527,3 +527,102 @@ class GogotarConfig:
 
     def __eq__(self, other):
         return isinstance(other, GogotarConfig) and self.to_dict() == other.to_dict()
+
+
+class LotazenConfig:
+    """Lotazen: a decoder whose layers are listed one by one in config.json; both sublayers of a layer read the same norm.
+
+    ``vocab``, ``width``, ``norm.eps``, ``max_positions`` (rows of the table of positions), ``logit_softcap``
+    (logits <- cap * tanh(logits / cap)) and ``layers``.  A layer is a ``parallel`` mixer (``left`` a windowed attention:
+    ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale``, ``rot`` with ``base``, ``dims`` and ``scaling.factor``,
+    ``mask.size`` the window; ``right`` HGRN2: ``heads``, ``dim``, ``vdim``; ``left_scale``, ``right_scale``) or a matrix
+    memory, ``mlstm`` or ``mlstm_2`` (``heads``, ``dim``, ``vdim``, ``gate_cap``), beside a feed-forward: ``mlp`` null
+    or ``moe`` (``expert`` and ``shared`` with ``ff`` and ``limit``, ``router.experts``, ``router.top``).  The
+    configuration is kept as the dictionary it came in; this class checks it and answers the few questions the engine asks.
+    """
+    architecture = "Lotazen"
+    model_type = "lotazen"
+    MEMORIES = ("mlstm", "mlstm_2")
+
+    def __init__(self, data: dict):
+        self.data = data
+        for key in ("vocab", "width", "max_positions"):
+            if not _positive_int(data.get(key)):
+                raise ConfigError(f"{key} must be a positive integer, got {data.get(key)!r}")
+        eps = (data.get("norm") or {}).get("eps")
+        if not _positive_number(eps):
+            raise ConfigError(f"norm.eps must be a positive number, got {eps!r}")
+        cap = data.get("logit_softcap")
+        if cap is not None and not _positive_number(cap):
+            raise ConfigError(f"logit_softcap must be a positive number or absent, got {cap!r}")
+        layers = data.get("layers")
+        if not isinstance(layers, list) or not layers:
+            raise ConfigError("layers must be a non-empty list")
+        for index, layer in enumerate(layers):
+            where = f"layers[{index}]"
+            kind, mixer = layer.get("type"), layer.get("mixer")
+            if not isinstance(mixer, dict):
+                raise ConfigError(f"{where}.mixer must be an object")
+            if kind == "parallel":
+                self._check_parallel(where, mixer)
+            elif kind in self.MEMORIES:
+                LarolornConfig._check_sizes(where, mixer, ("heads", "dim", "vdim"))
+                if not _positive_number(mixer.get("gate_cap")):
+                    raise ConfigError(f"{where}.gate_cap must be a positive number, got {mixer.get('gate_cap')!r}")
+            else:
+                raise ConfigError(f"{where}.type {kind!r} is none of parallel, {', '.join(self.MEMORIES)}")
+            if layer.get("mlp") is not None:
+                self._check_experts(where, layer["mlp"])
+        self.vocab_size, self.width, self.eps = data["vocab"], data["width"], float(eps)
+        self.logit_softcap, self.layers, self.max_positions = float(cap or 0.0), layers, data["max_positions"]
+        eos = data.get("eos_token_id")
+        self.eos_token_ids = frozenset() if eos is None else frozenset(eos if isinstance(eos, list) else [eos])
+
+    @staticmethod
+    def _check_parallel(where, mixer):
+        left, right = mixer.get("left"), mixer.get("right")
+        if not isinstance(left, dict) or not isinstance(right, dict):
+            raise ConfigError(f"{where}.mixer needs a left and a right mixer")
+        LarolornConfig._check_sizes(where + ".left", left, ("heads", "kv_heads", "dim", "vdim"))
+        if left["heads"] % left["kv_heads"]:
+            raise ConfigError(f"{where}: {left['heads']} heads do not divide into {left['kv_heads']} kv heads")
+        LarolornConfig._check_rotation(where + ".left", left, left["dim"])
+        scaling = left["rot"].get("scaling")
+        if scaling is not None and not _positive_number(scaling.get("factor")):
+            raise ConfigError(f"{where}.left.rot.scaling needs a positive factor, got {scaling!r}")
+        if left.get("mask") is not None:
+            LarolornConfig._check_mask(where + ".left", left)
+        if not _positive_number(left.get("scale")):
+            raise ConfigError(f"{where}.left.scale must be a positive number, got {left.get('scale')!r}")
+        LarolornConfig._check_sizes(where + ".right", right, ("heads", "dim", "vdim"))
+        for key in ("left_scale", "right_scale"):
+            value = mixer.get(key)
+            if isinstance(value, bool) or not isinstance(value, (int, float)):
+                raise ConfigError(f"{where}.{key} must be a number, got {value!r}")
+
+    @staticmethod
+    def _check_experts(where, mlp):
+        if mlp.get("kind") != "moe":
+            raise ConfigError(f"{where}.mlp.kind {mlp.get('kind')!r} is not moe")
+        router = mlp.get("router") or {}
+        if not _positive_int(router.get("experts")) or not _positive_int(router.get("top")) \
+                or router["top"] > router["experts"]:
+            raise ConfigError(f"{where}.mlp needs router.experts and router.top <= experts")
+        for key in ("expert", "shared"):
+            part = mlp.get(key)
+            if part is None and key == "shared":
+                continue
+            if not isinstance(part, dict) or not _positive_int(part.get("ff")) or not _positive_number(part.get("limit")):
+                raise ConfigError(f"{where}.mlp.{key} needs a positive ff and limit")
+
+    @classmethod
+    def from_dict(cls, data: dict) -> "LotazenConfig":
+        if data.get("architecture", cls.architecture) != cls.architecture:
+            raise ConfigError(f"architecture {data.get('architecture')!r} is not {cls.architecture}")
+        return cls(json.loads(json.dumps(data)))
+
+    def to_dict(self) -> dict:
+        return json.loads(json.dumps(self.data)) | {"architecture": self.architecture}
+
+    def __eq__(self, other):
+        return isinstance(other, LotazenConfig) and self.to_dict() == other.to_dict()

@@ -174,6 +174,9 @@ struct AtParams {
     // chunk > 0: a query sees only the keys of its own chunk of that many positions (counted from position 0): the
     // tiles start at the chunk of the tile's first row, and rows of a later chunk mask what lies before theirs
     int chunk;
+    // window > 0: a query sees the keys of the last `window` positions, its own included: tiles start at the first key
+    // that the tile's first row sees, later rows mask what lies before their own window
+    int window;
     // null, or one learned score per query head times log2(e): exp2 of it joins the softmax's denominator, a key
     // without a value whose score is neither scaled nor biased
     const float* sink_log2;
@@ -209,7 +212,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     const int4 info = tile_info[blockIdx.y];
     const int n0 = info.x, pos0 = info.y;
     const int hi = pos0 + AT_M - 1;                          // last key any row of the tile may see
-    const int tile0 = p.chunk > 0 ? pos0 / p.chunk * p.chunk / AT_N : 0;   // the key tile that holds the first key any row sees
+    // the first key that the query at a position sees
+    auto first_key_of = [&p](int position) {
+        const int of_chunk = p.chunk > 0 ? position / p.chunk * p.chunk : 0;
+        return p.window > 0 ? max(of_chunk, position - p.window + 1) : of_chunk;
+    };
+    const int tile0 = first_key_of(pos0) / AT_N;             // the key tile that holds the first key any row sees
     const int n_tiles = hi / AT_N + 1 - tile0;
     const int* table = p.block_table + (size_t)info.w * p.table_stride;
 
@@ -356,7 +364,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         const int quarter = warp & 3;
         const int row = quarter * 32 + lane;                 // query row of this thread = its TMEM lane
         const int pos = pos0 + row;
-        const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;   // the first key this row sees
+        const int lo = first_key_of(pos);                     // the first key this row sees
         const unsigned lane_base = (unsigned)(quarter * 32) << 16;
         // With a distance bias the scores are scaled and biased first and the steps below take them as they are.
         const bool capped = p.cap_log2 > 0.f;
@@ -406,7 +414,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 #pragma unroll
                 for (int i = 0; i < AT_N; ++i) s[i] = fmaf(s[i], p.scale_log2, fmaf(slope, (float)i, base));
             }
-            if (key0 + AT_N - 1 > pos0 || key0 < lo) {
+            if (key0 + AT_N - 1 > pos0 || key0 < lo) {        // tiles past the first row, or before this row's first key
 #pragma unroll
                 for (int i = 0; i < AT_N; ++i) s[i] = (key0 + i <= pos && key0 + i >= lo) ? s[i] : -INFINITY;
             }
@@ -547,12 +555,12 @@ extern "C" int qil_attn_tc_keys_per_tile() { return AT_N; }
 // page_size must divide the keys per tile and be a multiple of 8.  error_word: a device int, zeroed by the
 // caller once.  trace: null, or 3 * 1024 int64 for the time stamps of block (0, 0) in a build with AT_TRACE.
 // slopes_log2: null, or float32 [n_q_heads] on the device: a distance bias per query head (see AtParams).
-// chunk, sink_log2 (null, or float32 [n_q_heads] on the device): see AtParams.  softcap > 0: capped scores.
+// chunk, window, sink_log2 (null, or float32 [n_q_heads] on the device): see AtParams.  softcap > 0: capped scores.
 extern "C" int qil_attn_tc_prefill_capped(const void* q, const void* kv, void* out, const int* tile_info, int n_tiles,
                                           int n_tokens, const int* block_table, int table_stride, int n_q_heads,
                                           int n_kv_heads, int page_size, int num_pages, float scale,
                                           const float* slopes_log2, int chunk, const float* sink_log2, float softcap,
-                                          int* error_word, long long* trace, cudaStream_t stream);
+                                          int window, int* error_word, long long* trace, cudaStream_t stream);
 
 extern "C" int qil_attn_tc_prefill_masked(const void* q, const void* kv, void* out, const int* tile_info, int n_tiles,
                                           int n_tokens, const int* block_table, int table_stride, int n_q_heads,
@@ -561,16 +569,17 @@ extern "C" int qil_attn_tc_prefill_masked(const void* q, const void* kv, void* o
                                           long long* trace, cudaStream_t stream) {
     return qil_attn_tc_prefill_capped(q, kv, out, tile_info, n_tiles, n_tokens, block_table, table_stride, n_q_heads,
                                       n_kv_heads, page_size, num_pages, scale, slopes_log2, chunk, sink_log2, 0.f,
-                                      error_word, trace, stream);
+                                      0, error_word, trace, stream);
 }
 
 extern "C" int qil_attn_tc_prefill_capped(const void* q, const void* kv, void* out, const int* tile_info, int n_tiles,
                                           int n_tokens, const int* block_table, int table_stride, int n_q_heads,
                                           int n_kv_heads, int page_size, int num_pages, float scale,
                                           const float* slopes_log2, int chunk, const float* sink_log2, float softcap,
-                                          int* error_word, long long* trace, cudaStream_t stream) {
+                                          int window, int* error_word, long long* trace, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
-    if (chunk < 0 || softcap < 0.f) QIL_REFUSE("attn_tc: chunks of %d positions, a cap of %g", chunk, (double)softcap);
+    if (chunk < 0 || softcap < 0.f || window < 0)
+        QIL_REFUSE("attn_tc: chunks of %d positions, a cap of %g, a window of %d", chunk, (double)softcap, window);
     if (n_kv_heads <= 0 || n_q_heads % n_kv_heads) QIL_REFUSE("attn_tc: %d query heads, %d kv heads", n_q_heads, n_kv_heads);
     if (page_size < 8 || page_size > AT_N || AT_N % page_size || page_size % 8)
         QIL_REFUSE("attn_tc: pages of %d positions; this kernel takes multiples of 8 that divide %d", page_size, AT_N);
@@ -606,7 +615,7 @@ extern "C" int qil_attn_tc_prefill_capped(const void* q, const void* kv, void* o
     p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads; p.page_size = page_size;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.slopes_log2 = slopes_log2;
-    p.chunk = chunk; p.sink_log2 = sink_log2;
+    p.chunk = chunk; p.window = window; p.sink_log2 = sink_log2;
     p.tanh_arg = p.cap_log2 = 0.f;
     if (softcap > 0.f) {
         p.tanh_arg = (float)(2.0 * 1.4426950408889634 * (double)scale / (double)softcap);

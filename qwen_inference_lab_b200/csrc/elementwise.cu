@@ -12,13 +12,21 @@ QIL_ERROR_STORAGE
 // ---------------------------------------------------------------- embedding
 template <typename T, typename W>
 __global__ void embed_gather_kernel(const W* __restrict__ table, const int* __restrict__ ids,
-                                    T* __restrict__ out, int width, int vocab, float scale) {
+                                    T* __restrict__ out, int width, int vocab, float scale,
+                                    const W* __restrict__ pos_table, const int* __restrict__ positions, int n_positions) {
     const int row = blockIdx.x;
     int id = ids[row];
     // Host code validates ids; clamp so that a bad id can never read out of bounds.
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
     const W* src = table + (size_t)id * width;
     T* dst = out + (size_t)row * width;
+    if (pos_table != nullptr) {
+        int p = positions[row];
+        p = p < 0 ? 0 : (p >= n_positions ? n_positions - 1 : p);
+        const W* at = pos_table + (size_t)p * width;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = from_f32<T>(to_f32<W>(src[i]) * scale + to_f32<W>(at[i]));
+        return;
+    }
     for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = from_f32<T>(to_f32<W>(src[i]) * scale);
 }
 
@@ -36,18 +44,23 @@ __global__ void embed_gather_bf16x8_kernel(const bf16* __restrict__ table, const
 }
 
 extern "C" int qil_embed_gather(const void* table, int table_dtype, const int* ids, void* out,
-                                int out_dtype, int n_rows, int width, int vocab, float scale, cudaStream_t stream) {
-    // scale: what every row is multiplied by on its way out (float32 product, one rounding)
+                                int out_dtype, int n_rows, int width, int vocab, float scale, const void* pos_table,
+                                const int* positions, int n_positions, cudaStream_t stream) {
+    // scale: what every row is multiplied by on its way out (float32 product, one rounding).  pos_table (null: none), of
+    // the table's type, [n_positions, width]: the row of the token's position is added, unscaled, before the rounding
     if (n_rows <= 0) return 0;
     if (width <= 0 || vocab <= 0) QIL_REFUSE("embed_gather: width %d vocab %d", width, vocab);
-    if (scale == 1.0f && out_dtype == QIL_BF16 && table_dtype == QIL_BF16 && width % 8 == 0 &&
+    if (pos_table != nullptr && (positions == nullptr || n_positions <= 0))
+        QIL_REFUSE("embed_gather: a table of %d positions", n_positions);
+    if (pos_table == nullptr && scale == 1.0f && out_dtype == QIL_BF16 && table_dtype == QIL_BF16 && width % 8 == 0 &&
         (((uintptr_t)table | (uintptr_t)out) & 15) == 0) {
         qil_launch_chained(embed_gather_bf16x8_kernel, dim3(n_rows), dim3(128), 0, stream,
                            (const bf16*)table, ids, (bf16*)out, width, vocab);
         QIL_CHECK_LAUNCH();
     }
     QIL_DISPATCH_2(out_dtype, table_dtype,
-        embed_gather_kernel<T, W><<<n_rows, 256, 0, stream>>>((const W*)table, ids, (T*)out, width, vocab, scale));
+        embed_gather_kernel<T, W><<<n_rows, 256, 0, stream>>>((const W*)table, ids, (T*)out, width, vocab, scale,
+                                                        (const W*)pos_table, positions, n_positions));
     QIL_CHECK_LAUNCH();
 }
 

@@ -25,30 +25,66 @@ __device__ __forceinline__ float gated_value(int kind, float g, float u, float l
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-gated_activation_kernel(const T* __restrict__ gate_up, T* __restrict__ out, size_t total, int width, int pairs8,
+gated_activation_kernel(const T* __restrict__ gate_up, long long ld, T* __restrict__ out, size_t total, int width, int pairs8,
                         int kind, float limit, float alpha) {
     qil_wait_for_producer();
     qil_release_consumer();
     for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < total; i += (size_t)gridDim.x * 256) {
         const size_t row = i / width;
         const int col = (int)(i % width);
-        const T* src = gate_up + row * 2 * width;
+        const T* src = gate_up + row * ld;
         const int g_at = pairs8 ? (col / 8) * 16 + (col % 8) : col;
         const int u_at = pairs8 ? g_at + 8 : col + width;
         out[i] = from_f32<T>(gated_value(kind, to_f32<T>(src[g_at]), to_f32<T>(src[u_at]), limit, alpha));
     }
 }
 
-extern "C" int qil_gated_activation(const void* gate_up, void* out, int n_rows, int width, int act_dtype, int pairs8,
+// The same for a width and a row stride that allow 16-byte loads: eight (bfloat16) or four (float32) values a thread.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_activation_wide_kernel(const T* __restrict__ gate_up, long long ld, T* __restrict__ out, int n_rows, int width,
+                             int kind, float limit, float alpha) {
+    constexpr int V = 16 / (int)sizeof(T);
+    qil_wait_for_producer();
+    qil_release_consumer();
+    const int per_row = width / V;
+    const size_t total = (size_t)n_rows * per_row;
+    for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < total; i += (size_t)gridDim.x * 256) {
+        const size_t row = i / per_row;
+        const int col = (int)(i % per_row) * V;
+        const T* src = gate_up + row * ld;
+        const uint4 g4 = *reinterpret_cast<const uint4*>(src + col), u4 = *reinterpret_cast<const uint4*>(src + width + col);
+        const T* g = reinterpret_cast<const T*>(&g4);
+        const T* u = reinterpret_cast<const T*>(&u4);
+        uint4 packed;
+        T* o = reinterpret_cast<T*>(&packed);
+#pragma unroll
+        for (int k = 0; k < V; ++k) o[k] = from_f32<T>(gated_value(kind, to_f32<T>(g[k]), to_f32<T>(u[k]), limit, alpha));
+        *reinterpret_cast<uint4*>(out + row * width + col) = packed;
+    }
+}
+
+// ld: row stride of gate_up (its rows may be a column range of a wider buffer).
+extern "C" int qil_gated_activation(const void* gate_up, long long ld, void* out, int n_rows, int width, int act_dtype, int pairs8,
                                     int kind, float limit, float alpha, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     if (width <= 0 || kind < 0 || kind > 2) QIL_REFUSE("gated_activation: width %d kind %d", width, kind);
     if (pairs8 && width % 8) QIL_REFUSE("gated_activation: the paired layout needs a width that is a multiple of 8");
+    if (ld < 2ll * width) QIL_REFUSE("gated_activation: row stride %lld for width %d", ld, width);
+    const int vec = act_dtype == QIL_BF16 ? 8 : 4;
+    if (!pairs8 && width % vec == 0 && ld % vec == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0) {
+        const size_t pieces = (size_t)n_rows * (width / vec);
+        const int wide_blocks = (int)((pieces + 255) / 256 < 148 * 16 ? (pieces + 255) / 256 : 148 * 16);
+        QIL_DISPATCH_1(act_dtype,
+            qil_launch_chained(gated_activation_wide_kernel<T>, dim3(wide_blocks), dim3(256), 0, stream, (const T*)gate_up, ld,
+                               (T*)out, n_rows, width, kind, limit, alpha));
+        QIL_CHECK_LAUNCH();
+    }
     const size_t total = (size_t)n_rows * width;
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     QIL_DISPATCH_1(act_dtype,
         qil_launch_chained(gated_activation_kernel<T>, dim3(blocks), dim3(256), 0, stream,
-                           (const T*)gate_up, (T*)out, total, width, pairs8, kind, limit, alpha));
+                           (const T*)gate_up, ld, (T*)out, total, width, pairs8, kind, limit, alpha));
     QIL_CHECK_LAUNCH();
 }
 

@@ -32,6 +32,23 @@
 // and v as they are read (in float32).  Such a design norms all heads' outputs together: `force_raw` sends
 // the un-normed outputs to the float32 scratch buffer whatever the sizes, and lin_norm_gate_whole
 // finishes them (one norm over a token's whole row, times sigmoid of the gate).
+//
+// Further forms of what enters the recurrence (`ScanInputs`; all of it float32):
+//
+//   tied gate      k holds a gate's logits z: f = l + (1 - l) sigmoid(z + b) per head and key channel (bias b and lower
+//                  bound l, float or bfloat16 [heads * d]); the channel decays by f and is written with 1 - f, computed
+//                  as (1 - l) sigmoid(-(z + b)) so that a gate near one loses nothing
+//   token scalars  a decay and a write gain per token and head (float32 [tokens, heads], `mlstm_gates` makes them):
+//                  S_t = decay S_(t-1) + gain k_t v_t^T
+//   ones           the state has one column more than the values: its value is the constant one, so that the column
+//                  is the sum of the decayed keys, n_t = decay n_(t-1) + gain k_t, and its output is n_t . q_t
+//
+// mlstm_gates walks the two gates of a matrix memory (log input gate i, log forget gate f, both capped by
+// cap tanh(. / cap), the forget gate through a log sigmoid) over a segment's tokens from the running maximum m in the
+// request's slot: m_t = max(f_t + m_(t-1), i_t), decay_t = exp(f_t + m_(t-1) - m_t), gain_t = exp(i_t - m_t),
+// floor_t = exp(-m_t).  The maximum is a chain of single additions and comparisons in token order, the same bits under
+// every cut.  mlstm_finish divides a head's raw outputs by max(|n . q|, floor) + 1e-6, then by their own root mean
+// square, times a weight per element of all heads and sigmoid of a gate.
 #include "common.cuh"
 
 #define GLA_TB 8
@@ -80,14 +97,32 @@ __device__ __forceinline__ void gla_norm_gate_rows(const float* o_rows, int o_st
         const float scale = 1.0f / sqrtf(ss / (float)e + eps);
         const size_t token = first_token + tb;
         for (int c = lane; c < e; c += 32) {
-            const float gate = to_f32<T>(g[token * ld + head * e + c]);
-            const float y = o[c] * scale * to_f32<W>(norm_w[c]);
-            out[(token * n_heads + head) * e + c] = from_f32<T>(y * (gate / (1.f + expf(-gate))));
+            float y = o[c] * scale * to_f32<W>(norm_w[c]);
+            if (g != nullptr) {
+                const float gate = to_f32<T>(g[token * ld + head * e + c]);
+                y *= gate / (1.f + expf(-gate));
+            }
+            out[(token * n_heads + head) * e + c] = from_f32<T>(y);
         }
     }
 }
 
-__device__ __forceinline__ float scan_input(float x, int act) { return act == 1 ? x / (1.f + expf(-x)) : x; }
+__device__ __forceinline__ float scan_input(float x, int act) { return act ? x / (1.f + expf(-x)) : x; }
+
+// Where the decays come from, and what is done to q, k and v as they are read.
+struct ScanInputs {
+    const float* alpha;          // float32 [tokens, heads * d]: a decay per token and key channel
+    const float* head_decay;     // float32 [heads]: one fixed decay per head
+    const void* gate_bias;       // tied gate, in the weights' type [heads * d]: its bias ...
+    const void* gate_lower;      // ... and its lower bound; k then holds the gate's logits
+    const float* token_decay;    // float32 [tokens, heads]
+    const float* token_gain;     // float32 [tokens, heads]
+    int act;                     // bit 0: silu on q, bit 1: on k, bit 2: on v
+    int ones;                    // 1: the state's last column has the constant value one
+};
+#define SCAN_SILU_Q 1
+#define SCAN_SILU_K 2
+#define SCAN_SILU_V 4
 
 #define GLA_WHOLE 0        // from the state slot, outputs, state written back
 #define GLA_OWN_STATE 1    // from zero, no outputs; the chunk's state and the product of its decays are written
@@ -96,7 +131,7 @@ __device__ __forceinline__ float scan_input(float x, int act) { return act == 1 
 template <typename T, typename W, bool FUSED, int MODE>
 __global__ void __launch_bounds__(GLA_THREADS, GLA_MIN_BLOCKS)
 gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, const T* __restrict__ g,
-                const float* __restrict__ alpha, const float* __restrict__ head_decay, int qkv_act, int ld, float q_scale,
+                ScanInputs in, int ld, float q_scale,
                 const W* __restrict__ norm_w, float eps, float* __restrict__ state, float* __restrict__ decay_product, const int* __restrict__ seg_start,
                 const int* __restrict__ seg_len, const int* __restrict__ seg_row, int n_heads, int d, int e,
                 int ds_count, int tile_cols, float* __restrict__ o_raw, T* __restrict__ out) {
@@ -138,14 +173,39 @@ gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __res
             const int to = tb * stride + (dd / R) * (R + 4) + dd % R;
             const bool real = dd < d;           // rows past d: zeros, which keep their (zero) state rows zero
             const size_t at = (size_t)(first + t0 + tb) * ld + head * d + dd;
-            if (MODE != GLA_OWN_STATE) sq[to] = real ? scan_input(to_f32<T>(q[at]), qkv_act) * q_scale : 0.f;
-            sk[to] = real ? scan_input(to_f32<T>(k[at]), qkv_act) : 0.f;
-            sa[to] = !real ? 0.f : head_decay != nullptr ? head_decay[head]
-                                                         : alpha[(size_t)(first + t0 + tb) * n_heads * d + head * d + dd];
+            if (MODE != GLA_OWN_STATE) sq[to] = real ? scan_input(to_f32<T>(q[at]), in.act & SCAN_SILU_Q) * q_scale : 0.f;
+            const float kv = real ? to_f32<T>(k[at]) : 0.f;
+            float key = 0.f, decay = 0.f;
+            if (real) {
+                if (in.gate_lower != nullptr) {
+                    // both halves from one exponential of a negative number: sigmoid(z) and sigmoid(-z), neither by a
+                    // difference from one
+                    const float low = to_f32<W>(reinterpret_cast<const W*>(in.gate_lower)[head * d + dd]);
+                    const float z = kv + to_f32<W>(reinterpret_cast<const W*>(in.gate_bias)[head * d + dd]);
+                    const float small = expf(-fabsf(z)), inv = 1.f / (1.f + small);
+                    const float up = z >= 0.f ? inv : small * inv, down = z >= 0.f ? small * inv : inv;
+                    decay = fmaf(1.f - low, up, low);
+                    key = (1.f - low) * down;
+                } else {
+                    key = scan_input(kv, in.act & SCAN_SILU_K);
+                    if (in.token_decay != nullptr) {
+                        const size_t scalar = (size_t)(first + t0 + tb) * n_heads + head;
+                        decay = in.token_decay[scalar];
+                        key *= in.token_gain[scalar];
+                    } else {
+                        decay = in.head_decay != nullptr ? in.head_decay[head]
+                                                         : in.alpha[(size_t)(first + t0 + tb) * n_heads * d + head * d + dd];
+                    }
+                }
+            }
+            sk[to] = key;
+            sa[to] = decay;
         }
         for (int i = tid; i < nb * tile_cols; i += threads) {
             const int tb = i / tile_cols, c = col0 + i % tile_cols;
-            sv[i] = c < e ? scan_input(to_f32<T>(v[(size_t)(first + t0 + tb) * ld + head * e + c]), qkv_act) : 0.f;
+            const int values = e - in.ones;
+            sv[i] = c < values ? scan_input(to_f32<T>(v[(size_t)(first + t0 + tb) * ld + head * values + c]), in.act & SCAN_SILU_V)
+                               : (c < e ? 1.f : 0.f);
         }
         __syncthreads();
         if (MODE == GLA_OWN_STATE) {
@@ -249,14 +309,13 @@ gla_norm_gate_kernel(const float* __restrict__ o_raw, const T* __restrict__ g, i
 
 template <typename T, typename W, bool FUSED, int MODE>
 static cudaError_t gla_launch(dim3 grid, int threads, size_t smem, cudaStream_t stream, const void* q, const void* k,
-                              const void* v, const void* g, const float* alpha, const float* head_decay, int qkv_act,
-                              int ld, float q_scale, const void* norm_w, float eps, float* state,
+                              const void* v, const void* g, ScanInputs in, int ld, float q_scale, const void* norm_w, float eps, float* state,
                               float* decay_product, const int* seg_start, const int* seg_len, const int* seg_row, int n_heads, int d, int e,
                               int ds_count, int tile_cols, float* o_raw, void* out) {
     cudaError_t err = cudaFuncSetAttribute(gla_scan_kernel<T, W, FUSED, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) return err;
     return qil_launch_chained(gla_scan_kernel<T, W, FUSED, MODE>, grid, dim3(threads), smem, stream,
-                              (const T*)q, (const T*)k, (const T*)v, (const T*)g, alpha, head_decay, qkv_act, ld, q_scale,
+                              (const T*)q, (const T*)k, (const T*)v, (const T*)g, in, ld, q_scale,
                               (const W*)norm_w, eps, state, decay_product,
                               seg_start, seg_len,
                               seg_row, n_heads, d, e, ds_count, tile_cols, o_raw, (T*)out);
@@ -271,7 +330,8 @@ extern "C" int qil_gla_scan_needs_scratch(int d, int e) {
 }
 
 extern "C" int qil_gla_scan(const void* q, const void* k, const void* v, const void* g, const float* alpha,
-                            const float* head_decay, int qkv_act, int force_raw, int ld, float q_scale, const void* norm_w, float eps, float* state, const int* seg_start, const int* seg_len,
+                            const float* head_decay, const void* gate_bias, const void* gate_lower, const float* token_decay,
+                            const float* token_gain, int act, int ones, int force_raw, int ld, float q_scale, const void* norm_w, float eps, float* state, const int* seg_start, const int* seg_len,
                             const int* seg_row, int n_segments, int n_tokens, int n_heads, int d, int e, float* o_raw,
                             void* out, int mode, float* decay_product, int act_dtype, int weight_dtype,
                             cudaStream_t stream) {
@@ -279,14 +339,20 @@ extern "C" int qil_gla_scan(const void* q, const void* k, const void* v, const v
     // [chunks, heads, d]); GLA_FROM_STATE (state and seg_row as before; the states are read only)
     if (n_segments <= 0) return 0;
     if (mode < 0 || mode > 2 || (mode == GLA_OWN_STATE && decay_product == nullptr)) QIL_REFUSE("gla_scan: mode %d", mode);
-    if (n_heads <= 0 || d <= 0 || e <= 0 || (alpha == nullptr) == (head_decay == nullptr) || n_segments > 65535)
+    const int sources = (alpha != nullptr) + (head_decay != nullptr) + (gate_lower != nullptr) + (token_decay != nullptr);
+    if (sources != 1 || (gate_lower == nullptr) != (gate_bias == nullptr) || (token_decay == nullptr) != (token_gain == nullptr))
+        QIL_REFUSE("gla_scan: exactly one source of decays, a gate with its bias, token decays with their gains");
+    if (ones != 0 && (ones != 1 || e < 2 || !force_raw)) QIL_REFUSE("gla_scan: a column of ones goes with values beside it and raw outputs");
+    if (n_heads <= 0 || d <= 0 || e <= 0 || n_segments > 65535)
         QIL_REFUSE("gla_scan: heads %d sizes %d/%d segments %d", n_heads, d, e, n_segments);
     // a thread holds GLA_R rows of one column; ds_count threads (a power of two within a warp) share a column
     int ds_count = 1;
     while (ds_count * GLA_R < d) ds_count <<= 1;
     if (ds_count > 32) QIL_REFUSE("gla_scan: %d key channels per head are more than %d", d, 32 * GLA_R);
-    const int tile_cols = e < GLA_THREADS / ds_count ? e : GLA_THREADS / ds_count;
-    const int tiles = (e + tile_cols - 1) / tile_cols;
+    const int most_cols = GLA_THREADS / ds_count;
+    const int tiles = (e + most_cols - 1) / most_cols;
+    const int tile_cols = (e + tiles - 1) / tiles;         // even tiles
+    const ScanInputs in = {alpha, head_decay, gate_bias, gate_lower, token_decay, token_gain, act, ones};
     const bool fused = tiles == 1 && !force_raw;
     if (!fused && o_raw == nullptr && mode != GLA_OWN_STATE) QIL_REFUSE("gla_scan: %d value columns per head need the scratch buffer", e);
     const int threads = (tile_cols * ds_count + 31) / 32 * 32;
@@ -295,7 +361,7 @@ extern "C" int qil_gla_scan(const void* q, const void* k, const void* v, const v
     cudaError_t err = cudaSuccess;
 #define QIL_GLA_GO(F, M)                                                                                         \
     QIL_DISPATCH_2(act_dtype, weight_dtype,                                                                      \
-        (err = gla_launch<T, W, F, M>(grid, threads, smem, stream, q, k, v, g, alpha, head_decay, qkv_act, ld,              \
+        (err = gla_launch<T, W, F, M>(grid, threads, smem, stream, q, k, v, g, in, ld,              \
                                       q_scale, norm_w, eps, state, decay_product, seg_start, seg_len, seg_row, n_heads, \
                                       d, e, ds_count, tile_cols, o_raw, out)))
     if (mode == GLA_OWN_STATE) QIL_GLA_GO(false, GLA_OWN_STATE);
@@ -371,5 +437,103 @@ extern "C" int qil_lin_norm_gate_whole(const float* o_raw, const void* g, int ld
     QIL_DISPATCH_2(act_dtype, weight_dtype,
         qil_launch_chained(lin_norm_gate_whole_kernel<T, W>, dim3(n_tokens), dim3(256), 0, stream, o_raw, (const T*)g, ld,
                            (const W*)norm_w, eps, width, (T*)out));
+    QIL_CHECK_LAUNCH();
+}
+
+// ------------------------------------------------------------------ matrix memory: gates and finish
+// One warp per (segment, head).  igate, fgate: the gates' columns of the projection (head h at column h), row stride ld.
+// m_slots float32 [slots, heads].  decay, gain, floor_ float32 [tokens, heads].
+template <typename T, typename W>
+__global__ void __launch_bounds__(128)
+mlstm_gates_kernel(const T* __restrict__ igate, const T* __restrict__ fgate, int ld, const W* __restrict__ i_bias,
+                   const W* __restrict__ f_bias, float cap, float* __restrict__ m_slots, const int* __restrict__ seg_start,
+                   const int* __restrict__ seg_len, const int* __restrict__ seg_row, int n_heads, float* __restrict__ decay,
+                   float* __restrict__ gain, float* __restrict__ floor_) {
+    __shared__ float2 gates[4][32];       // a warp's 32 tokens: (log forget gate, log input gate)
+    __shared__ float after[4][33];        // the maximum before the first of them and after each
+    qil_wait_for_producer();
+    qil_release_consumer();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int head = blockIdx.x * 4 + warp, seg = blockIdx.y;
+    if (head >= n_heads) return;
+    const int first = seg_start[seg], count = seg_len[seg], row = seg_row[seg];
+    const float bi = to_f32<W>(i_bias[head]), bf = to_f32<W>(f_bias[head]);
+    float m = m_slots[(size_t)row * n_heads + head];
+    for (int t0 = 0; t0 < count; t0 += 32) {
+        const int nb = count - t0 < 32 ? count - t0 : 32;
+        float fl = 0.f, il = 0.f;
+        if (lane < nb) {
+            const size_t at = (size_t)(first + t0 + lane) * ld + head;
+            il = cap * tanhf((to_f32<T>(igate[at]) + bi) / cap);
+            const float z = cap * tanhf((to_f32<T>(fgate[at]) + bf) / cap);
+            fl = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+        }
+        __syncwarp();                     // the last round's maxima have been read
+        gates[warp][lane] = make_float2(fl, il);
+        if (lane == 0) after[warp][0] = m;
+        __syncwarp();
+        for (int j = 0; j < nb; ++j) {    // every lane walks the chain: no broadcast at its end
+            const float2 g = gates[warp][j];
+            m = fmaxf(g.x + m, g.y);
+            if (lane == 0) after[warp][j + 1] = m;
+        }
+        __syncwarp();
+        if (lane < nb) {
+            const float before = after[warp][lane], now = after[warp][lane + 1];
+            const size_t at = (size_t)(first + t0 + lane) * n_heads + head;
+            decay[at] = expf(fl + before - now);
+            gain[at] = expf(il - now);
+            floor_[at] = expf(-now);
+        }
+    }
+    if (lane == 0) m_slots[(size_t)row * n_heads + head] = m;
+}
+
+extern "C" int qil_mlstm_gates(const void* igate, const void* fgate, int ld, const void* i_bias, const void* f_bias, float cap,
+                               float* m_slots, const int* seg_start, const int* seg_len, const int* seg_row, int n_segments,
+                               int n_heads, float* decay, float* gain, float* floor_, int act_dtype, int weight_dtype,
+                               cudaStream_t stream) {
+    if (n_segments <= 0) return 0;
+    if (n_heads <= 0 || !(cap > 0.f) || n_segments > 65535) QIL_REFUSE("mlstm_gates: heads %d cap %g segments %d", n_heads, (double)cap, n_segments);
+    QIL_DISPATCH_2(act_dtype, weight_dtype,
+        qil_launch_chained(mlstm_gates_kernel<T, W>, dim3((n_heads + 3) / 4, n_segments), dim3(128), 0, stream, (const T*)igate,
+                           (const T*)fgate, ld, (const W*)i_bias, (const W*)f_bias, cap, m_slots, seg_start, seg_len, seg_row,
+                           n_heads, decay, gain, floor_));
+    QIL_CHECK_LAUNCH();
+}
+
+// raw float32 [tokens, heads, e + 1]: a head's e outputs and n . q behind them.  A warp per (token, head).
+template <typename T, typename W>
+__global__ void __launch_bounds__(256)
+mlstm_finish_kernel(const float* __restrict__ raw, const float* __restrict__ floor_, const T* __restrict__ g, int ld,
+                    const W* __restrict__ norm_w, float eps, int n_pairs, int n_heads, int e, T* __restrict__ out) {
+    qil_wait_for_producer();
+    qil_release_consumer();
+    const int lane = threadIdx.x & 31;
+    const size_t pair = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (pair >= (size_t)n_pairs) return;
+    const size_t token = pair / n_heads;
+    const int head = (int)(pair % n_heads);
+    const float* o = raw + pair * (e + 1);
+    const float size = fmaxf(fabsf(o[e]), floor_[pair]) + 1e-6f;
+    float ss = 0.f;
+    for (int c = lane; c < e; c += 32) { const float v = o[c] / size; ss = fmaf(v, v, ss); }
+    ss = warp_sum(ss);
+    const float scale = 1.0f / sqrtf(ss / (float)e + eps);
+    for (int c = lane; c < e; c += 32) {
+        const float gate = to_f32<T>(g[token * ld + head * e + c]);
+        out[pair * e + c] = from_f32<T>(o[c] / size * scale * to_f32<W>(norm_w[head * e + c]) * (1.f / (1.f + expf(-gate))));
+    }
+}
+
+extern "C" int qil_mlstm_finish(const float* raw, const float* floor_, const void* g, int ld, const void* norm_w, float eps,
+                                int n_tokens, int n_heads, int e, void* out, int act_dtype, int weight_dtype,
+                                cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (n_heads <= 0 || e <= 0 || (long long)n_tokens * n_heads > 2000000000ll) QIL_REFUSE("mlstm_finish: heads %d values %d", n_heads, e);
+    const int n_pairs = n_tokens * n_heads;
+    QIL_DISPATCH_2(act_dtype, weight_dtype,
+        qil_launch_chained(mlstm_finish_kernel<T, W>, dim3((n_pairs + 7) / 8), dim3(256), 0, stream, raw, floor_, (const T*)g, ld,
+                           (const W*)norm_w, eps, n_pairs, n_heads, e, (T*)out));
     QIL_CHECK_LAUNCH();
 }

@@ -22,8 +22,13 @@
 //   route, mode 1   scores = softmax over all outputs of the router; the choice goes by score + correction[e],
 //                   the weights are the chosen scores alone, divided by their sum (+ 1e-20), times weight_scale.
 //   route, mode 2   as mode 1, but the chosen scores are the weights as they are (times weight_scale): no division.
+//   route, mode 3   scores = sigmoid of every output by itself; the largest (score + correction) are chosen and weigh as
+//                   they are (times weight_scale).  Without corrections the choice goes by the logits: the same order, and
+//                   scores that round to one do not tie.
 //                   One more row behind the router's (`gate_logit`) is a dot product that is handed out as it is:
 //                   the logit of a gate, one number per token, for an expert that every token uses.
+//   input weights   the routing weight multiplies the expert's input instead of its output: W (w x) = w (W x), so gate_up
+//                   scales its float32 sums before the activation and down leaves its sums as they are.
 //   experts         without a gate matrix: h = act(A W_up[e]^T) with act the squared relu (kind 3), silu or gelu.
 //   identity        router outputs from `n_experts` on name no expert: grouping skips them and combine adds
 //                   weight * x, the token's own row.
@@ -60,7 +65,15 @@ __device__ __forceinline__ void moe_select(float* logits, float* choice, float* 
     if (gate_logit != nullptr) {
         if (lane == 0) gate_logit[token] = logits[n_outputs];
     }
-    if (mode >= 1) {
+    if (mode == 3) {
+        for (int e = lane; e < n_outputs; e += 32) {
+            const float z = logits[e], small = expf(-fabsf(z));
+            const float score = z >= 0.f ? 1.f / (1.f + small) : small / (1.f + small);
+            logits[e] = score;
+            choice[e] = correction != nullptr ? score + correction[e] : z;
+        }
+        __syncwarp();
+    } else if (mode >= 1) {
         // softmax over all outputs; the choice by score + correction, the weights from the scores alone
         float peak = -INFINITY;
         for (int e = lane; e < n_outputs; e += 32) peak = fmaxf(peak, logits[e]);
@@ -74,6 +87,8 @@ __device__ __forceinline__ void moe_select(float* logits, float* choice, float* 
             choice[e] = score + (correction != nullptr ? correction[e] : 0.f);
         }
         __syncwarp();
+    }
+    if (mode >= 1) {
         float picked = 0.f;
         for (int k = 0; k < top; ++k) {
             float best = -INFINITY;
@@ -99,8 +114,8 @@ __device__ __forceinline__ void moe_select(float* logits, float* choice, float* 
         }
         for (int k = lane; k < top; k += 32) {
             chosen[token * top + k] = sel_at[k];
-            // mode 2: the chosen scores weigh their experts as they are, not divided by their sum
-            weights[token * top + k] = (mode == 2 ? sel_p[k] : sel_p[k] / (picked + 1e-20f)) * weight_scale;
+            // modes 2 and 3: the chosen scores weigh their experts as they are, not divided by their sum
+            weights[token * top + k] = (mode >= 2 ? sel_p[k] : sel_p[k] / (picked + 1e-20f)) * weight_scale;
         }
         return;
     }
@@ -413,18 +428,19 @@ moe_expert_gemm_kernel(const T* __restrict__ A, int lda, const W* __restrict__ w
     for (int i = 0; i < 4; ++i) {
         const int r = ty * 4 + i;
         if (r >= rows) continue;
-        const int pair = UP ? 0 : sorted_pairs[row0 + r];
-        const float scale = UP ? 1.f : pair_weight[pair];
+        // pair_weight: of the output (down), or of the input (up products); null: one
+        const int pair = (!UP || pair_weight != nullptr) ? sorted_pairs[row0 + r] : 0;
+        const float scale = pair_weight != nullptr ? pair_weight[pair] : 1.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
             if (n >= n_out) continue;
             if (DUAL) {
                 // the products are rounded to the activation type first, as a projection's output is
-                const float g = round_to<T>(acc0[i][j]), u = round_to<T>(acc1[i][j]);
+                const float g = round_to<T>(scale * acc0[i][j]), u = round_to<T>(scale * acc1[i][j]);
                 hidden[(size_t)(row0 + r) * n_out + n] = from_f32<T>(expert_activation(kind, g, u, limit, alpha));
             } else if (UP) {
-                hidden[(size_t)(row0 + r) * n_out + n] = from_f32<T>(expert_plain_activation(kind, round_to<T>(acc0[i][j])));
+                hidden[(size_t)(row0 + r) * n_out + n] = from_f32<T>(expert_plain_activation(kind, round_to<T>(scale * acc0[i][j])));
             } else {
                 y[(size_t)pair * n_out + n] = scale * acc0[i][j];
             }
@@ -560,8 +576,8 @@ moe_expert_mma_kernel(const bf16* __restrict__ A, int lda, const bf16* __restric
         for (int half = 0; half < 2; ++half) {
             const int r = wm + m * 16 + (lane >> 2) + half * 8;
             if (r >= rows) continue;
-            const int pair = UP ? 0 : sorted_pairs[row0 + r];
-            const float scale = UP ? 1.f : pair_weight[pair];
+            const int pair = (!UP || pair_weight != nullptr) ? sorted_pairs[row0 + r] : 0;
+            const float scale = pair_weight != nullptr ? pair_weight[pair] : 1.f;
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) {
 #pragma unroll
@@ -569,11 +585,11 @@ moe_expert_mma_kernel(const bf16* __restrict__ A, int lda, const bf16* __restric
                     const int n = n0 + wn + nt * 8 + (lane & 3) * 2 + e;
                     if (n >= n_out) continue;
                     if (DUAL) {
-                        const float g = round_to<bf16>(acc0[m][nt][half * 2 + e]), u = round_to<bf16>(acc1[m][nt][half * 2 + e]);
+                        const float g = round_to<bf16>(scale * acc0[m][nt][half * 2 + e]), u = round_to<bf16>(scale * acc1[m][nt][half * 2 + e]);
                         hidden[(size_t)(row0 + r) * n_out + n] = __float2bfloat16_rn(expert_activation(kind, g, u, limit, alpha));
                     } else if (UP) {
                         hidden[(size_t)(row0 + r) * n_out + n] =
-                            __float2bfloat16_rn(expert_plain_activation(kind, round_to<bf16>(acc0[m][nt][half * 2 + e])));
+                            __float2bfloat16_rn(expert_plain_activation(kind, round_to<bf16>(scale * acc0[m][nt][half * 2 + e])));
                     } else {
                         y[(size_t)pair * n_out + n] = scale * acc0[m][nt][half * 2 + e];
                     }
@@ -699,7 +715,7 @@ extern "C" int qil_moe_route(const void* x, const void* router, const void* bias
     if (n_experts <= 0 || n_experts + (gate_logit != nullptr ? 1 : 0) > MOE_MAX_EXPERTS || top <= 0 || top > n_experts
         || top > MOE_MAX_TOP || width <= 0)
         QIL_REFUSE("moe_route: %d experts (at most %d), %d of them per token, width %d", n_experts, MOE_MAX_EXPERTS, top, width);
-    if (mode < 0 || mode > 2) QIL_REFUSE("moe_route: mode %d", mode);
+    if (mode < 0 || mode > 3) QIL_REFUSE("moe_route: mode %d", mode);
     if (gate_logit != nullptr && bias != nullptr) QIL_REFUSE("moe_route: a gate row goes without router biases");
     if (n_tokens >= 64 && width % 8 == 0 && (((uintptr_t)x | (uintptr_t)router) & 15) == 0) {
         QIL_DISPATCH_2(act_dtype, weight_dtype,
@@ -737,8 +753,9 @@ extern "C" int qil_moe_group(const int* chosen, int n_pairs, int n_experts, int*
 
 extern "C" int qil_moe_gate_up(const void* x, int lda, const void* gate_w, const void* up_w, const int* tiles,
                                const int* info, int max_tiles, const int* sorted_pairs, int top, void* hidden,
-                               int n_out, int K, int kind, float limit, float alpha, int act_dtype, int weight_dtype,
-                               cudaStream_t stream) {
+                               int n_out, int K, int kind, float limit, float alpha, const float* input_weight,
+                               int act_dtype, int weight_dtype, cudaStream_t stream) {
+    // input_weight: null, or float32 per pair: what the pair's input row is multiplied by
     if (max_tiles <= 0) return 0;
     if (max_tiles > 65535) QIL_REFUSE("moe_gate_up: %d row tiles are too many for one launch", max_tiles);
     dim3 grid((n_out + MOE_BN - 1) / MOE_BN, max_tiles);
@@ -749,11 +766,11 @@ extern "C" int qil_moe_gate_up(const void* x, int lda, const void* gate_w, const
         if (moe_mma_configure()) return -1;
         if (gated)
             qil_launch_chained(moe_expert_mma_kernel<1>, grid, dim3(256), moe_mma_smem(true), stream, (const bf16*)x, lda,
-                               (const bf16*)gate_w, (const bf16*)up_w, tiles, info, sorted_pairs, top, (const float*)nullptr,
+                               (const bf16*)gate_w, (const bf16*)up_w, tiles, info, sorted_pairs, top, input_weight,
                                (bf16*)hidden, (float*)nullptr, n_out, K, kind, limit, alpha);
         else
             qil_launch_chained(moe_expert_mma_kernel<2>, grid, dim3(256), moe_mma_smem(false), stream, (const bf16*)x, lda,
-                               (const bf16*)gate_w, (const bf16*)nullptr, tiles, info, sorted_pairs, top, (const float*)nullptr,
+                               (const bf16*)gate_w, (const bf16*)nullptr, tiles, info, sorted_pairs, top, input_weight,
                                (bf16*)hidden, (float*)nullptr, n_out, K, kind, limit, alpha);
         QIL_CHECK_LAUNCH();
     }
@@ -761,12 +778,12 @@ extern "C" int qil_moe_gate_up(const void* x, int lda, const void* gate_w, const
     if (gated)
         QIL_DISPATCH_2(act_dtype, weight_dtype,
             (qil_launch_chained(moe_expert_gemm_kernel<T, W, 1>, grid, dim3(256), 0, stream, (const T*)x, lda,
-                                (const W*)gate_w, (const W*)up_w, tiles, info, sorted_pairs, top, (const float*)nullptr,
+                                (const W*)gate_w, (const W*)up_w, tiles, info, sorted_pairs, top, input_weight,
                                 (T*)hidden, (float*)nullptr, n_out, K, kind, limit, alpha)));
     else
         QIL_DISPATCH_2(act_dtype, weight_dtype,
             (qil_launch_chained(moe_expert_gemm_kernel<T, W, 2>, grid, dim3(256), 0, stream, (const T*)x, lda,
-                                (const W*)gate_w, (const W*)nullptr, tiles, info, sorted_pairs, top, (const float*)nullptr,
+                                (const W*)gate_w, (const W*)nullptr, tiles, info, sorted_pairs, top, input_weight,
                                 (T*)hidden, (float*)nullptr, n_out, K, kind, limit, alpha)));
     QIL_CHECK_LAUNCH();
 }

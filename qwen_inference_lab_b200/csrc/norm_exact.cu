@@ -384,3 +384,179 @@ extern "C" int qil_norm_join(void* x, int x_dtype, const float* a, const void* w
 #undef QIL_JOIN_ARGS
     QIL_CHECK_LAUNCH();
 }
+
+// Several branches of one layer join the stream at once (a layer whose sublayers read the same normed row), and the
+// norm of whoever reads the stream next rides along:
+//   x += sum_k scale_k * b_k + sum_s y[row * top + s],   rows = norm(x; next_w)   (rows optional; without next_w: x rounded)
+// b_k: up to four float32 branches [N, width]; y (optional): float32 rows of a token's `top` routed experts.  norm as in
+// norm_join.  float32 arithmetic; every sum in the order of the arguments, every reduction a fixed tree over one row.
+#define JOIN_MOST 4
+struct JoinBranches {
+    const float* b[JOIN_MOST];
+    float scale[JOIN_MOST];
+    int n;
+    const float* y;
+    int top;
+};
+
+template <typename T> __device__ __forceinline__ float4 join_load4(const T* p);
+template <> __device__ __forceinline__ float4 join_load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 join_load4<bf16>(const bf16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+__device__ __forceinline__ void join_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void join_store4(bf16* p, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 raw;
+    raw.x = *reinterpret_cast<const unsigned*>(&lo);
+    raw.y = *reinterpret_cast<const unsigned*>(&hi);
+    *reinterpret_cast<uint2*>(p) = raw;
+}
+
+// Rows of up to 1024 * V4 values, a multiple of four, held in registers: 16 bytes a load.
+template <typename TX, typename W, typename TO, int V4>
+__global__ void __launch_bounds__(256)
+branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, const W* __restrict__ next_w, float next_eps,
+                        int next_center, TO* __restrict__ rows) {
+    __shared__ float scratch[32];
+    qil_wait_for_producer();
+    qil_release_consumer();
+    const size_t row = blockIdx.x;
+    TX* dst = x + row * width;
+    float4 v[V4];
+    float sum = 0.f;
+#pragma unroll
+    for (int c = 0; c < V4; ++c) {
+        const int col = (threadIdx.x + c * 256) * 4;
+        v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (col >= width) continue;
+        float4 add = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int k = 0; k < JOIN_MOST; ++k) {
+            if (k >= in.n) break;
+            const float4 b = *reinterpret_cast<const float4*>(in.b[k] + row * width + col);
+            add.x = fmaf(in.scale[k], b.x, add.x); add.y = fmaf(in.scale[k], b.y, add.y);
+            add.z = fmaf(in.scale[k], b.z, add.z); add.w = fmaf(in.scale[k], b.w, add.w);
+        }
+        if (in.y != nullptr)
+            for (int t = 0; t < in.top; ++t) {
+                const float4 b = *reinterpret_cast<const float4*>(in.y + (row * in.top + t) * width + col);
+                add.x += b.x; add.y += b.y; add.z += b.z; add.w += b.w;
+            }
+        float4 now = join_load4<TX>(dst + col);
+        now.x += add.x; now.y += add.y; now.z += add.z; now.w += add.w;
+        now.x = round_to<TX>(now.x); now.y = round_to<TX>(now.y); now.z = round_to<TX>(now.z); now.w = round_to<TX>(now.w);
+        join_store4(dst + col, now);
+        v[c] = now;
+        sum += (now.x + now.y) + (now.z + now.w);
+    }
+    if (rows == nullptr) return;
+    TO* out = rows + row * width;
+    if (next_w == nullptr) {
+#pragma unroll
+        for (int c = 0; c < V4; ++c) {
+            const int col = (threadIdx.x + c * 256) * 4;
+            if (col < width) join_store4(out + col, v[c]);
+        }
+        return;
+    }
+    float mean = 0.f;
+    if (next_center) mean = block_sum(sum, scratch) / (float)width;
+    float sq = 0.f;
+#pragma unroll
+    for (int c = 0; c < V4; ++c) {
+        if ((threadIdx.x + c * 256) * 4 >= width) continue;
+        v[c].x -= mean; v[c].y -= mean; v[c].z -= mean; v[c].w -= mean;
+        sq = fmaf(v[c].x, v[c].x, sq); sq = fmaf(v[c].y, v[c].y, sq);
+        sq = fmaf(v[c].z, v[c].z, sq); sq = fmaf(v[c].w, v[c].w, sq);
+    }
+    sq = block_sum(sq, scratch);
+    const float scale = 1.0f / sqrtf(sq / (float)width + next_eps);
+#pragma unroll
+    for (int c = 0; c < V4; ++c) {
+        const int col = (threadIdx.x + c * 256) * 4;
+        if (col >= width) continue;
+        const float4 w = join_load4<W>(next_w + col);
+        join_store4(out + col, make_float4(v[c].x * scale * w.x, v[c].y * scale * w.y, v[c].z * scale * w.z, v[c].w * scale * w.w));
+    }
+}
+
+// Any width: the stream's row is read back by the threads that wrote it.
+template <typename TX, typename W, typename TO>
+__global__ void __launch_bounds__(256)
+branch_join_kernel(TX* __restrict__ x, JoinBranches in, int width, const W* __restrict__ next_w, float next_eps,
+                   int next_center, TO* __restrict__ rows) {
+    __shared__ float scratch[32];
+    qil_wait_for_producer();
+    qil_release_consumer();
+    const size_t row = blockIdx.x;
+    TX* dst = x + row * width;
+    float sum = 0.f;
+    for (int i = threadIdx.x; i < width; i += 256) {
+        float add = 0.f;
+        for (int k = 0; k < in.n; ++k) add = fmaf(in.scale[k], in.b[k][row * width + i], add);
+        if (in.y != nullptr)
+            for (int t = 0; t < in.top; ++t) add += in.y[(row * in.top + t) * width + i];
+        const TX next = from_f32<TX>(to_f32<TX>(dst[i]) + add);
+        dst[i] = next;
+        sum += to_f32<TX>(next);
+    }
+    if (rows == nullptr) return;
+    TO* out = rows + row * width;
+    if (next_w == nullptr) {
+        for (int i = threadIdx.x; i < width; i += 256) out[i] = from_f32<TO>(to_f32<TX>(dst[i]));
+        return;
+    }
+    float mean = 0.f;
+    if (next_center) mean = block_sum(sum, scratch) / (float)width;
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < width; i += 256) {
+        const float v = to_f32<TX>(dst[i]) - mean;
+        sq = fmaf(v, v, sq);
+    }
+    sq = block_sum(sq, scratch);
+    const float scale = 1.0f / sqrtf(sq / (float)width + next_eps);
+    for (int i = threadIdx.x; i < width; i += 256)
+        out[i] = from_f32<TO>((to_f32<TX>(dst[i]) - mean) * scale * to_f32<W>(next_w[i]));
+}
+
+// branches: host array of n device pointers; scales: host array of n.
+extern "C" int qil_branch_join(void* x, int x_dtype, const float* const* branches, const float* scales, int n_branches,
+                               const float* y, int top, int n_rows, int width, const void* next_w, int weight_dtype,
+                               float next_eps, int next_center, void* rows, int rows_dtype, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (width <= 0 || n_branches < 0 || n_branches > JOIN_MOST || (y != nullptr && top < 1))
+        QIL_REFUSE("branch_join: width %d, %d branches (at most %d), %d experts a token", width, n_branches, JOIN_MOST, top);
+    if (next_w != nullptr && rows == nullptr) QIL_REFUSE("branch_join: the next norm needs rows to write");
+    JoinBranches in = {};
+    uintptr_t bits = (uintptr_t)x | (uintptr_t)y | (uintptr_t)next_w | (uintptr_t)rows;
+    for (int k = 0; k < n_branches; ++k) { in.b[k] = branches[k]; in.scale[k] = scales[k]; bits |= (uintptr_t)branches[k]; }
+    in.n = n_branches; in.y = y; in.top = top;
+    const bool wide = width % 4 == 0 && (bits & 15) == 0;
+#define QIL_JOIN_ARGS(TX, WT, TO) \
+    dim3(n_rows), dim3(256), 0, stream, (TX*)x, in, width, (const WT*)next_w, next_eps, next_center, (TO*)rows
+#define QIL_JOIN_GO(TX, WT, TO)                                                                                       \
+    do {                                                                                                              \
+        if (wide && width <= 1024) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 1>, QIL_JOIN_ARGS(TX, WT, TO));      \
+        else if (wide && width <= 2048) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 2>, QIL_JOIN_ARGS(TX, WT, TO)); \
+        else if (wide && width <= 4096) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 4>, QIL_JOIN_ARGS(TX, WT, TO)); \
+        else qil_launch_chained(branch_join_kernel<TX, WT, TO>, QIL_JOIN_ARGS(TX, WT, TO));                           \
+    } while (0)
+#define QIL_JOIN_O(TX, WT)                                                                                            \
+    do { if (rows_dtype == QIL_F32) QIL_JOIN_GO(TX, WT, float); else QIL_JOIN_GO(TX, WT, bf16); } while (0)
+#define QIL_JOIN_W(TX)                                                                                                \
+    do { if (weight_dtype == QIL_F32) QIL_JOIN_O(TX, float); else QIL_JOIN_O(TX, bf16); } while (0)
+    if (next_w != nullptr && weight_dtype != QIL_F32 && weight_dtype != QIL_BF16) QIL_REFUSE("branch_join: weight dtype %d", weight_dtype);
+    if (rows != nullptr && rows_dtype != QIL_F32 && rows_dtype != QIL_BF16) QIL_REFUSE("branch_join: rows dtype %d", rows_dtype);
+    if (x_dtype == QIL_F32) QIL_JOIN_W(float);
+    else if (x_dtype == QIL_BF16) QIL_JOIN_W(bf16);
+    else QIL_REFUSE("branch_join: stream dtype %d", x_dtype);
+#undef QIL_JOIN_W
+#undef QIL_JOIN_O
+#undef QIL_JOIN_GO
+#undef QIL_JOIN_ARGS
+    QIL_CHECK_LAUNCH();
+}

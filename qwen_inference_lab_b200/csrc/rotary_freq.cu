@@ -10,7 +10,9 @@
 // qk_rotate_store: q [Hq * d], k [Hkv * d], v [Hkv * e] are column ranges of one row-major buffer (a stacked
 // projection).  Optionally q and k are first divided by their root mean square over the WHOLE projection (all
 // heads at once) and multiplied by a weight per element (float32 arithmetic), or (per_head) every head by its own
-// root mean square over its d dimensions, with one weight of d that all heads share; then every head is rotated;
+// root mean square over its d dimensions, with one weight of d that all heads share (per_head 2: without a weight, in
+// which case it makes no difference whether a head is normed before or after it is turned: a rotation keeps the sum
+// of squares); then every head is rotated;
 // queries go to q_out, keys and values into the request's page (a page holds its key rows
 // [kv_head][slot][d] followed by its value rows [kv_head][slot][e]).
 //
@@ -92,7 +94,7 @@ qk_rotate_store_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col,
         for (int i = tid; i < q_width; i += 256) { const float x = to_f32<T>(row[q_col + i]); vals[i] = x; sq = fmaf(x, x, sq); }
         for (int i = tid; i < k_width; i += 256) { const float x = to_f32<T>(row[k_col + i]); vals[q_width + i] = x; sk = fmaf(x, x, sk); }
     }
-    if (q_norm_w != nullptr && per_head) {
+    if (per_head == 2 || (q_norm_w != nullptr && per_head)) {
         // a warp per head: the head's sum of squares by a fixed tree over the lanes, whatever else the step holds
         __syncthreads();
         const int lane = tid & 31, warp = tid >> 5;
@@ -103,7 +105,7 @@ qk_rotate_store_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col,
             for (int j = lane; j < d; j += 32) ss = fmaf(v[j], v[j], ss);
             ss = warp_sum(ss);
             const float r = 1.0f / sqrtf(ss / (float)d + eps);
-            for (int j = lane; j < d; j += 32) v[j] = v[j] * r * to_f32<W>(w[j]);
+            for (int j = lane; j < d; j += 32) v[j] = per_head == 2 ? v[j] * r : v[j] * r * to_f32<W>(w[j]);
         }
     } else if (q_norm_w != nullptr) {
         sq = block_sum(sq, scratch);

@@ -139,16 +139,23 @@ def _need(tensor, name, dtype=None, ndim=None):
         raise KernelError(f"{name} must have {ndim} dimensions, got {tuple(tensor.shape)}")
 
 
-def embed_gather(table, ids, out, scale=1.0):
-    """out[r] = table[ids[r]] * scale cast to out's dtype (a float32 product, one rounding).  table [V,H]; ids int32
-    [N]; out [N,H]."""
+def embed_gather(table, ids, out, scale=1.0, pos_table=None, positions=None):
+    """out[r] = table[ids[r]] * scale (+ pos_table[positions[r]]) cast to out's dtype (float32 arithmetic, one rounding).
+    table [V,H]; ids int32 [N]; out [N,H]; pos_table [P,H] of the table's dtype and positions int32 [N], or neither."""
     _need(table, "table", ndim=2); _need(ids, "ids", torch.int32, 1); _need(out, "out", ndim=2)
     if out.shape != (ids.shape[0], table.shape[1]):
         raise KernelError(f"embed_gather: out {tuple(out.shape)} for ids {tuple(ids.shape)} table {tuple(table.shape)}")
+    if (pos_table is None) != (positions is None):
+        raise KernelError("embed_gather: a table of positions goes with the tokens' positions")
+    if pos_table is not None:
+        _need(pos_table, "pos_table", table.dtype, 2); _need(positions, "positions", torch.int32, 1)
+        if pos_table.shape[1] != table.shape[1] or positions.shape != ids.shape:
+            raise KernelError("embed_gather: the table of positions or the positions do not fit")
     lib = core()
     _check(lib, lib.qil_embed_gather(_p(table), c_int(dtype_code(table.dtype)), _p(ids), _p(out),
                                      c_int(dtype_code(out.dtype)), c_int(ids.shape[0]), c_int(table.shape[1]),
-                                     c_int(table.shape[0]), c_float(scale), _stream()), "embed_gather")
+                                     c_int(table.shape[0]), c_float(scale), _p(pos_table), _p(positions),
+                                     c_int(pos_table.shape[0] if pos_table is not None else 0), _stream()), "embed_gather")
     return out
 
 
@@ -579,20 +586,27 @@ def short_conv_store(u, taps_weight, state, q_out, kv_cache, positions, token_ro
     return q_out
 
 
-def gated_activation(gate_up, kind, *, limit=0.0, alpha=1.0, pairs8=False, out=None):
+def gated_activation(gate_up, kind, *, limit=0.0, alpha=1.0, pairs8=False, out=None, column=0, width=None):
     """out = act(gate) * f(up) for rows of [gate columns, up columns]: ``kind`` is ``silu``, ``gelu_tanh``, or
-    ``clamped_swish``: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + 1)."""
+    ``clamped_swish``: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + 1).
+    ``width``: of the gate (and of the up) columns, which begin at ``column`` of a wider buffer; None: the whole buffer."""
     _need(gate_up, "gate_up", ndim=2)
-    if gate_up.shape[1] % 2:
+    if width is None and gate_up.shape[1] % 2:
         raise KernelError("gated_activation: the input's width must be even (gate columns then up columns)")
     if kind not in ACTIVATIONS:
         raise KernelError(f"gated_activation: unknown kind {kind!r} (known: {sorted(ACTIVATIONS)})")
-    width = gate_up.shape[1] // 2
+    if width is None:
+        width = gate_up.shape[1] // 2
+    if column < 0 or column + 2 * width > gate_up.shape[1]:
+        raise KernelError("gated_activation: the columns lie outside the buffer")
     if out is None:
         out = torch.empty((gate_up.shape[0], width), dtype=gate_up.dtype, device=gate_up.device)
     _need(out, "out", gate_up.dtype, 2)
+    if out.shape != (gate_up.shape[0], width):
+        raise KernelError("gated_activation: out has the wrong shape")
     lib = core()
-    _check(lib, lib.qil_gated_activation(_p(gate_up), _p(out), c_int(gate_up.shape[0]), c_int(width),
+    _check(lib, lib.qil_gated_activation(c_void_p(gate_up.data_ptr() + column * gate_up.element_size()),
+                                         c_longlong(gate_up.shape[1]), _p(out), c_int(gate_up.shape[0]), c_int(width),
                                          c_int(dtype_code(gate_up.dtype)), c_int(1 if pairs8 else 0),
                                          c_int(ACTIVATIONS[kind]), c_float(limit), c_float(alpha), _stream()),
            "gated_activation")
@@ -653,7 +667,7 @@ def gla_decay(projected, low_column, a2, a2_bias, tau, out=None):
 
 def gla_scan(projected, columns, alpha, q_scale, norm_weight, eps, state, seg_start, seg_len, seg_row,
              n_segments, n_heads, d, e, out, scratch=None, mode=GLA_WHOLE, decay_product=None, head_decay=None,
-             silu_inputs=False, raw_only=False):
+             silu_inputs="", raw_only=False, tied_gate=None, token_scalars=None, ones=False):
     """Gated linear attention over segments of a step (see csrc/gla_scan.cu for the equations).
 
     ``projected`` [N, width]: the stacked projection; ``columns`` = (q, k, v, g) first columns in it
@@ -666,28 +680,53 @@ def gla_scan(projected, columns, alpha, q_scale, norm_weight, eps, state, seg_st
     the state.
 
     ``head_decay`` float32 [n_heads] (with ``alpha`` None): one fixed decay per head instead of a decay per token and
-    key channel.  ``silu_inputs``: silu on q, k and v as they are read.  ``raw_only``: the un-normed outputs go to
-    ``scratch`` whatever the sizes and nothing is normed or gated here (``out`` and ``norm_weight`` may be None)."""
+    key channel.  ``silu_inputs``: those of "q", "k", "v" that pass silu as they are read ("qkv": all).  ``raw_only``:
+    the un-normed outputs go to ``scratch`` whatever the sizes and nothing is normed or gated here (``out`` and
+    ``norm_weight`` may be None).  A column g of None: normed, not gated.
+    ``tied_gate`` = (bias, lower bound), each [n_heads * d] of one dtype: k's columns are a gate's logits z, a channel
+    decays by f = l + (1 - l) sigmoid(z + b) and is written with 1 - f.  ``token_scalars`` = (decay, gain), float32
+    [N, n_heads]: a decay and a gain of k per token and head (``mlstm_gates``).  ``ones``: the state has a last column
+    whose value is one (``e`` counts it, v's columns do not; raw outputs only)."""
     _need(projected, "projected", ndim=2)
     if not raw_only:
         _need(out, "out", projected.dtype, 2); _need(norm_weight, "norm_weight", ndim=1)
     elif scratch is None and mode != GLA_OWN_STATE:
         raise KernelError("gla_scan: raw outputs need the scratch buffer")
-    if (alpha is None) == (head_decay is None):
-        raise KernelError("gla_scan: give the decays per token or one per head")
+    if sum(source is not None for source in (alpha, head_decay, tied_gate, token_scalars)) != 1:
+        raise KernelError("gla_scan: give one source of decays: per token, per head, a tied gate, or per token and head")
+    if set(silu_inputs) - set("qkv"):
+        raise KernelError(f"gla_scan: silu on {silu_inputs!r}")
+    gate_bias, gate_lower = tied_gate if tied_gate is not None else (None, None)
+    token_decay, token_gain = token_scalars if token_scalars is not None else (None, None)
+    param_dtype = norm_weight.dtype if norm_weight is not None else torch.float32
+    if tied_gate is not None:
+        _need(gate_bias, "the gate's bias", ndim=1); _need(gate_lower, "the gate's lower bound", gate_bias.dtype, 1)
+        if gate_bias.shape[0] != n_heads * d or gate_lower.shape[0] != n_heads * d:
+            raise KernelError("gla_scan: one bias and one lower bound per head and key channel")
+        if not raw_only and param_dtype != gate_bias.dtype:
+            raise KernelError("gla_scan: the gate's bias and the norm's weight share a dtype")
+        param_dtype = gate_bias.dtype
+    if ones and not raw_only:
+        raise KernelError("gla_scan: a column of ones goes with raw outputs")
+    if token_scalars is not None:
+        for t in token_scalars:
+            _need(t, "token scalars", torch.float32, 2)
+            if t.shape != (projected.shape[0], n_heads):
+                raise KernelError("gla_scan: one decay and one gain per token and head")
     if alpha is not None:
         _need(alpha, "alpha", torch.float32, 2)
-    else:
+    elif head_decay is not None:
         _need(head_decay, "head_decay", torch.float32, 1)
         if head_decay.shape[0] != n_heads:
             raise KernelError("gla_scan: one decay per head")
     _need(state, "state", torch.float32, 4)
     n, ld = projected.shape
-    q_at, k_at, v_at, g_at = (int(c) for c in columns[:4])
+    q_at, k_at, v_at, g_at = (int(c) if c is not None else None for c in columns[:4])
+    values = e - 1 if ones else e
     if ((alpha is not None and alpha.shape != (n, n_heads * d)) or tuple(state.shape[1:]) != (n_heads, d, e)
             or (not raw_only and (norm_weight.shape[0] != e or out.shape != (n, n_heads * e)))):
         raise KernelError("gla_scan: shapes do not match the head counts")
-    if max(q_at + n_heads * d, k_at + n_heads * d, v_at + n_heads * e, g_at + n_heads * e) > ld:
+    if max(q_at + n_heads * d, k_at + n_heads * d, v_at + n_heads * values, (g_at or 0) + n_heads * values) > ld:
         raise KernelError("gla_scan: a column range lies outside the projection")
     for t in (seg_start, seg_len, seg_row):
         _need(t, "segments", torch.int32, 1)
@@ -706,11 +745,12 @@ def gla_scan(projected, columns, alpha, q_scale, norm_weight, eps, state, seg_st
     lib = core()
     _check(lib, lib.qil_gla_scan(
         c_void_p(base + q_at * size), c_void_p(base + k_at * size), c_void_p(base + v_at * size),
-        c_void_p(base + g_at * size), _p(alpha), _p(head_decay), c_int(1 if silu_inputs else 0),
+        c_void_p(base + g_at * size if g_at is not None else 0), _p(alpha), _p(head_decay), _p(gate_bias), _p(gate_lower),
+        _p(token_decay), _p(token_gain), c_int(sum(1 << "qkv".index(c) for c in set(silu_inputs))), c_int(1 if ones else 0),
         c_int(1 if raw_only else 0), c_int(ld), c_float(q_scale), _p(norm_weight), c_float(eps), _p(state),
         _p(seg_start), _p(seg_len), _p(seg_row), c_int(n_segments), c_int(n), c_int(n_heads), c_int(d), c_int(e),
         _p(scratch), _p(out), c_int(mode), _p(decay_product), c_int(dtype_code(projected.dtype)),
-        c_int(dtype_code(norm_weight.dtype) if norm_weight is not None else F32), _stream()), "gla_scan")
+        c_int(dtype_code(param_dtype)), _stream()), "gla_scan")
     return out
 
 
@@ -731,16 +771,60 @@ def gla_carry(chunk_state, decay_product, slots, carry, n_carries):
 
 def gla_norm_gate(scratch, projected, gate_column, norm_weight, eps, n_heads, e, out):
     """out = rmsnorm over each head's e values of ``scratch`` (weight ``norm_weight``) * silu(gate), the gate
-    being the columns of ``projected`` from ``gate_column`` on."""
+    being the columns of ``projected`` from ``gate_column`` on (None: no gate)."""
     _need(scratch, "scratch", torch.float32); _need(projected, "projected", ndim=2); _need(out, "out", projected.dtype, 2)
     n = projected.shape[0]
-    if out.shape != (n, n_heads * e) or scratch.numel() < n * n_heads * e or gate_column + n_heads * e > projected.shape[1]:
+    if out.shape != (n, n_heads * e) or scratch.numel() < n * n_heads * e or (gate_column or 0) + n_heads * e > projected.shape[1]:
         raise KernelError("gla_norm_gate: shapes do not fit together")
     lib = core()
-    _check(lib, lib.qil_gla_norm_gate(_p(scratch), c_void_p(projected.data_ptr() + gate_column * projected.element_size()),
+    gate = 0 if gate_column is None else projected.data_ptr() + gate_column * projected.element_size()
+    _check(lib, lib.qil_gla_norm_gate(_p(scratch), c_void_p(gate),
                                       c_int(projected.shape[1]), _p(norm_weight), c_float(eps), c_int(n), c_int(n_heads),
                                       c_int(e), _p(out), c_int(dtype_code(projected.dtype)),
                                       c_int(dtype_code(norm_weight.dtype)), _stream()), "gla_norm_gate")
+    return out
+
+
+def mlstm_gates(projected, columns, biases, cap, m_slots, seg_start, seg_len, seg_row, n_segments):
+    """(decay, gain, floor), each float32 [N, heads], of a matrix memory's two gates over a step's segments (see
+    csrc/gla_scan.cu).  ``columns`` = (input gate, forget gate): the first of each gate's ``heads`` columns of
+    ``projected``; ``biases`` = (input, forget) [heads]; ``m_slots`` float32 [slots, heads]: the running maximum per
+    request, read and written at the rows ``seg_row`` names."""
+    _need(projected, "projected", ndim=2); _need(m_slots, "m_slots", torch.float32, 2)
+    n, ld = projected.shape
+    heads = m_slots.shape[1]
+    _need(biases[0], "the input gate's bias", ndim=1); _need(biases[1], "the forget gate's bias", biases[0].dtype, 1)
+    if any(b.shape[0] != heads for b in biases) or any(c < 0 or c + heads > ld for c in columns):
+        raise KernelError("mlstm_gates: shapes do not fit together")
+    for t in (seg_start, seg_len, seg_row):
+        _need(t, "segments", torch.int32, 1)
+        if t.shape[0] < n_segments:
+            raise KernelError("mlstm_gates: fewer segment entries than segments")
+    decay, gain, floor = (torch.empty((n, heads), dtype=torch.float32, device=projected.device) for _ in range(3))
+    size, base, lib = projected.element_size(), projected.data_ptr(), core()
+    _check(lib, lib.qil_mlstm_gates(c_void_p(base + columns[0] * size), c_void_p(base + columns[1] * size), c_int(ld),
+                                    _p(biases[0]), _p(biases[1]), c_float(cap), _p(m_slots), _p(seg_start), _p(seg_len),
+                                    _p(seg_row), c_int(n_segments), c_int(heads), _p(decay), _p(gain), _p(floor),
+                                    c_int(dtype_code(projected.dtype)), c_int(dtype_code(biases[0].dtype)), _stream()),
+           "mlstm_gates")
+    return decay, gain, floor
+
+
+def mlstm_finish(raw, floor, projected, gate_column, norm_weight, eps, out):
+    """out [N, heads * e] from the raw outputs of a matrix memory (float32 [N, heads, e + 1]: e outputs and n . q): a
+    head's outputs over max(|n . q|, floor) + 1e-6, over their own root mean square, times ``norm_weight`` [heads * e]
+    and sigmoid of the gate's columns of ``projected``."""
+    _need(raw, "raw", torch.float32, 3); _need(floor, "floor", torch.float32, 2); _need(projected, "projected", ndim=2)
+    _need(out, "out", projected.dtype, 2); _need(norm_weight, "norm_weight", ndim=1)
+    n, heads, e = raw.shape[0], raw.shape[1], raw.shape[2] - 1
+    if floor.shape != (n, heads) or out.shape != (n, heads * e) or norm_weight.shape[0] != heads * e \
+            or projected.shape[0] != n or gate_column < 0 or gate_column + heads * e > projected.shape[1]:
+        raise KernelError("mlstm_finish: shapes do not fit together")
+    lib = core()
+    _check(lib, lib.qil_mlstm_finish(_p(raw), _p(floor), c_void_p(projected.data_ptr() + gate_column * projected.element_size()),
+                                     c_int(projected.shape[1]), _p(norm_weight), c_float(eps), c_int(n), c_int(heads),
+                                     c_int(e), _p(out), c_int(dtype_code(projected.dtype)),
+                                     c_int(dtype_code(norm_weight.dtype)), _stream()), "mlstm_finish")
     return out
 
 
@@ -825,6 +909,48 @@ def norm_join(x, branch, weight, eps, kind="rms", *, next_weight=None, next_eps=
     return x
 
 
+JOIN_MOST_BRANCHES = 4
+
+
+def branch_join(x, branches, *, routed=None, next_weight=None, next_eps=0.0, next_kind="rms", rows=None):
+    """x += sum of scale * branch over ``branches`` (pairs of a float32 [N, width] and a number, at most four) + the sum
+    of each row's routed experts (``routed`` float32 [N, top, width]), row by row in float32; x [N, width] is the stream
+    (float32 or bfloat16), updated in place.  ``rows`` and ``next_weight``: as in :func:`norm_join`."""
+    _need(x, "x", ndim=2)
+    n, width = x.shape
+    if len(branches) > JOIN_MOST_BRANCHES:
+        raise KernelError(f"branch_join: {len(branches)} branches are more than {JOIN_MOST_BRANCHES}")
+    for branch, _ in branches:
+        _need(branch, "branch", torch.float32, 2)
+        if branch.shape != x.shape:
+            raise KernelError("branch_join: shapes differ")
+    top = 0
+    if routed is not None:
+        _need(routed, "routed", torch.float32, 3)
+        top = routed.shape[1]
+        if routed.shape != (n, top, width):
+            raise KernelError("branch_join: the experts' rows have another shape")
+    if next_kind not in NORM_KINDS:
+        raise KernelError(f"branch_join: a norm is one of {sorted(NORM_KINDS)}")
+    if rows is not None:
+        _need(rows, "rows", ndim=2)
+        if rows.shape != x.shape:
+            raise KernelError("branch_join: the next sublayer's rows have another shape")
+    if next_weight is not None:
+        _need(next_weight, "next_weight", ndim=1)
+        if rows is None or next_weight.shape[0] != width:
+            raise KernelError("branch_join: the next norm needs rows to write and a weight of the stream's width")
+    pointers = (c_void_p * JOIN_MOST_BRANCHES)(*(branch.data_ptr() for branch, _ in branches))
+    scales = (c_float * JOIN_MOST_BRANCHES)(*(float(scale) for _, scale in branches))
+    lib = core()
+    _check(lib, lib.qil_branch_join(_p(x), c_int(dtype_code(x.dtype)), pointers, scales, c_int(len(branches)), _p(routed),
+                                    c_int(top), c_int(n), c_int(width), _p(next_weight),
+                                    c_int(dtype_code(next_weight.dtype) if next_weight is not None else F32),
+                                    c_float(next_eps), c_int(NORM_KINDS[next_kind]), _p(rows),
+                                    c_int(dtype_code(rows.dtype) if rows is not None else F32), _stream()), "branch_join")
+    return x
+
+
 def scale_inplace(x, factor):
     """x *= factor for float32 ``x`` (logits)."""
     _need(x, "x", torch.float32)
@@ -846,13 +972,15 @@ def _check_rotation(freq, rot_dims, layout, most, what):
 
 
 def qk_rotate_store(proj, columns, q_out, kv_cache, q_norm_w, k_norm_w, eps, freq, rot_dims, layout, positions,
-                    token_row, block_table, n_q_heads, n_kv_heads, head_dim, v_dim, page_size, per_head=False):
+                    token_row, block_table, n_q_heads, n_kv_heads, head_dim, v_dim, page_size, per_head=False,
+                    unit_heads=False):
     """The tail of a q/k/v projection with rotation from frequencies (float32 angles position * freq[i]).
 
     ``proj`` [N, width] holds q, k, v from the columns ``columns`` = (q, k, v) on.  With ``q_norm_w`` [Hq * d] and
     ``k_norm_w`` [Hkv * d], q and k are first divided by their root mean square over the whole projection (all heads
     at once) and multiplied by the weight; with ``per_head`` every head is normed by itself over its d dimensions and
-    the weights are [d], one for all query heads and one for all key heads.  The values are copied as projected from
+    the weights are [d], one for all query heads and one for all key heads.  ``unit_heads`` (no weights): every head is
+    divided by its own root mean square and that is all, which a rotation before or after does not change.  The values are copied as projected from
     column v on: giving the keys' column there stores the keys as projected, before norm and rotation, as values.
     Then the first ``rot_dims`` dimensions of every head are rotated
     (``layout``: ``ROTARY_HALVES`` or ``ROTARY_INTERLEAVED``); queries go to ``q_out`` [N, Hq * d], keys and values
@@ -865,6 +993,8 @@ def qk_rotate_store(proj, columns, q_out, kv_cache, q_norm_w, k_norm_w, eps, fre
         raise KernelError("qk_rotate_store: shapes do not match the head counts")
     _check_rotation(freq, rot_dims, layout, head_dim, "qk_rotate_store")
     norm_code = F32
+    if unit_heads and (q_norm_w is not None or k_norm_w is not None):
+        raise KernelError("qk_rotate_store: heads of unit size have no norm weights")
     if q_norm_w is not None:
         _need(q_norm_w, "q_norm_w", ndim=1)
         if n_kv_heads:
@@ -887,8 +1017,8 @@ def qk_rotate_store(proj, columns, q_out, kv_cache, q_norm_w, k_norm_w, eps, fre
         _p(q_norm_w), _p(k_norm_w), c_int(norm_code), c_float(eps), _p(freq), c_int(rot_dims), c_int(layout),
         _p(positions), _p(token_row), _p(block_table if n_kv_heads else None),
         c_int(block_table.shape[1] if n_kv_heads else 0), c_int(n), c_int(n_q_heads), c_int(n_kv_heads), c_int(head_dim),
-        c_int(v_dim), c_int(page_size), c_int(num_pages), c_int(dtype_code(proj.dtype)), c_int(1 if per_head else 0),
-        _stream()), "qk_rotate_store")
+        c_int(v_dim), c_int(page_size), c_int(num_pages), c_int(dtype_code(proj.dtype)), 
+        c_int(2 if unit_heads else 1 if per_head else 0), _stream()), "qk_rotate_store")
     return q_out
 
 
@@ -972,13 +1102,14 @@ def head_gate(y, width, gate, gate_column):
 
 
 def moe_route(x, router, bias, top, *, softmax_all=False, correction=None, weight_scale=1.0, gate_row=False,
-              renormalize=True):
+              renormalize=True, sigmoid=False):
     """(chosen int32 [N, top], weights float32 [N, top]): the ``top`` largest of x R^T + b per row (float32
     arithmetic; the lower index wins a tie) and the softmax over those logits alone.
 
     ``softmax_all``: scores are the softmax over all outputs; the choice goes by score + ``correction`` (float32
     [outputs]), the weights are the chosen scores divided by their sum (+ 1e-20), times ``weight_scale``; with
-    ``renormalize=False`` the chosen scores themselves, undivided.
+    ``renormalize=False`` the chosen scores themselves, undivided.  ``sigmoid``: scores are the sigmoid of every output by
+    itself; chosen by score + ``correction``, weights the chosen scores as they are, times ``weight_scale``.
     ``gate_row``: the last row of ``router`` is not an output but a gate's weights: its dot products are returned
     as a third result, float32 [N]."""
     _need(x, "x", ndim=2); _need(router, "router", ndim=2)
@@ -988,7 +1119,9 @@ def moe_route(x, router, bias, top, *, softmax_all=False, correction=None, weigh
         _need(bias, "bias", router.dtype, 1)
     n = x.shape[0]
     outputs = router.shape[0] - (1 if gate_row else 0)
-    if not renormalize and not softmax_all:
+    if sigmoid and softmax_all:
+        raise KernelError("moe_route: scores are a softmax or sigmoids, not both")
+    if not renormalize and not softmax_all and not sigmoid:
         raise KernelError("moe_route: only scores of a softmax over all outputs can stay as they are")
     if correction is not None:
         _need(correction, "correction", torch.float32, 1)
@@ -999,16 +1132,19 @@ def moe_route(x, router, bias, top, *, softmax_all=False, correction=None, weigh
     gate = torch.empty((n,), dtype=torch.float32, device=x.device) if gate_row else None
     lib = core()
     _check(lib, lib.qil_moe_route(_p(x), _p(router), _p(bias), c_int(n), c_int(x.shape[1]), c_int(outputs),
-                                  c_int(top), _p(chosen), _p(weights), c_int((1 if renormalize else 2) if softmax_all else 0),
-                                  _p(correction),
+                                  c_int(top), _p(chosen), _p(weights), 
+                                  c_int(3 if sigmoid else (1 if renormalize else 2) if softmax_all else 0), _p(correction),
                                   c_float(weight_scale), _p(gate), c_int(dtype_code(x.dtype)),
                                   c_int(dtype_code(router.dtype)), _stream()), "moe_route")
     return (chosen, weights, gate) if gate_row else (chosen, weights)
 
 
 def moe_experts(x, chosen, weights, gate_w, up_w, down_w, kind, *, limit=0.0, alpha=1.0, residual=None, out=None,
-                identity=False, extra=None, extra_gate=None, col_scale=None):
+                identity=False, extra=None, extra_gate=None, col_scale=None, weigh_input=False, combine=True):
     """out = residual + sum over a token's chosen experts of weight * down_e(act(gate_e x, up_e x)).
+
+    ``weigh_input``: the weight multiplies the expert's input instead, down_e(act(gate_e (weight x), up_e (weight x))).
+    ``combine=False``: returns the experts' rows one by one, float32 [N, top, width], for a kernel that sums them itself.
 
     gate_w, up_w [E, ff, width]; down_w [E, width, ff]; ``kind`` as in ``gated_activation`` (``silu`` or
     ``clamped_swish``).  ``residual`` and ``out`` [N, width] share a dtype (the residual stream's).
@@ -1037,9 +1173,12 @@ def moe_experts(x, chosen, weights, gate_w, up_w, down_w, kind, *, limit=0.0, al
     if col_scale is not None:
         _need(col_scale, "col_scale", torch.float32, 1)
     stream_dtype = residual.dtype if residual is not None else (out.dtype if out is not None else x.dtype)
-    if out is None:
+    if not combine and (residual is not None or out is not None or identity or extra is not None or col_scale is not None):
+        raise KernelError("moe_experts: the experts' own rows come without anything that is added to them")
+    if out is None and combine:
         out = torch.empty((n, width), dtype=stream_dtype, device=x.device)
-    _need(out, "out", stream_dtype, 2)
+    if combine:
+        _need(out, "out", stream_dtype, 2)
     if residual is not None:
         _need(residual, "residual", stream_dtype, 2)
     lib = core()
@@ -1055,10 +1194,13 @@ def moe_experts(x, chosen, weights, gate_w, up_w, down_w, kind, *, limit=0.0, al
                                   c_int(max_tiles), _stream()), "moe_group", kernels=1 if pairs <= lib.qil_moe_one_block_pairs() else 2)
     _check(lib, lib.qil_moe_gate_up(_p(x), c_int(width), _p(gate_w), _p(up_w), _p(tiles), _p(info), c_int(max_tiles),
                                     _p(sorted_pairs), c_int(top), _p(hidden), c_int(ff), c_int(width),
-                                    c_int(ACTIVATIONS[kind]), c_float(limit), c_float(alpha), act, wt, _stream()),
-           "moe_gate_up")
+                                    c_int(ACTIVATIONS[kind]), c_float(limit), c_float(alpha),
+                                    _p(weights if weigh_input else None), act, wt, _stream()), "moe_gate_up")
     _check(lib, lib.qil_moe_down(_p(hidden), _p(down_w), _p(tiles), _p(info), c_int(max_tiles), _p(sorted_pairs),
-                                 _p(weights), _p(y), c_int(width), c_int(ff), act, wt, _stream()), "moe_down")
+                                 _p(None if weigh_input else weights), _p(y), c_int(width), c_int(ff), act, wt,
+                                 _stream()), "moe_down")
+    if not combine:
+        return y.view(n, top, width)
     _check(lib, lib.qil_moe_combine(_p(y), _p(residual), _p(out), c_int(n), c_int(width), c_int(top),
                                     c_int(dtype_code(stream_dtype)), _p(chosen), _p(weights), _p(x if identity else None),
                                     c_int(dtype_code(x.dtype)), c_int(experts), _p(extra), _p(extra_gate), _p(col_scale),

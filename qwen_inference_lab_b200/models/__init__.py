@@ -4,3 +4,4 @@ from . import virulix  # noqa: F401
 from . import debisun  # noqa: F401
 from . import larolorn  # noqa: F401
 from . import gogotar  # noqa: F401
+from . import lotazen  # noqa: F401

@@ -31,7 +31,9 @@ their root mean square over the whole projection, all heads at once, and multipl
 ``names["q_norm"]``, ``names["k_norm"]``, before the rotation) go with every option above but the per-head norms,
 the short convolution and the query temperature.  With such a rotation ``qk_norm_eps`` norms every head by itself
 (one weight of head_dim for all query heads, one for all key heads) in the same kernel.  ``values_from_keys``: there
-is no value projection; a position's value is its key as projected, before norm and rotation.  ``head_gate``: the
+is no value projection; a position's value is its key as projected, before norm and rotation.  ``unit_qk_norm_eps``
+divides every q and k head by its own root mean square without a weight (after the rotation or before it, which is
+the same: a rotation keeps the sum of squares); such a layer may have a sliding window.  ``head_gate``: the
 name of a [query heads, hidden] matrix G; head h's output is multiplied by sigmoid(G x)_h before the output
 projection (G's rows ride behind the keys' in the stacked projection).
 """
@@ -94,7 +96,7 @@ class GroupedQueryAttention(Mixer):
                  v_head_dim=None, distance_slopes=None, q_temperature=None, out_bias=None,
                  suffixes=(".weight", ".bias"), conv_taps=0, conv_suffix=".conv", softcap=0.0, distance_bias=None,
                  chunk=0, sink=False, whole_qk_norm_eps=None, norm_suffix=".weight", values_from_keys=False,
-                 head_gate=None):
+                 head_gate=None, unit_qk_norm_eps=None):
         if n_q_heads % n_kv_heads:
             raise ValueError(f"{n_q_heads} query heads do not divide into {n_kv_heads} kv heads")
         self.hidden_size, self.head_dim = int(hidden_size), int(head_dim)
@@ -115,7 +117,11 @@ class GroupedQueryAttention(Mixer):
         self.learned_sink = sink == "learned"
         self.whole_qk_norm_eps = None if whole_qk_norm_eps is None else float(whole_qk_norm_eps)
         # the projection's tail is the kernel that norms over the whole projection and rotates by frequencies
-        self.frequency_tail = isinstance(position, RotaryFrequencies) or self.whole_qk_norm_eps is not None
+        self.unit_qk_norm_eps = None if unit_qk_norm_eps is None else float(unit_qk_norm_eps)
+        if self.unit_qk_norm_eps is not None and (qk_norm_eps is not None or self.whole_qk_norm_eps is not None):
+            raise ValueError("heads of unit size go without another q/k norm")
+        self.frequency_tail = isinstance(position, RotaryFrequencies) or self.whole_qk_norm_eps is not None \
+            or self.unit_qk_norm_eps is not None
         if self.frequency_tail and (conv_taps or q_temperature is not None
                                     or (qk_norm_eps is not None and self.whole_qk_norm_eps is not None)
                                     or (position is not None and not isinstance(position, RotaryFrequencies))):
@@ -243,14 +249,18 @@ class GroupedQueryAttention(Mixer):
     def takes_out_scale(self):
         return self.plain_tail or self.frequency_tail
 
-    def forward(self, ctx, x, cache, residual=None, norm=None, out_scale=None, out_float32=False):
+    def input_projections(self):
+        """The products of the mixer's input that may run as part of a wider one (``parts.linear.JointProjection``)."""
+        return [self.qkv] if self.frequency_tail else []
+
+    def forward(self, ctx, x, cache, residual=None, norm=None, out_scale=None, out_float32=False, joint=None):
         """x [N, hidden] -> [N, hidden] (+ residual).  ``cache`` is a KVCacheView (with a short convolution: a
         pair of it and a StateView).  With ``norm`` x is the block's un-normed input and the first projection
-        applies the norm."""
+        applies the norm.  ``joint``: the rows of a product that holds the first projection already."""
         n = x.shape[0]
         n_kv = 0 if self.reads_shared_cache else self.n_kv_heads
         if self.frequency_tail:
-            qkv = self.qkv.forward(ctx, x, norm=norm)
+            qkv, at = self.qkv.columns_of(ctx, x, joint, norm)
             q = ctx.empty((n, self.n_q_heads * self.head_dim))
             q_width, k_width = self.n_q_heads * self.head_dim, n_kv * self.head_dim
             rotation = self.position
@@ -259,19 +269,19 @@ class GroupedQueryAttention(Mixer):
             k_weight = self.k_norm if per_head else self.whole_k_norm
             # keys as values: the value rows are copied from the keys' columns, as projected
             v_column = q_width if self.values_from_keys else q_width + k_width
-            ops.qk_rotate_store(qkv, (0, q_width, v_column), q, cache.pages,
+            ops.qk_rotate_store(qkv, (at, at + q_width, at + v_column), q, cache.pages,
                                 q_weight.data if q_weight is not None else None,
                                 k_weight.data if k_weight is not None else None,
-                                (self.qk_norm_eps if per_head else self.whole_qk_norm_eps) or 0.0,
+                                (self.qk_norm_eps if per_head else self.whole_qk_norm_eps or self.unit_qk_norm_eps) or 0.0,
                                 rotation.freq if rotation is not None else None,
                                 rotation.rotary_dim if rotation is not None else 0,
                                 rotation.layout if rotation is not None else 0, ctx.positions, ctx.token_row,
                                 cache.block_table, self.n_q_heads, n_kv, self.head_dim, self.v_head_dim, cache.page_size,
-                                per_head=per_head)
+                                per_head=per_head, unit_heads=self.unit_qk_norm_eps is not None)
             attended = ctx.empty((n, self.n_q_heads * self.v_head_dim))
             self._attend(ctx, q, cache, attended)
             if self.head_gate:
-                ops.head_gate(attended, self.v_head_dim, qkv, qkv.shape[1] - self.n_q_heads)
+                ops.head_gate(attended, self.v_head_dim, qkv, at + self.qkv.out_features - self.n_q_heads)
             return self.out.forward(ctx, attended, residual=residual, out_scale=out_scale, out_float32=out_float32)
         if out_float32:
             raise ValueError("a float32 result is given by the layers that rotate by frequencies only")

@@ -139,6 +139,11 @@ class Norm(Part):
         may apply itself, else None."""
         return None
 
+    def as_join(self):
+        """(weight [width], eps, kind) if this norm is one that the kernels which join branches to the stream can
+        apply to the new stream (``kernels.ops.NORM_KINDS``), else None."""
+        return None
+
 
 class PositionEncoding(Part):
     rotary_dim = 0

@@ -13,6 +13,7 @@ of the block's.  And parts that run on the stream after the feed-forward (``afte
 
 :class:`PostNormBlock` is the other arrangement: the sublayers read the stream itself and the norm sits on each
 sublayer's output, x <- x + m * norm1(mixer(x)), x <- x + m * norm2(ff(x)) with a fixed multiplier m.
+:class:`ParallelBlock` has one norm whose output both sublayers read: x <- x + mixer(h) + ff(h), h = norm(x).
 :class:`SandwichNormBlock` norms on both sides of each sublayer: x <- x + post1(mixer(pre1 x)), x <- x + post2(ff(pre2 x)).
 """
 from __future__ import annotations
@@ -21,6 +22,7 @@ import torch
 
 from ..kernels import ops
 from .base import Param, Part
+from .linear import JointProjection
 
 
 class PreNormBlock(Part):
@@ -195,7 +197,7 @@ class SandwichNormBlock(Part):
     def forward(self, ctx, x, cache):
         """x [N, width] is the residual stream; updated in place and returned."""
         pending = ctx.extras.pop("pending_join", None)
-        if pending is not None and pending.stream is x and pending.weight.dtype == self.pre1.data.dtype:
+        if isinstance(pending, PendingJoin) and pending.stream is x and pending.weight.dtype == self.pre1.data.dtype:
             rows = ctx.empty(x.shape)
             ops.norm_join(x, pending.branch, pending.weight, pending.eps, pending.kind, next_weight=self.pre1.data,
                           next_eps=self.eps, next_kind=self.kind, rows=rows)
@@ -225,8 +227,75 @@ class PendingJoin:
         ops.norm_join(self.stream, self.branch, self.weight, self.eps, self.kind)
 
 
+class ParallelBlock(Part):
+    """x <- x + (mixer(h) + ff(h)) with h = norm(x): one norm, both sublayers read its output.
+
+    Since they share their input, the first projections of all sublayers that can (``input_projections()``) run as one
+    product (:class:`JointProjection`).  The sublayers give their results unsummed (``branches``: float32 rows with a
+    scale each; a routed feed-forward also its experts' rows), and ``ops.branch_join`` adds them all to the stream and
+    norms the new stream in the same kernel.  That norm is the next block's: a block leaves its branches in
+    ``ctx.extras["pending_join"]`` and the next block of this kind joins them together with its own norm; the decoder
+    settles what is left before anyone else reads the stream.  ``feed_forward`` may be None."""
+    takes_pending_join = True
+    graph_safe = True
+
+    def __init__(self, norm, mixer, feed_forward):
+        self.norm, self.mixer, self.feed_forward = norm, mixer, feed_forward
+        self.input = JointProjection([p for part in (mixer, feed_forward) if hasattr(part, "input_projections")
+                                      for p in part.input_projections()])
+
+    def children(self):
+        return [part for part in (self.norm, self.mixer, self.feed_forward) if part is not None]
+
+    def finalize(self, device, dtype):
+        super().finalize(device, dtype)
+        self.input.join()
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def forward(self, ctx, x, cache):
+        """x [N, width] is the residual stream; updated in place (by the next reader of the stream) and returned."""
+        pending = ctx.extras.pop("pending_join", None)
+        how = self.norm.as_join()
+        if isinstance(pending, PendingBranches) and pending.stream is x and how is not None:
+            rows = ctx.empty(x.shape)
+            pending.settle(next_weight=how[0], next_eps=how[1], next_kind=how[2], rows=rows)
+        else:
+            if pending is not None:
+                pending.settle()
+            rows = self.norm.forward(ctx, x)
+        joint = self.input.forward_joint(ctx, rows)
+        options = {} if joint is None else dict(joint=joint)
+        if hasattr(self.mixer, "branches"):
+            branches = list(self.mixer.branches(ctx, rows, cache, **options))
+        else:
+            branches = [(self.mixer.forward(ctx, rows, cache, out_float32=True, **options), 1.0)]
+        routed = None
+        if self.feed_forward is not None:
+            if hasattr(self.feed_forward, "branches"):
+                more, routed = self.feed_forward.branches(ctx, rows, **options)
+                branches += more
+            else:
+                branches.append((self.feed_forward.forward(ctx, rows, out_float32=True, **options), 1.0))
+        ctx.extras["pending_join"] = PendingBranches(x, branches, routed)
+        return x
+
+
+class PendingBranches:
+    """Branches that have not joined their stream yet: stream += sum of scale * branch + the experts' rows."""
+    __slots__ = ("stream", "branches", "routed")
+
+    def __init__(self, stream, branches, routed):
+        self.stream, self.branches, self.routed = stream, branches, routed
+
+    def settle(self, **norm):
+        ops.branch_join(self.stream, self.branches, routed=self.routed, **norm)
+
+
 def settle_stream(ctx):
-    """Join what a block left unjoined (see :class:`SandwichNormBlock`); for whoever reads the stream next."""
+    """Join what a block left unjoined (see :class:`SandwichNormBlock`, :class:`ParallelBlock`); for whoever reads the
+    stream next."""
     pending = ctx.extras.pop("pending_join", None)
     if pending is not None:
         pending.settle()

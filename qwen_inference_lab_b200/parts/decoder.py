@@ -33,19 +33,30 @@ class LayerCall:
 class TokenEmbedding(Part):
     graph_safe = True
 
-    def __init__(self, vocab_size, hidden_size, *, name, suffix=".weight", scale=1.0):
-        """``scale``: what a row of the table is multiplied by as it enters the stream."""
+    def __init__(self, vocab_size, hidden_size, *, name, suffix=".weight", scale=1.0, positions=None):
+        """``scale``: what a row of the table is multiplied by as it enters the stream.  ``positions`` = (name, count): a
+        learned vector per position, added unscaled (the model's requests are then at most ``count`` tokens long)."""
         self.vocab_size, self.hidden_size, self.name, self.suffix = int(vocab_size), int(hidden_size), name, suffix
         self.scale = float(scale)
         self.weight = Param((vocab_size, hidden_size))
+        self.positions = None if positions is None else Param((positions[1], hidden_size))
+        self.positions_name = None if positions is None else positions[0] + suffix
 
     def named_params(self):
-        return {self.name + self.suffix: self.weight}
+        if self.positions is None:
+            return {self.name + self.suffix: self.weight}
+        return {self.name + self.suffix: self.weight, self.positions_name: self.positions}
+
+    def finalize(self, device, dtype):
+        if self.positions is not None:         # the kernel reads both tables as one dtype
+            self.positions.data = self.positions.data.to(self.weight.data.dtype)
 
     def forward(self, ctx, token_ids):
         """Rows of the table in the dtype of the residual stream (the activations' unless the model keeps
         its stream in float32)."""
         out = ctx.empty((token_ids.shape[0], self.hidden_size), dtype=ctx.stream_dtype)
+        if self.positions is not None:
+            return ops.embed_gather(self.weight.data, token_ids, out, self.scale, self.positions.data, ctx.positions)
         return ops.embed_gather(self.weight.data, token_ids, out, self.scale)
 
 
@@ -64,6 +75,9 @@ class DecoderModel(Part):
         self.embedding, self.layers, self.final_norm, self.head = embedding, list(layers), final_norm, head
         self.order = [call if isinstance(call, LayerCall) else LayerCall(*call) for call in order]
         self.max_positions = int(max_positions)
+        table = getattr(embedding, "positions", None)
+        if table is not None and table.shape[0] < self.max_positions:
+            raise ValueError(f"{self.max_positions} positions of a model whose table holds {table.shape[0]}")
         self.vocab_size = embedding.vocab_size
         self.device = None
         self.dtype = None

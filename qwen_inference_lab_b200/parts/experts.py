@@ -17,6 +17,9 @@ Options for other designs of routing:
                            correction (``names["correction"]``), the weights are the chosen scores themselves,
                            divided by their sum (+ 1e-20) and multiplied by ``weight_scale``;
                            ``renormalize=False`` leaves out the division: the chosen scores are the weights
+``routing="sigmoid"``      scores = sigmoid of every output by itself, chosen by score + correction, the chosen scores
+                           are the weights (times ``weight_scale``)
+``weigh_input``            the weight multiplies the expert's input, not its output: down_e(act(gate_e (w x), up_e (w x)))
 ``identity``               so many further outputs of the router, behind the experts', name no expert: a token
                            that chooses one gets weight * x, its own input
 ``gated=False``            experts without a gate matrix: down_e(act(up_e x)), ``activation`` one without a gate
@@ -39,20 +42,23 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, hidden_size, expert_size, n_experts, top, *, names, activation="silu", limit=0.0, alpha=1.0,
                  shared=None, routing="softmax_chosen", weight_scale=1.0, identity=0, gated=True, shared_gate=None,
-                 renormalize=True):
+                 renormalize=True, weigh_input=False):
         self.hidden_size, self.expert_size = int(hidden_size), int(expert_size)
         self.n_experts, self.top, self.identity = int(n_experts), int(top), int(identity)
         if self.identity < 0 or not 1 <= self.top <= self.n_experts + self.identity:
             raise ValueError(f"{top} of {n_experts} experts (+ {identity} that hand the input through) per token")
-        if routing not in ("softmax_chosen", "softmax_all"):
+        if routing not in ("softmax_chosen", "softmax_all", "sigmoid"):
             raise ValueError(f"unknown routing {routing!r}")
         if activation not in (("silu", "clamped_swish") if gated else ops.PLAIN_ACTIVATIONS):
             raise ValueError(f"activation {activation!r} does not fit experts {'with' if gated else 'without'} a gate matrix")
         self.activation, self.limit, self.alpha = activation, float(limit), float(alpha)
         self.routing, self.weight_scale, self.gated = routing, float(weight_scale), bool(gated)
         self.renormalize = bool(renormalize)
-        if not self.renormalize and routing != "softmax_all":
+        if not self.renormalize and routing == "softmax_chosen":
             raise ValueError("only the scores of a softmax over all outputs can weigh the experts undivided")
+        self.weigh_input = bool(weigh_input)
+        if self.weigh_input and self.identity:
+            raise ValueError("a weighed input goes without outputs that hand the input through")
         self.shared = shared
         outputs = self.n_experts + self.identity
         self.router = Param((outputs, hidden_size), std=0.5)
@@ -108,7 +114,7 @@ class RoutedExperts(FeedForward):
             if residual is not None or out_scale is not None:
                 raise ValueError("a float32 result goes without a residual")
             return self._forward_general(ctx, x, None, None, torch.float32)
-        if self.routing == "softmax_all" or self.identity or not self.gated or self.shared_gate is not None \
+        if self.routing != "softmax_chosen" or self.weigh_input or self.identity or not self.gated or self.shared_gate is not None \
                 or out_scale is not None:
             return self._forward_general(ctx, x, residual, out_scale)
         chosen, weights = ops.moe_route(x, self.router.data, self.router_bias.data if self.router_bias else None, self.top)
@@ -119,18 +125,38 @@ class RoutedExperts(FeedForward):
             out = self.shared.forward(ctx, x, residual=out)
         return out
 
+    def _route(self, x):
+        return ops.moe_route(x, self._router, self.router_bias.data if self.router_bias else None, self.top,
+                             softmax_all=self.routing == "softmax_all", sigmoid=self.routing == "sigmoid",
+                             correction=self.correction.data if self.correction is not None else None,
+                             weight_scale=self.weight_scale, gate_row=self.shared_gate is not None,
+                             renormalize=self.renormalize)
+
+    def input_projections(self):
+        shared = getattr(self.shared, "input_projections", None)
+        return shared() if shared is not None else []
+
+    def branches(self, ctx, x, joint=None):
+        """(branches, routed): what joins the stream, unsummed (``kernels.ops.branch_join``): the shared expert's float32
+        rows and the chosen experts' rows [N, top, hidden]."""
+        if self.identity or self.shared_gate is not None:
+            return [(self._forward_general(ctx, x, None, None, torch.float32), 1.0)], None
+        chosen, weights = self._route(x)[:2]
+        shared = [(self.shared.forward(ctx, x, out_float32=True, **({} if joint is None else dict(joint=joint))), 1.0)] \
+            if self.shared is not None else []
+        first, second = (self._gate, self._up) if self.gated else (self._up, None)
+        return shared, ops.moe_experts(x, chosen, weights, first, second, self._down, self.activation, limit=self.limit,
+                                       alpha=self.alpha, weigh_input=self.weigh_input, combine=False)
+
     def _forward_general(self, ctx, x, residual, out_scale, out_dtype=None):
         """Every option at once: the shared expert's float32 output, its gate and the output scale go into the
         kernel that sums a token's experts onto the residual."""
-        routed = ops.moe_route(x, self._router, self.router_bias.data if self.router_bias else None, self.top,
-                               softmax_all=self.routing == "softmax_all",
-                               correction=self.correction.data if self.correction is not None else None,
-                               weight_scale=self.weight_scale, gate_row=self.shared_gate is not None,
-                               renormalize=self.renormalize)
+        routed = self._route(x)
         chosen, weights = routed[:2]
         extra = self.shared.forward(ctx, x, out_float32=True) if self.shared is not None else None
         first, second = (self._gate, self._up) if self.gated else (self._up, None)
         return ops.moe_experts(x, chosen, weights, first, second, self._down, self.activation, limit=self.limit,
                                alpha=self.alpha, residual=residual, identity=self.identity > 0, extra=extra,
+                               weigh_input=self.weigh_input,
                                extra_gate=routed[2] if self.shared_gate is not None else None, col_scale=out_scale,
                                out=None if residual is not None else ctx.empty(x.shape, dtype=out_dtype or ctx.stream_dtype))

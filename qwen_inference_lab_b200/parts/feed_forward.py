@@ -52,13 +52,18 @@ class GatedMLP(FeedForward):
 
     takes_norm = True
 
-    def forward(self, ctx, x, residual=None, norm=None, out_float32=False):
+    def input_projections(self):
+        """The products of the input that may run as part of a wider one (``parts.linear.JointProjection``)."""
+        return [self.gate_up] if self.activation != "silu" else []
+
+    def forward(self, ctx, x, residual=None, norm=None, out_float32=False, joint=None):
         """With ``norm`` x is the block's un-normed input; a decode step's few rows get the norm inside
         the gate/up kernel, longer steps a norm kernel of their own.  ``out_float32``: the down product's float32
         sums are returned as they are (for a block that norms the branch before it joins the stream)."""
         if self.activation != "silu" or self.bias or out_float32:
-            gate_up = self.gate_up.forward(ctx, x, norm=norm)
-            hidden = ops.gated_activation(gate_up, self.activation, limit=self.limit, alpha=self.alpha, pairs8=self.pairs8)
+            gate_up, at = self.gate_up.columns_of(ctx, x, joint, norm)
+            hidden = ops.gated_activation(gate_up, self.activation, limit=self.limit, alpha=self.alpha, pairs8=self.pairs8,
+                                          column=at, width=self.intermediate_size)
             return self.down.forward(ctx, hidden, residual=residual, out_float32=out_float32)
         rms = norm.as_rms() if norm is not None else None
         if self.pairs8 and ops.small_m_ok(x, self.gate_up._w) and rms is not None and rms[0].dtype == torch.bfloat16:

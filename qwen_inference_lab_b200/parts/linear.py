@@ -182,3 +182,63 @@ class StackedLinear(Linear):
 
     def _bias(self):
         return self._b
+
+    def columns_of(self, ctx, x, joint=None, norm=None):
+        """(buffer, first column) of this projection of ``x``: its place in the rows of a :class:`JointProjection` that
+        has run already, or a product of its own."""
+        if joint is not None and id(self) in joint.first_column:
+            return joint.rows, joint.first_column[id(self)]
+        return self.forward(ctx, x, norm=norm), 0
+
+
+class JointProjection(Linear):
+    """Several :class:`StackedLinear` of the same input (the first projections of sublayers that run side by side), as
+    one product.  It owns no parameters: ``join`` (called once the parts are finalized) lays their stacked weights one
+    below the other, each from a row that is a multiple of ``ALIGN`` on so that every part's columns start on a 16-byte
+    boundary, and leaves the parts views of it: they still run by themselves as well.  Parts with biases or with
+    weights of different dtypes are not joined (``forward_joint`` gives None and every part runs its own product)."""
+    ALIGN = 8
+
+    def __init__(self, projections):
+        self.projections = list(projections)
+        self._w = None
+        self._first = {}
+
+    def named_params(self):
+        return {}
+
+    def finalize(self, device, dtype):
+        pass
+
+    def join(self):
+        weights = [p._weight() for p in self.projections]
+        if len(weights) < 2 or any(p._bias() is not None for p in self.projections) or len({w.dtype for w in weights}) != 1 \
+                or len({w.shape[1] for w in weights}) != 1:
+            return
+        at = 0
+        for projection, w in zip(self.projections, weights):
+            self._first[id(projection)] = at
+            at += -(-w.shape[0] // self.ALIGN) * self.ALIGN
+        self._w = torch.zeros((at, weights[0].shape[1]), dtype=weights[0].dtype, device=weights[0].device)
+        for projection, w in zip(self.projections, weights):
+            first = self._first[id(projection)]
+            self._w[first:first + w.shape[0]] = w
+            projection._w = self._w[first:first + w.shape[0]]
+        self.out_features, self.in_features = self._w.shape
+
+    def _weight(self):
+        return self._w
+
+    def _bias(self):
+        return None
+
+    def forward_joint(self, ctx, x):
+        return None if self._w is None else JointRows(self.forward(ctx, x), self._first)
+
+
+class JointRows:
+    """The rows of a :class:`JointProjection` and the first column of every part's projection in them."""
+    __slots__ = ("rows", "first_column")
+
+    def __init__(self, rows, first_column):
+        self.rows, self.first_column = rows, first_column

@@ -198,7 +198,7 @@ class DecayLinearAttention(Mixer):
         plan = ctx.plans[_PLANNER.key]
         raw = ctx.empty((n, heads * e), dtype=torch.float32)
         common = (projected, self.columns, None, 1.0, None, self.norm_eps)
-        options = dict(head_decay=self._decay, silu_inputs=True, raw_only=True)
+        options = dict(head_decay=self._decay, silu_inputs="qkv", raw_only=True)
         n_short, n_chunks = plan.count["short_start"], plan.count["chunk_start"]
         if n_short:
             ops.gla_scan(*common, cache.slots, plan.array["short_start"], plan.array["short_len"], plan.array["short_row"],
@@ -211,3 +211,183 @@ class DecayLinearAttention(Mixer):
             ops.gla_carry(states, decays, cache.slots, plan.array["carry"], plan.count["carry"] // 3)
             ops.gla_scan(*common, states, *chunk, heads, d, e, None, scratch=raw, mode=ops.GLA_FROM_STATE, **options)
         return raw
+
+
+def _scan_step(ctx, slots, run, sizes):
+    """The recurrence over a step's segments through ``run(state, starts, lens, rows, count, **mode)``: short segments
+    from the request's slot and back, long ones as chunks with a carry (``ScanPlanner``)."""
+    heads, d, e = sizes
+    plan = ctx.plans[_PLANNER.key]
+    n_short, n_chunks = plan.count["short_start"], plan.count["chunk_start"]
+    if n_short:
+        run(slots, plan.array["short_start"], plan.array["short_len"], plan.array["short_row"], n_short)
+    if n_chunks:
+        chunk = (plan.array["chunk_start"], plan.array["chunk_len"], plan.array["chunk_index"], n_chunks)
+        states = ctx.empty((n_chunks, heads, d, e), dtype=torch.float32)
+        decays = ctx.empty((n_chunks, heads, d), dtype=torch.float32)
+        run(states, *chunk, mode=ops.GLA_OWN_STATE, decay_product=decays)
+        ops.gla_carry(states, decays, slots, plan.array["carry"], plan.count["carry"] // 3)
+        run(states, *chunk, mode=ops.GLA_FROM_STATE)
+
+
+class TiedGateLinearAttention(Mixer):
+    """Linear attention whose forget gate also decides what is written (HGRN2); per head, d channels and e values:
+
+        q_t = silu(Wq x_t),  v_t = Wv x_t,  f_t = l + (1 - l) sigmoid(Wf x_t + b)      l, b: one number per channel
+        S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,   o_t = S_t^T q_t                    S_0 = 0, float32
+        y_t = Wo rms_e(o_t; w)                                                          w [e] shared by heads
+
+    q, f and v are one stacked product.  The recurrence is the scan of :class:`GatedLinearAttention`
+    (``kernels.ops.gla_scan``) with the gate made where the scan reads its logits, and the norm inside the scan where a
+    head's values fit one block.
+
+    names: dict with keys q, f, v, o (projection names), lower (the bound's full name) and norm."""
+    graph_safe = True
+
+    def __init__(self, hidden_size, n_heads, key_dim, value_dim, *, norm_eps, names, suffixes=(".weight", ".bias"),
+                 norm_suffix=".weight"):
+        self.hidden_size, self.n_heads = int(hidden_size), int(n_heads)
+        self.key_dim, self.value_dim, self.norm_eps = int(key_dim), int(value_dim), float(norm_eps)
+        kw, vw = self.n_heads * self.key_dim, self.n_heads * self.value_dim
+        self.projection = StackedLinear(hidden_size, [(names["q"], kw), (names["f"], kw), (names["v"], vw)], suffixes=suffixes)
+        self.columns = (0, kw, 2 * kw)
+        self.gate_bias = Param((kw,), init="normal", std=1.0)
+        self.gate_lower = Param((kw,), init="zeros")
+        self.norm_weight = Param((self.value_dim,), init="norm", std=0.05)
+        self._names = {names["f"] + suffixes[1]: self.gate_bias, names["lower"]: self.gate_lower,
+                       names["norm"] + norm_suffix: self.norm_weight}
+        self.out = Linear(vw, hidden_size, name=names["o"], suffixes=suffixes)
+        self._needs_scratch = False
+
+    def named_params(self):
+        return dict(self._names)
+
+    def children(self):
+        return [self.projection, self.out]
+
+    def finalize(self, device, dtype):
+        super().finalize(device, dtype)
+        for param in (self.gate_bias, self.gate_lower, self.norm_weight):      # float32 arithmetic: read as float32
+            param.data = param.data.to(torch.float32).contiguous()
+        self._needs_scratch = ops.gla_scan_needs_scratch(self.key_dim, self.value_dim)
+
+    def cache_spec(self):
+        return StateSpec((self.n_heads, self.key_dim, self.value_dim), torch.float32)
+
+    def step_planners(self):
+        return {**super().step_planners(), _PLANNER.key: _PLANNER}
+
+    def input_projections(self):
+        return [self.projection]
+
+    def forward(self, ctx, x, cache, residual=None, out_float32=False, joint=None):
+        """x [N, hidden] -> [N, hidden] (+ residual); ``cache`` is a StateView with one slot per request row."""
+        projected, at = self.projection.columns_of(ctx, x, joint)
+        mixed = self.scan(ctx, projected, at, cache)
+        return self.out.forward(ctx, mixed, residual=residual, out_float32=out_float32)
+
+    def scan(self, ctx, projected, at, cache):
+        """The recurrence and the norm over the step's segments: columns of ``projected`` from ``at`` on -> [N, heads * e]."""
+        n, sizes = projected.shape[0], (self.n_heads, self.key_dim, self.value_dim)
+        mixed = ctx.empty((n, self.n_heads * self.value_dim))
+        scratch = ctx.empty((n, self.n_heads * self.value_dim), dtype=torch.float32) if self._needs_scratch else None
+        columns = (*(at + c for c in self.columns), None)
+
+        def run(state, starts, lens, rows, count, **mode):
+            ops.gla_scan(projected, columns, None, 1.0, self.norm_weight.data, self.norm_eps, state, starts, lens, rows, count,
+                         *sizes, mixed, scratch=scratch, silu_inputs="q",
+                         tied_gate=(self.gate_bias.data, self.gate_lower.data), **mode)
+
+        _scan_step(ctx, cache.slots, run, sizes)
+        if scratch is not None:
+            ops.gla_norm_gate(scratch, projected, None, self.norm_weight.data, self.norm_eps, self.n_heads, self.value_dim,
+                              mixed)
+        return mixed
+
+
+class MatrixMemory(Mixer):
+    """The matrix memory of xLSTM (mLSTM); per head, d key channels and e values:
+
+        q_t = Wq x_t d^(-1/2),  k_t = Wk x_t,  v_t = Wv x_t
+        i_t = cap tanh((Wi x_t + bi) / cap),  f_t = log sigmoid(cap tanh((Wf x_t + bf) / cap))     one number per head
+        m_t = max(f_t + m_(t-1), i_t)                                                              m_0 = 0
+        S_t = exp(f_t + m_(t-1) - m_t) S_(t-1) + exp(i_t - m_t) k_t v_t^T,   n_t the same with k_t alone
+        o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + 1e-6)
+        y_t = Wo ( rms_e(o_t) * w * sigmoid(Wg x_t) )                              w: one number per value of all heads
+
+    q, k, v, g, i and f are one stacked product.  ``kernels.ops.mlstm_gates`` walks the gates and the running maximum of
+    every segment and leaves a decay, a gain and a floor per token and head; with those the memory is the scan of
+    :class:`GatedLinearAttention` (``kernels.ops.gla_scan``) with a column of ones behind the values, which is n;
+    ``kernels.ops.mlstm_finish`` divides, norms and gates.  State: (S beside n, m), float32.
+
+    names: dict with keys q, k, v, g, i, f, o (projection names) and norm."""
+    graph_safe = True
+
+    def __init__(self, hidden_size, n_heads, key_dim, value_dim, gate_cap, *, norm_eps, names,
+                 suffixes=(".weight", ".bias"), norm_suffix=".weight", q_scale=None):
+        self.hidden_size, self.n_heads = int(hidden_size), int(n_heads)
+        self.key_dim, self.value_dim = int(key_dim), int(value_dim)
+        self.gate_cap, self.norm_eps = float(gate_cap), float(norm_eps)
+        if not self.gate_cap > 0:
+            raise ValueError("the gates' cap must be positive")
+        self.q_scale = float(q_scale) if q_scale is not None else self.key_dim ** -0.5
+        kw, vw = self.n_heads * self.key_dim, self.n_heads * self.value_dim
+        pieces = [("q", kw), ("k", kw), ("v", vw), ("g", vw), ("i", self.n_heads), ("f", self.n_heads)]
+        self.projection = StackedLinear(hidden_size, [(names[k], rows) for k, rows in pieces], suffixes=suffixes)
+        self.columns, at = {}, 0
+        for key, rows in pieces:
+            self.columns[key] = at
+            at += rows
+        self.i_bias = Param((self.n_heads,), init="normal", std=1.0)
+        self.f_bias = Param((self.n_heads,), init="norm", std=1.0)
+        self.norm_weight = Param((vw,), init="norm", std=0.05)
+        self._names = {names["i"] + suffixes[1]: self.i_bias, names["f"] + suffixes[1]: self.f_bias,
+                       names["norm"] + norm_suffix: self.norm_weight}
+        self.out = Linear(vw, hidden_size, name=names["o"], suffixes=suffixes)
+
+    def named_params(self):
+        return dict(self._names)
+
+    def children(self):
+        return [self.projection, self.out]
+
+    def finalize(self, device, dtype):
+        super().finalize(device, dtype)
+        for param in (self.i_bias, self.f_bias, self.norm_weight):
+            param.data = param.data.to(torch.float32).contiguous()
+        ops.gla_scan_needs_scratch(self.key_dim, self.value_dim + 1)       # refuses key sizes the scan cannot hold
+
+    def cache_spec(self):
+        return (StateSpec((self.n_heads, self.key_dim, self.value_dim + 1), torch.float32),
+                StateSpec((self.n_heads,), torch.float32))
+
+    def step_planners(self):
+        return {**super().step_planners(), _PLANNER.key: _PLANNER}
+
+    def input_projections(self):
+        return [self.projection]
+
+    def forward(self, ctx, x, cache, residual=None, out_float32=False, joint=None):
+        """x [N, hidden] -> [N, hidden] (+ residual); ``cache`` is a pair of StateViews (the memory, the maximum)."""
+        projected, at = self.projection.columns_of(ctx, x, joint)
+        mixed = self.scan(ctx, projected, at, cache)
+        return self.out.forward(ctx, mixed, residual=residual, out_float32=out_float32)
+
+    def scan(self, ctx, projected, at, cache):
+        """Gates, recurrence, norm and output gate: columns of ``projected`` from ``at`` on -> [N, heads * e]."""
+        memory, maximum = cache
+        n, sizes = projected.shape[0], (self.n_heads, self.key_dim, self.value_dim + 1)
+        column = {key: at + first for key, first in self.columns.items()}
+        decay, gain, floor = ops.mlstm_gates(projected, (column["i"], column["f"]), (self.i_bias.data, self.f_bias.data),
+                                             self.gate_cap, maximum.slots, ctx.seg_start, ctx.seg_len, ctx.seg_row,
+                                             ctx.n_segments)
+        raw = ctx.empty((n, self.n_heads, self.value_dim + 1), dtype=torch.float32)
+        columns = (column["q"], column["k"], column["v"], None)
+
+        def run(state, starts, lens, rows, count, **mode):
+            ops.gla_scan(projected, columns, None, self.q_scale, None, 0.0, state, starts, lens, rows, count, *sizes, None,
+                         scratch=raw, token_scalars=(decay, gain), ones=True, raw_only=True, **mode)
+
+        _scan_step(ctx, memory.slots, run, sizes)
+        mixed = ctx.empty((n, self.n_heads * self.value_dim))
+        return ops.mlstm_finish(raw, floor, projected, column["g"], self.norm_weight.data, self.norm_eps, mixed)

@@ -48,6 +48,33 @@ class ExactRMSNorm(Norm):
     def forward(self, ctx, x, rows=None):
         return ops.rmsnorm_exact(x, self.weight.data, self.eps, self.offset, out_dtype=ctx.dtype, rows=rows)
 
+    def as_join(self):
+        return (self.weight.data, self.eps, "rms") if self.offset == 0.0 else None
+
+
+class ScalarRMSNorm(Norm):
+    """``y = x / sqrt(mean(x^2) + eps) * g`` with one learned number g for all coordinates (a tensor without
+    dimensions): float32 arithmetic and a single rounding, like :class:`ExactRMSNorm`, whose kernels it shares: the
+    number is spread over a row of the width after loading."""
+    graph_safe = True
+
+    def __init__(self, width, eps, *, name, suffix=".weight"):
+        self.width, self.eps, self.name, self.suffix = int(width), float(eps), name, suffix
+        self.gain = Param((), init="norm", std=0.05)
+        self._row = None
+
+    def named_params(self):
+        return {self.name + self.suffix: self.gain}
+
+    def finalize(self, device, dtype):
+        self._row = self.gain.data.reshape(1).expand(self.width).contiguous()
+
+    def forward(self, ctx, x, rows=None):
+        return ops.rmsnorm_exact(x, self._row, self.eps, 0.0, out_dtype=ctx.dtype, rows=rows)
+
+    def as_join(self):
+        return self._row, self.eps, "rms"
+
 
 class LayerNorm(Norm):
     """``y = (x - mean) / sqrt(var + eps) * w + b`` with ``var`` the mean of the squared deviations: float32
@@ -74,3 +101,6 @@ class LayerNorm(Norm):
     def forward(self, ctx, x, rows=None):
         return ops.layernorm_exact(x, self.weight.data, self.bias.data if self.bias is not None else None, self.eps,
                                    out_dtype=ctx.dtype, rows=rows)
+
+    def as_join(self):
+        return (self.weight.data, self.eps, "layer") if self.bias is None else None

@@ -4,6 +4,9 @@ its own, and the mixer's result is a weighted sum of the two (half the sum, by d
     y = share * ( left(h) / rms(left(h)) * w_left + right(h) / rms(right(h)) * w_right )
 
 The two keep their own caches: the mixer's cache spec is the tuple of theirs, its view the tuple of their views.
+A pair of scales in place of ``norm_eps``, weights and share (``scales`` = (left, right)) gives the plain weighted sum
+y = left_scale * left(h) + right_scale * right(h); a block that joins several branches at once takes the two unsummed
+(``branches``).
 Inside a block that norms its branches on the way into the stream (:class:`PostNormBlock`) the two norms, the sum,
 the block's own norm and the residual sum are one kernel (``kernels.ops.rms_join``), so the mixer joins the stream
 itself (``joins_stream``); ``forward`` without a stream returns y in float32.
@@ -19,14 +22,18 @@ from .base import Mixer, Param
 class ParallelMixers(Mixer):
     """``left`` and ``right``: two mixers whose ``forward(ctx, h, cache, out_float32=True)`` gives float32 rows.
     names: dict with keys left_out, right_out (the two output norms' weights)."""
-    joins_stream = True
-
-    def __init__(self, hidden_size, left, right, *, norm_eps, names, share=0.5, norm_suffix=".weight"):
+    def __init__(self, hidden_size, left, right, *, norm_eps=None, names=None, share=0.5, norm_suffix=".weight", scales=None):
         self.hidden_size, self.left, self.right = int(hidden_size), left, right
-        self.norm_eps, self.share = float(norm_eps), float(share)
-        self.left_weight = Param((hidden_size,), init="norm", std=0.05)
-        self.right_weight = Param((hidden_size,), init="norm", std=0.05)
-        self._names = {names["left_out"] + norm_suffix: self.left_weight, names["right_out"] + norm_suffix: self.right_weight}
+        self.scales = None if scales is None else (float(scales[0]), float(scales[1]))
+        if (self.scales is None) == (norm_eps is None):
+            raise ValueError("two mixers side by side are summed through a norm each, or by a scale each")
+        self._names = {}
+        if self.scales is None:
+            self.norm_eps, self.share = float(norm_eps), float(share)
+            self.left_weight = Param((hidden_size,), init="norm", std=0.05)
+            self.right_weight = Param((hidden_size,), init="norm", std=0.05)
+            self._names = {names["left_out"] + norm_suffix: self.left_weight, names["right_out"] + norm_suffix: self.right_weight}
+        self.joins_stream = self.scales is None
         self.graph_safe = True
         self._counts = tuple(len(spec) if isinstance(spec, tuple) else 1 for spec in (left.cache_spec(), right.cache_spec()))
 
@@ -38,7 +45,7 @@ class ParallelMixers(Mixer):
 
     def finalize(self, device, dtype):
         super().finalize(device, dtype)
-        if self.left_weight.data.dtype != self.right_weight.data.dtype:
+        if self.scales is None and self.left_weight.data.dtype != self.right_weight.data.dtype:
             self.left_weight.data, self.right_weight.data = self.left_weight.data.float(), self.right_weight.data.float()
 
     def cache_spec(self):
@@ -52,10 +59,27 @@ class ParallelMixers(Mixer):
         left, right = cache[:n_left], cache[n_left:]
         return (left if n_left > 1 else left[0]), (right if self._counts[1] > 1 else right[0])
 
+    def input_projections(self):
+        found = []
+        for part in (self.left, self.right):
+            found += part.input_projections() if hasattr(part, "input_projections") else []
+        return found
+
+    def branches(self, ctx, x, cache, joint=None):
+        """[(left's float32 rows, its scale), (right's, its scale)], of a pair that is summed by scales."""
+        views = self._views(cache)
+        how = {} if joint is None else dict(joint=joint)
+        return [(part.forward(ctx, x, view, out_float32=True, **how), scale)
+                for part, view, scale in zip((self.left, self.right), views, self.scales)]
+
     def forward(self, ctx, x, cache, stream=None, norm_weight=None, mult=1.0, out_float32=True, rows=None):
         """x [N, hidden] -> y float32 [N, hidden]; with ``stream`` (the residual stream, updated in place and
         returned): stream += mult * rms(y) * norm_weight, and ``rows`` (bfloat16, optional) receives the stream's
         new values rounded."""
+        if self.scales is not None:
+            if stream is not None:
+                raise ValueError("a pair that is summed by scales gives its branches to the block")
+            return ops.branch_join(torch.zeros(x.shape, dtype=torch.float32, device=x.device), self.branches(ctx, x, cache))
         left_view, right_view = self._views(cache)
         a = self.left.forward(ctx, x, left_view, out_float32=True)
         b = self.right.forward(ctx, x, right_view, out_float32=True)

@@ -49,16 +49,20 @@ class RotaryFrequencies(PositionEncoding):
     ``scaling`` = (factor, low, high, original) stretches long waves for contexts beyond the ``original`` one: with
     wavelength l = 2 pi / freq, a frequency stays when l < original / high, becomes freq / factor when
     l > original / low, and between the two is (1 - s) freq / factor + s freq with
-    s = (original / l - low) / (high - low)."""
+    s = (original / l - low) / (high - low).  ``stretch`` divides every frequency, whatever its wavelength (linear
+    scaling of the positions)."""
     graph_safe = True
     LAYOUTS = {"halves": 0, "interleaved": 1}
 
-    def __init__(self, dims, base, layout="halves", scaling=None):
+    def __init__(self, dims, base, layout="halves", scaling=None, stretch=1.0):
         if dims % 2 or dims <= 0:
             raise ValueError(f"the number of rotated dimensions must be positive and even, got {dims}")
         if layout not in self.LAYOUTS:
             raise ValueError(f"unknown rotary layout {layout!r} (known: {sorted(self.LAYOUTS)})")
         self.rotary_dim, self.base, self.layout = int(dims), float(base), self.LAYOUTS[layout]
+        self.stretch = float(stretch)
+        if not self.stretch > 0:
+            raise ValueError(f"frequencies are divided by a positive number, not {stretch}")
         self.scaling = None if scaling is None else tuple(float(v) for v in scaling)
         if self.scaling is not None and (len(self.scaling) != 4 or self.scaling[0] <= 0 or self.scaling[3] <= 0
                                          or not 0 < self.scaling[1] < self.scaling[2]):
@@ -67,7 +71,7 @@ class RotaryFrequencies(PositionEncoding):
 
     def frequencies(self) -> list:
         """The frequency of every rotated pair as Python floats (float64)."""
-        values = [self.base ** (-2.0 * i / self.rotary_dim) for i in range(self.rotary_dim // 2)]
+        values = [self.base ** (-2.0 * i / self.rotary_dim) / self.stretch for i in range(self.rotary_dim // 2)]
         if self.scaling is None:
             return values
         factor, low, high, original = self.scaling
