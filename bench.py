@@ -1275,6 +1275,190 @@ def run_gogotar(args):
         torch.cuda.empty_cache()
 
 
+# --------------------------------------------------------------------------- Lotazen beside Virulix
+LOTAZEN_SHAPES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, lin_heads=8, lin_dim=128, lin_vdim=128, experts=32, top=4,
+                 expert_ff=768, shared_ff=1536, span=1024, vocab=32768),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, lin_heads=16, lin_dim=128, lin_vdim=128, experts=64, top=6,
+                 expert_ff=1024, shared_ff=2048, span=1024, vocab=32768),
+}
+
+
+def _lotazen_sizes(width, heads, kv_heads, dim, lin_heads, lin_dim, lin_vdim, experts, top, expert_ff, shared_ff, span, vocab):
+    """Eight layers: windowed attention beside HGRN2, and a matrix memory, in turn; routed experts throughout."""
+    left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, mask=dict(size=span),
+                rot=dict(base=1000000.0, dims=dim, scaling=dict(factor=4.0)))
+    recurrent = dict(heads=lin_heads, dim=lin_dim, vdim=lin_vdim)
+    mlp = dict(kind="moe", expert=dict(ff=expert_ff, limit=7.0), router=dict(experts=experts, top=top),
+               shared=dict(ff=shared_ff, limit=7.0))
+    pair = dict(type="parallel", mixer=dict(left=left, right=recurrent, left_scale=0.5, right_scale=0.5), mlp=mlp)
+    memory = lambda kind: dict(type=kind, mixer=dict(recurrent, gate_cap=15.0), mlp=mlp)
+    return dict(architecture="Lotazen", vocab=vocab, width=width, norm=dict(eps=1e-6), max_positions=8192, logit_softcap=30.0,
+                layers=[pair, memory("mlstm"), pair, memory("mlstm_2")] * 2)
+
+
+def _virulix_beside_lotazen(width, heads, kv_heads, dim, lin_heads, lin_dim, lin_vdim, experts, top, expert_ff, shared_ff,
+                            vocab, **_):
+    """Virulix of equal width, heads, layer count, experts and vocabulary: attention and gated linear attention in turn,
+    routed experts with a shared one throughout."""
+    attention = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, q_temp=dict(coef=0.1, every=256))
+    gla = dict(heads=lin_heads, dim=lin_dim, vdim=lin_vdim, tau=16.0, rank=16)
+    mlp = dict(kind="moe", expert=dict(ff=expert_ff, limit=7.0), router=dict(experts=experts, top=top),
+               shared=dict(ff=shared_ff, limit=7.0))
+    layers = [dict(type=kind, mixer=mixer, mlp=mlp) for kind, mixer in (("attention", attention), ("gla", gla)) * 4]
+    return dict(architecture="Virulix", vocab=vocab, width=width, norm=dict(eps=1e-6), layers=layers)
+
+
+def _lotazen_kernels(torch, lotazen, virulix, sizes, pk, tokens_n, batch, context, flush):
+    """The kernels of Lotazen's mechanisms alone, each beside the like kernel of Virulix (the join: of Gogotar), with what
+    the roofline allows."""
+    from qwen_inference_lab_b200.kernels import ops
+    bench = _PartKernels(torch, pk, tokens_n, batch, context, flush)
+    H, G, d, W, span = sizes["heads"], sizes["kv_heads"], sizes["dim"], sizes["width"], sizes["span"]
+    pair = next(l.mixer for l in lotazen.layers if hasattr(l.mixer, "left"))
+    memory = next(l.mixer for l in lotazen.layers if hasattr(l.mixer, "gate_cap"))
+    theirs = next(l.mixer for l in virulix.layers if hasattr(l.mixer, "plain_tail"))
+    their_gla = next(l.mixer for l in virulix.layers if hasattr(l.mixer, "decay_rank"))
+    pairs_window = sum(min(i, span - 1) + 1 for i in range(tokens_n))
+    pairs_all = tokens_n * (tokens_n + 1) // 2
+    first_view = lambda view: view[0] if isinstance(view, tuple) else view
+
+    # ---- attention itself
+    def attention(mixer):
+        def kernel(ctx, x, view):
+            q = x[:, :H * d].contiguous()
+            out = torch.empty_like(q)
+            bench.timed(lambda: mixer._attend(ctx, q, first_view(view), out))
+            return out
+        return kernel
+    bench.measure("lotazen windowed attention", pair.left, H * d, attention(pair.left), (4.0 * H * d * pairs_window, None),
+                  batch * min(context + 1, span) * 2 * G * d * 2)
+    bench.measure("virulix attention (distance slopes)", theirs, H * d, attention(theirs), (4.0 * H * d * pairs_all, None),
+                  batch * (context + 1) * 2 * G * d * 2)
+
+    # ---- what stands between the projection and the attention
+    channels = (H + 2 * G) * d
+    moved = lambda n, width: 2 * n * width * 2          # every row read once and written once
+    left = pair.left
+    def rotate_store(ctx, x, view):
+        qkv = x[:, :channels].contiguous()
+        q = torch.empty((x.shape[0], H * d), dtype=x.dtype, device=x.device)
+        bench.timed(lambda: ops.qk_rotate_store(qkv, (0, H * d, (H + G) * d), q, view.pages, None, None, left.unit_qk_norm_eps,
+                                                left.position.freq, left.position.rotary_dim, left.position.layout,
+                                                ctx.positions, ctx.token_row, view.block_table, H, G, d, d, view.page_size,
+                                                unit_heads=True))
+        return q
+    def plain_store(ctx, x, view):
+        qkv = x[:, :channels].contiguous()
+        q = torch.empty((x.shape[0], H * d), dtype=x.dtype, device=x.device)
+        bench.timed(lambda: ops.qkv_store(qkv, q, view.pages, ctx.positions, ctx.token_row, view.block_table, H, G, d, d,
+                                          view.page_size, 0.1, 256))
+        return q
+    bench.measure("lotazen heads of unit size + rotation + page write", left, channels, rotate_store,
+                  (None, moved(tokens_n, channels)), moved(batch, channels))
+    bench.measure("virulix query temperature + page write", theirs, channels, plain_store,
+                  (None, moved(tokens_n, channels)), moved(batch, channels))
+
+    # ---- the recurrences: float32 on the CUDA cores by both designs, so the prompt's bound is the float32 FMA rate
+    fma = (148 * 128 * 2 * 1.9e9, "of the float32 FMA rate (72 TFLOP/s nominal)")
+    def scan(part, whole):
+        width = part.projection.out_features
+        def kernel(ctx, x, view):
+            projected = x[:, :width].contiguous()
+            return bench.timed(lambda: part.scan(ctx, projected, 0, view))
+        state = part.n_heads * part.key_dim * part.value_dim
+        bench.measure(whole, part, width, kernel, (5.0 * state * tokens_n, None), batch * state * 4 * 2, prompt_of=fma)
+    scan(pair.right, "lotazen hgrn2 scan (gate and norm with it)")
+    scan(memory, "lotazen matrix memory (gates, scan, normaliser, norm and output gate)")
+    gh, gd, ge = their_gla.n_heads, their_gla.key_dim, their_gla.value_dim
+    their_width = their_gla.projection.out_features
+    def gla_scan(ctx, x, view):
+        projected = x[:, :their_width].contiguous()
+        mixed = torch.empty((x.shape[0], gh * ge), dtype=x.dtype, device=x.device)
+        bench.timed(lambda: their_gla.scan(ctx, projected, view, mixed))
+        return mixed
+    bench.measure("virulix gated linear attention scan (decays, norm and gate with it)", their_gla, their_width, gla_scan,
+                  (5.0 * gh * gd * ge * tokens_n, None), batch * gh * gd * ge * 4 * 2, prompt_of=fma)
+
+    # ---- the sublayers' first product, joining the stream, the experts
+    for label, block in (("pair", lotazen.layers[0]), ("memory", lotazen.layers[1])):
+        rows_n = block.input.out_features
+        def first_product(ctx, x, view, block=block):
+            h = x[:, :W].contiguous()
+            return bench.timed(lambda: block.input.forward_joint(ctx, h)).rows
+        bench.measure(f"lotazen joint first product ({label}: {rows_n} rows)", block.mixer, W, first_product,
+                      (2.0 * tokens_n * rows_n * W, None), rows_n * W * 2)
+    qkv_rows = theirs.qkv.out_features
+    def their_product(ctx, x, view):
+        h = x[:, :W].contiguous()
+        return bench.timed(lambda: theirs.qkv.forward(ctx, h))
+    bench.measure(f"virulix q/k/v product ({qkv_rows} rows)", theirs, W, their_product, (2.0 * tokens_n * qkv_rows * W, None),
+                  qkv_rows * W * 2)
+    ours = next(l.feed_forward for l in lotazen.layers)
+    top = ours.top
+    weight = torch.ones(W, dtype=torch.bfloat16, device="cuda")
+    def branch_join(ctx, x, view):
+        stream = x[:, :W].float()
+        branches = [(x[:, :W].float() * c, c) for c in (0.5, 0.25, 1.0)]
+        routed = x[:, None, :W].float().expand(-1, top, -1).contiguous()
+        out = torch.empty((x.shape[0], W), dtype=x.dtype, device=x.device)
+        return bench.timed(lambda: ops.branch_join(stream, branches, routed=routed, next_weight=weight, next_eps=1e-6, rows=out))
+    def norm_join(ctx, x, view):
+        stream, branch = x[:, :W].float(), x[:, :W].float() * 3.0
+        out = torch.empty((x.shape[0], W), dtype=x.dtype, device=x.device)
+        return bench.timed(lambda: ops.norm_join(stream, branch, weight, 1e-6, "rms", next_weight=weight, rows=out))
+    bench.measure(f"lotazen three branches and {top} experts join the stream, the next norm behind them (1 kernel)", memory, W,
+                  branch_join, (None, tokens_n * W * (4 * (2 + 3 + top) + 2)), batch * W * (4 * (2 + 3 + top) + 2))
+    bench.measure("gogotar's join (one normed branch, the next norm behind it)", memory, W, norm_join,
+                  (None, tokens_n * W * (4 * 3 + 2)), batch * W * (4 * 3 + 2))
+    their_experts = next(l.feed_forward for l in virulix.layers if hasattr(l.feed_forward, "n_experts"))
+    active = 3 * ours.expert_size * W
+    shared = 3 * ours.shared.intermediate_size * W
+    touched = lambda n: (min(ours.n_experts, n * top) * active + shared) * 2
+    def our_experts(ctx, x, view):
+        h = x[:, :W].contiguous()
+        return bench.timed(lambda: ours.branches(ctx, h))[1].view(h.shape[0], -1)
+    def their_ff(ctx, x, view):
+        h, residual = x[:, :W].contiguous(), x[:, :W].float()
+        return bench.timed(lambda: their_experts.forward(ctx, h, residual=residual))
+    work = 2.0 * tokens_n * (top * active + shared)
+    bench.measure("lotazen routed and shared experts (input weighed, unsummed)", ours, W, our_experts, (work, None), touched(batch))
+    bench.measure("virulix routed and shared experts (summed onto the stream)", their_experts, W, their_ff, (work, None), touched(batch))
+    return bench.rows
+
+
+def run_lotazen(args):
+    """Prefill and decode of Lotazen at sizes like a real model's layers, beside Virulix (the engine's closest design: a
+    float32 stream, attention and gated linear attention with a float32 state, routed experts beside a shared one) of
+    equal width, heads, layer count, experts and vocabulary, and the kernels of its mechanisms against their rooflines."""
+    import torch
+    from qwen_inference_lab_b200.config.model_config import LotazenConfig, VirulixConfig
+    from qwen_inference_lab_b200.loading import random_model
+    pk = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    for name in ([args.lotazen_shape] if args.lotazen_shape else sorted(LOTAZEN_SHAPES)):
+        sizes = LOTAZEN_SHAPES[name]
+        lotazen = random_model(LotazenConfig.from_dict(_lotazen_sizes(**sizes)), seed=0, device="cuda", dtype=torch.bfloat16)
+        virulix = random_model(VirulixConfig.from_dict(_virulix_beside_lotazen(**sizes)), seed=0, device="cuda", dtype=torch.bfloat16)
+        result = {"workload": "lotazen", "width": sizes["width"], "layers": 8, "dtype": "bfloat16",
+                  "peaks": "of measured" if pk["source"] == "measured" else "of fallback", "models": {}, "kernels": []}
+        for label, model in (("lotazen", lotazen), ("virulix", virulix)):
+            bench = _ModelBench(model, sizes["vocab"])
+            entry = {}
+            for tokens_n in (512, 2048):
+                ms = bench.prefill(tokens_n, flush)
+                entry[f"prefill_{tokens_n}"] = {"ms": round(ms, 3), "tokens_per_s": round(tokens_n / ms * 1e3, 1)}
+            for batch, context in ((1, 2048), (8, 2048), (32, 2048)):
+                ms = bench.decode(batch, context, args.steps, max(args.warmup, 6))
+                entry[f"decode_b{batch}_c{context}"] = {"ms": round(ms, 4), "tokens_per_s": round(batch / ms * 1e3, 1)}
+            result["models"][label] = entry
+        for kernel, ms, frac, of in _lotazen_kernels(torch, lotazen, virulix, sizes, pk, 2048, 8, 2048 + 511, flush):
+            result["kernels"].append({"kernel": kernel, "ms": round(ms, 4), "frac": round(frac, 4), "of": of})
+        print(json.dumps(result), flush=True)
+        del lotazen, virulix
+        torch.cuda.empty_cache()
+
+
 def run_reference(args):
     ref = ROOT / "baseline" / "_ref"
     def unavailable(why):
@@ -1361,13 +1545,14 @@ def main():
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--layers", type=int, default=None, help="run fewer layers than the configuration has")
     parser.add_argument("--quick", action="store_true", help="skip the batch 1 and 64 points")
-    parser.add_argument("--only", choices=["decode", "prefill", "mixed", "virulix", "debisun", "larolorn", "gogotar"], default=None,
+    parser.add_argument("--only", choices=["decode", "prefill", "mixed", "virulix", "debisun", "larolorn", "gogotar", "lotazen"], default=None,
                         help="run just this part and print its result instead of the JSON line; mixed = 64 requests "
                              "with prompts of 16 to 2048 tokens and 128 new tokens each through Engine.generate; "
                              "virulix = the Virulix design beside dense Qwen3 of equal size, and its mixers' kernels; "
                              "debisun = the Debisun design beside Virulix of equal size, and its mechanisms' kernels; "
                              "larolorn = the Larolorn design beside Virulix of equal size, and its mechanisms' kernels; "
-                             "gogotar = the Gogotar design beside Larolorn of equal size, and its mechanisms' kernels")
+                             "gogotar = the Gogotar design beside Larolorn of equal size, and its mechanisms' kernels; "
+                             "lotazen = the Lotazen design beside Virulix of equal size, and its mechanisms' kernels")
     parser.add_argument("--virulix-shape", choices=sorted(VIRULIX_SHAPES), default=None,
                         help="width of --only virulix (default: all)")
     parser.add_argument("--debisun-shape", choices=sorted(DEBISUN_SHAPES), default=None,
@@ -1376,6 +1561,8 @@ def main():
                         help="width of --only larolorn (default: all)")
     parser.add_argument("--gogotar-shape", choices=sorted(LAROLORN_SHAPES), default=None,
                         help="width of --only gogotar (default: all)")
+    parser.add_argument("--lotazen-shape", choices=sorted(LOTAZEN_SHAPES), default=None,
+                        help="width of --only lotazen (default: all)")
     parser.add_argument("--shape", choices=sorted(SHAPES), default="8b", help="layer sizes (default: Qwen3-8B)")
     parser.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16")
     parser.add_argument("--context", type=int, default=CONTEXT, help="cached tokens per request (profiling aid)")
@@ -1394,6 +1581,9 @@ def main():
         return
     if args.only == "gogotar":
         run_gogotar(args)
+        return 0
+    if args.only == "lotazen":
+        run_lotazen(args)
         return 0
     if args.only == "debisun":
         run_debisun(args)

@@ -160,6 +160,84 @@ qk_rotate_store_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col,
     }
 }
 
+// The same for pairs of neighbours and norms per head (or none), 16 bytes a lane: a head is d / V lanes (a power of two),
+// which hold their values in registers, sum their squares by shuffles and turn their own pairs, so that nothing but the
+// token's angles goes through shared memory.  Every head of the token is asked for before the angles are made.
+#define ROTATE_PIECES 4      // pieces of a token's q and k that a thread may hold
+template <typename T, typename W>
+__global__ void __launch_bounds__(256)
+qk_rotate_store_lanes_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col, int v_col, T* __restrict__ q_out,
+                             T* __restrict__ pages, const W* __restrict__ q_norm_w, const W* __restrict__ k_norm_w, float eps,
+                             const float* __restrict__ freq, int rot_dims, const int* __restrict__ positions,
+                             const int* __restrict__ token_row, const int* __restrict__ block_table, int table_stride,
+                             int n_q_heads, int n_kv_heads, int d, int e, int page_size, int num_pages, int per_head) {
+    constexpr int V = 16 / (int)sizeof(T);
+    extern __shared__ __align__(16) float angles[];        // [rot_dims]: cosines, then sines
+    qil_wait_for_producer();
+    qil_release_consumer();
+    const int token = blockIdx.x, tid = threadIdx.x;
+    const int pos = positions[token];
+    const T* row = proj + (size_t)token * ld;
+    const int lanes = d / V;                                // of a head
+    const int q_pieces = n_q_heads * lanes, pieces = q_pieces + n_kv_heads * lanes;
+    uint4 raw[ROTATE_PIECES];
+#pragma unroll
+    for (int u = 0; u < ROTATE_PIECES; ++u) {
+        const int c = tid + u * 256;
+        raw[u] = make_uint4(0u, 0u, 0u, 0u);
+        if (c < pieces) raw[u] = *reinterpret_cast<const uint4*>(c < q_pieces ? row + q_col + c * V : row + k_col + (c - q_pieces) * V);
+    }
+    const int index = pos / page_size;
+    int page = (n_kv_heads > 0 && pos >= 0 && index < table_stride) ? block_table[(size_t)token_row[token] * table_stride + index] : -1;
+    if (page >= num_pages) page = -1;                       // never write outside the pool
+    angle_table(angles, rot_dims, pos, freq);
+    __syncthreads();
+    const int half = rot_dims >> 1, slot = pos % page_size;
+    T* page_base = pages + (size_t)(page < 0 ? 0 : page) * n_kv_heads * page_size * (d + e);
+#pragma unroll
+    for (int u = 0; u < ROTATE_PIECES; ++u) {
+        const int c = tid + u * 256;
+        if (u * 256 >= pieces) break;                       // the whole block: shuffles below take part warp by warp
+        const T* x = reinterpret_cast<const T*>(&raw[u]);
+        const bool is_q = c < q_pieces;
+        const int piece = is_q ? c : c - q_pieces, head = piece / lanes, j0 = (piece - head * lanes) * V;
+        float v[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = to_f32<T>(x[i]);
+        if (per_head) {
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < V; ++i) ss = fmaf(v[i], v[i], ss);
+            for (int step = 1; step < lanes; step <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, step);
+            const float r = 1.0f / sqrtf(ss / (float)d + eps);
+            const W* w = is_q ? q_norm_w : k_norm_w;
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] = (per_head == 2 || c >= pieces) ? v[i] * r : v[i] * r * to_f32<W>(w[j0 + i]);
+        }
+#pragma unroll
+        for (int i = 0; i < V; i += 2) {
+            if (j0 + i >= rot_dims) continue;
+            const float cos_a = angles[(j0 + i) >> 1], sin_a = angles[half + ((j0 + i) >> 1)];
+            const float first = v[i], second = v[i + 1];
+            v[i] = first * cos_a - second * sin_a;
+            v[i + 1] = second * cos_a + first * sin_a;
+        }
+        uint4 packed;
+        T* o = reinterpret_cast<T*>(&packed);
+#pragma unroll
+        for (int i = 0; i < V; ++i) o[i] = from_f32<T>(v[i]);
+        if (c >= pieces) continue;
+        if (is_q) *reinterpret_cast<uint4*>(q_out + (size_t)token * n_q_heads * d + c * V) = packed;
+        else if (page >= 0) *reinterpret_cast<uint4*>(page_base + ((size_t)head * page_size + slot) * d + j0) = packed;
+    }
+    if (page < 0) return;
+    T* values = page_base + (size_t)n_kv_heads * page_size * d;
+    for (int c = tid; c < n_kv_heads * e / V; c += 256) {
+        const int head = c * V / e, j = c * V - head * e;
+        *reinterpret_cast<uint4*>(values + ((size_t)head * page_size + slot) * e + j) = *reinterpret_cast<const uint4*>(row + v_col + c * V);
+    }
+}
+
 extern "C" int qil_qk_rotate_store(const void* proj, int ld, int q_col, int k_col, int v_col, void* q_out, void* pages,
                                    const void* q_norm_w, const void* k_norm_w, int norm_dtype, float eps, const float* freq,
                                    int rot_dims, int layout, const int* positions, const int* token_row,
@@ -180,6 +258,15 @@ extern "C" int qil_qk_rotate_store(const void* proj, int ld, int q_col, int k_co
         constexpr int V = 16 / (int)sizeof(T);
         const int wide = (d % V == 0 && e % V == 0 && ld % V == 0 && q_col % V == 0 && k_col % V == 0 && v_col % V == 0 &&
                           (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)pages) & 15) == 0) ? 1 : 0;
+        const int lanes = d / V;
+        if (wide && layout == 1 && (per_head || q_norm_w == nullptr) && lanes <= 32 && (lanes & (lanes - 1)) == 0
+            && (n_q_heads + n_kv_heads) * lanes <= 256 * ROTATE_PIECES) {
+            qil_launch_chained(qk_rotate_store_lanes_kernel<T, W>, dim3(n_tokens), dim3(256), (size_t)rot_dims * sizeof(float), stream,
+                               (const T*)proj, ld, q_col, k_col, v_col, (T*)q_out, (T*)pages, (const W*)q_norm_w,
+                               (const W*)k_norm_w, eps, freq, rot_dims, positions, token_row, block_table, table_stride,
+                               n_q_heads, n_kv_heads, d, e, page_size, num_pages, per_head);
+            QIL_CHECK_LAUNCH();
+        }
         if (smem > 48 * 1024)
             err = cudaFuncSetAttribute(qk_rotate_store_kernel<T, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (err == cudaSuccess)

@@ -637,8 +637,11 @@ def qkv_store(qkv, q_out, kv_cache, positions, token_row, block_table, n_q_heads
     return q_out
 
 
-def gla_scan_needs_scratch(d, e) -> bool:
-    code = core().qil_gla_scan_needs_scratch(c_int(d), c_int(e))
+def gla_scan_needs_scratch(d, e, ones=False, mode=None) -> bool:
+    """Do a head's ``e`` value columns (a column of ones counted) take more than one block of the scan?  ``mode``: of
+    that mode's blocks (GLA_WHOLE has narrower ones)."""
+    whole = mode is None or mode == GLA_WHOLE
+    code = core().qil_gla_scan_needs_scratch(c_int(d), c_int(e), c_int(1 if ones else 0), c_int(1 if whole else 0))
     if code < 0:
         raise KernelError(f"gla_scan: {d} key channels per head are too many")
     return bool(code)
@@ -667,14 +670,14 @@ def gla_decay(projected, low_column, a2, a2_bias, tau, out=None):
 
 def gla_scan(projected, columns, alpha, q_scale, norm_weight, eps, state, seg_start, seg_len, seg_row,
              n_segments, n_heads, d, e, out, scratch=None, mode=GLA_WHOLE, decay_product=None, head_decay=None,
-             silu_inputs="", raw_only=False, tied_gate=None, token_scalars=None, ones=False):
+             silu_inputs="", raw_only=False, tied_gate=None, token_scalars=None, ones=False, floor=None):
     """Gated linear attention over segments of a step (see csrc/gla_scan.cu for the equations).
 
     ``projected`` [N, width]: the stacked projection; ``columns`` = (q, k, v, g) first columns in it
     (q, k: n_heads * d wide; v, g: n_heads * e).  ``alpha`` float32 [N, n_heads * d]: the decays
     (``gla_decay``).  ``state`` float32 [slots, n_heads, d, e] is read and written at the rows ``seg_row`` names.
-    ``out`` [N, n_heads * e].  ``scratch``: float32 [N, n_heads * e], needed when ``gla_scan_needs_scratch``: the
-    outputs then go there un-normed and ``gla_norm_gate`` finishes them.  ``mode``: GLA_WHOLE; GLA_OWN_STATE scans
+    ``out`` [N, n_heads * e].  ``scratch``: float32 [N, n_heads * e], needed when ``gla_scan_needs_scratch``: where it is
+    given the outputs go there un-normed and ``gla_norm_gate`` finishes them.  ``mode``: GLA_WHOLE; GLA_OWN_STATE scans
     from zero and writes only the segment's own state to ``state[seg_row]`` and the product of its decays to
     ``decay_product`` [slots, n_heads, d]; GLA_FROM_STATE reads ``state[seg_row]``, writes the outputs and leaves
     the state.
@@ -686,7 +689,9 @@ def gla_scan(projected, columns, alpha, q_scale, norm_weight, eps, state, seg_st
     ``tied_gate`` = (bias, lower bound), each [n_heads * d] of one dtype: k's columns are a gate's logits z, a channel
     decays by f = l + (1 - l) sigmoid(z + b) and is written with 1 - f.  ``token_scalars`` = (decay, gain), float32
     [N, n_heads]: a decay and a gain of k per token and head (``mlstm_gates``).  ``ones``: the state has a last column
-    whose value is one (``e`` counts it, v's columns do not; raw outputs only)."""
+    whose value is one (``e`` counts it; v's and g's columns, ``norm_weight`` and ``out`` do not).  It goes with raw
+    outputs, or with ``floor`` (float32 [N, n_heads], of ``mlstm_gates``): the outputs are then finished as
+    ``mlstm_finish`` does, ``norm_weight`` [n_heads * (e - 1)] and g's columns being the output gate."""
     _need(projected, "projected", ndim=2)
     if not raw_only:
         _need(out, "out", projected.dtype, 2); _need(norm_weight, "norm_weight", ndim=1)
@@ -706,8 +711,12 @@ def gla_scan(projected, columns, alpha, q_scale, norm_weight, eps, state, seg_st
         if not raw_only and param_dtype != gate_bias.dtype:
             raise KernelError("gla_scan: the gate's bias and the norm's weight share a dtype")
         param_dtype = gate_bias.dtype
-    if ones and not raw_only:
-        raise KernelError("gla_scan: a column of ones goes with raw outputs")
+    if floor is not None:
+        _need(floor, "floor", torch.float32, 2)
+        if not ones or token_scalars is None or raw_only or columns[3] is None or floor.shape != (projected.shape[0], n_heads):
+            raise KernelError("gla_scan: a floor goes with a column of ones, token scalars and an output gate")
+    elif ones and not raw_only:
+        raise KernelError("gla_scan: a column of ones without a floor goes with raw outputs")
     if token_scalars is not None:
         for t in token_scalars:
             _need(t, "token scalars", torch.float32, 2)
@@ -724,7 +733,8 @@ def gla_scan(projected, columns, alpha, q_scale, norm_weight, eps, state, seg_st
     q_at, k_at, v_at, g_at = (int(c) if c is not None else None for c in columns[:4])
     values = e - 1 if ones else e
     if ((alpha is not None and alpha.shape != (n, n_heads * d)) or tuple(state.shape[1:]) != (n_heads, d, e)
-            or (not raw_only and (norm_weight.shape[0] != e or out.shape != (n, n_heads * e)))):
+            or (not raw_only and (norm_weight.shape[0] != (n_heads * values if floor is not None else e)
+                                  or out.shape != (n, n_heads * values)))):
         raise KernelError("gla_scan: shapes do not match the head counts")
     if max(q_at + n_heads * d, k_at + n_heads * d, v_at + n_heads * values, (g_at or 0) + n_heads * values) > ld:
         raise KernelError("gla_scan: a column range lies outside the projection")
@@ -746,8 +756,8 @@ def gla_scan(projected, columns, alpha, q_scale, norm_weight, eps, state, seg_st
     _check(lib, lib.qil_gla_scan(
         c_void_p(base + q_at * size), c_void_p(base + k_at * size), c_void_p(base + v_at * size),
         c_void_p(base + g_at * size if g_at is not None else 0), _p(alpha), _p(head_decay), _p(gate_bias), _p(gate_lower),
-        _p(token_decay), _p(token_gain), c_int(sum(1 << "qkv".index(c) for c in set(silu_inputs))), c_int(1 if ones else 0),
-        c_int(1 if raw_only else 0), c_int(ld), c_float(q_scale), _p(norm_weight), c_float(eps), _p(state),
+        _p(token_decay), _p(token_gain), _p(floor), c_int(sum(1 << "qkv".index(c) for c in set(silu_inputs))), c_int(1 if ones else 0),
+        c_int(1 if raw_only or scratch is not None else 0), c_int(ld), c_float(q_scale), _p(norm_weight), c_float(eps), _p(state),
         _p(seg_start), _p(seg_len), _p(seg_row), c_int(n_segments), c_int(n), c_int(n_heads), c_int(d), c_int(e),
         _p(scratch), _p(out), c_int(mode), _p(decay_product), c_int(dtype_code(projected.dtype)),
         c_int(dtype_code(param_dtype)), _stream()), "gla_scan")

@@ -55,6 +55,16 @@ class ScanPlanner(StepPlanner):
 _PLANNER = ScanPlanner()
 
 
+def _scratch_needs(d, e, ones=False):
+    """(short segments, chunks): does the scan of each need the scratch buffer, since no block holds a whole head's row?"""
+    return tuple(ops.gla_scan_needs_scratch(d, e, ones, mode) for mode in (ops.GLA_WHOLE, ops.GLA_FROM_STATE))
+
+
+def _step_needs_scratch(plan, needs):
+    """Of a step: the kernel that finishes the scratch buffer runs over all its tokens, so all scans use it or none."""
+    return (plan.count["short_start"] > 0 and needs[0]) or (plan.count["chunk_start"] > 0 and needs[1])
+
+
 class GatedLinearAttention(Mixer):
     """names: dict with keys q, k, v, g, o, a1, a2 (projection names) and norm (the output norm's weight).
     ``suffixes``: what the checkpoint appends to a projection's name for weight and bias."""
@@ -92,7 +102,7 @@ class GatedLinearAttention(Mixer):
         common = self.projection._weight().dtype
         for param in (self.decay_up, self.decay_bias, self.norm_weight):
             param.data = param.data.to(common).contiguous()
-        self._needs_scratch = ops.gla_scan_needs_scratch(self.key_dim, self.value_dim)
+        self._needs_scratch = _scratch_needs(self.key_dim, self.value_dim)
 
     def cache_spec(self):
         return StateSpec((self.n_heads, self.key_dim, self.value_dim), torch.float32)
@@ -113,7 +123,8 @@ class GatedLinearAttention(Mixer):
         """The recurrence, the norm and the gate over the step's segments: ``projected`` -> ``mixed``."""
         n = projected.shape[0]
         plan = ctx.plans[_PLANNER.key]
-        scratch = ctx.empty((n, self.n_heads * self.value_dim), dtype=torch.float32) if self._needs_scratch else None
+        scratch = ctx.empty((n, self.n_heads * self.value_dim), dtype=torch.float32) \
+            if _step_needs_scratch(plan, self._needs_scratch) else None
         alpha = ops.gla_decay(projected, self.columns[4], self.decay_up.data, self.decay_bias.data, self.tau)
         common = (projected, self.columns, alpha, self.q_scale, self.norm_weight.data, self.norm_eps)
         sizes = (self.n_heads, self.key_dim, self.value_dim, mixed)
@@ -269,7 +280,7 @@ class TiedGateLinearAttention(Mixer):
         super().finalize(device, dtype)
         for param in (self.gate_bias, self.gate_lower, self.norm_weight):      # float32 arithmetic: read as float32
             param.data = param.data.to(torch.float32).contiguous()
-        self._needs_scratch = ops.gla_scan_needs_scratch(self.key_dim, self.value_dim)
+        self._needs_scratch = _scratch_needs(self.key_dim, self.value_dim)
 
     def cache_spec(self):
         return StateSpec((self.n_heads, self.key_dim, self.value_dim), torch.float32)
@@ -290,7 +301,8 @@ class TiedGateLinearAttention(Mixer):
         """The recurrence and the norm over the step's segments: columns of ``projected`` from ``at`` on -> [N, heads * e]."""
         n, sizes = projected.shape[0], (self.n_heads, self.key_dim, self.value_dim)
         mixed = ctx.empty((n, self.n_heads * self.value_dim))
-        scratch = ctx.empty((n, self.n_heads * self.value_dim), dtype=torch.float32) if self._needs_scratch else None
+        scratch = ctx.empty((n, self.n_heads * self.value_dim), dtype=torch.float32) \
+            if _step_needs_scratch(ctx.plans[_PLANNER.key], self._needs_scratch) else None
         columns = (*(at + c for c in self.columns), None)
 
         def run(state, starts, lens, rows, count, **mode):
@@ -317,8 +329,8 @@ class MatrixMemory(Mixer):
 
     q, k, v, g, i and f are one stacked product.  ``kernels.ops.mlstm_gates`` walks the gates and the running maximum of
     every segment and leaves a decay, a gain and a floor per token and head; with those the memory is the scan of
-    :class:`GatedLinearAttention` (``kernels.ops.gla_scan``) with a column of ones behind the values, which is n;
-    ``kernels.ops.mlstm_finish`` divides, norms and gates.  State: (S beside n, m), float32.
+    :class:`GatedLinearAttention` (``kernels.ops.gla_scan``) with a column of ones behind the values, which is n; the
+    scan divides, norms and gates its outputs too where a head's columns fit one block.  State: (S beside n, m), float32.
 
     names: dict with keys q, k, v, g, i, f, o (projection names) and norm."""
     graph_safe = True
@@ -344,6 +356,7 @@ class MatrixMemory(Mixer):
         self._names = {names["i"] + suffixes[1]: self.i_bias, names["f"] + suffixes[1]: self.f_bias,
                        names["norm"] + norm_suffix: self.norm_weight}
         self.out = Linear(vw, hidden_size, name=names["o"], suffixes=suffixes)
+        self._needs_scratch = False
 
     def named_params(self):
         return dict(self._names)
@@ -355,7 +368,7 @@ class MatrixMemory(Mixer):
         super().finalize(device, dtype)
         for param in (self.i_bias, self.f_bias, self.norm_weight):
             param.data = param.data.to(torch.float32).contiguous()
-        ops.gla_scan_needs_scratch(self.key_dim, self.value_dim + 1)       # refuses key sizes the scan cannot hold
+        self._needs_scratch = _scratch_needs(self.key_dim, self.value_dim + 1, ones=True)
 
     def cache_spec(self):
         return (StateSpec((self.n_heads, self.key_dim, self.value_dim + 1), torch.float32),
@@ -381,13 +394,17 @@ class MatrixMemory(Mixer):
         decay, gain, floor = ops.mlstm_gates(projected, (column["i"], column["f"]), (self.i_bias.data, self.f_bias.data),
                                              self.gate_cap, maximum.slots, ctx.seg_start, ctx.seg_len, ctx.seg_row,
                                              ctx.n_segments)
-        raw = ctx.empty((n, self.n_heads, self.value_dim + 1), dtype=torch.float32)
-        columns = (column["q"], column["k"], column["v"], None)
+        mixed = ctx.empty((n, self.n_heads * self.value_dim))
+        columns = (column["q"], column["k"], column["v"], column["g"])
+        raw, finish = None, dict(floor=floor)
+        if _step_needs_scratch(ctx.plans[_PLANNER.key], self._needs_scratch):      # a head's columns are spread over several blocks, which cannot norm them
+            raw, finish = ctx.empty((n, self.n_heads, self.value_dim + 1), dtype=torch.float32), dict(raw_only=True)
 
         def run(state, starts, lens, rows, count, **mode):
-            ops.gla_scan(projected, columns, None, self.q_scale, None, 0.0, state, starts, lens, rows, count, *sizes, None,
-                         scratch=raw, token_scalars=(decay, gain), ones=True, raw_only=True, **mode)
+            ops.gla_scan(projected, columns, None, self.q_scale, self.norm_weight.data, self.norm_eps, state, starts, lens, rows,
+                         count, *sizes, mixed, scratch=raw, token_scalars=(decay, gain), ones=True, **finish, **mode)
 
         _scan_step(ctx, memory.slots, run, sizes)
-        mixed = ctx.empty((n, self.n_heads * self.value_dim))
-        return ops.mlstm_finish(raw, floor, projected, column["g"], self.norm_weight.data, self.norm_eps, mixed)
+        if raw is not None:
+            ops.mlstm_finish(raw, floor, projected, column["g"], self.norm_weight.data, self.norm_eps, mixed)
+        return mixed
