@@ -580,11 +580,21 @@ mlstm_gates_kernel(const T* __restrict__ igate, const T* __restrict__ fgate, int
         }
         __syncthreads();
         if (tid == 0) {
+            // sixteen tokens' gates are read before their maxima are written: a load does not wait for the store before it
             float m = after[0];
-#pragma unroll 8
-            for (int j = 0; j < nb; ++j) {
-                const float2 g = gates[j];
-                m = fmaxf(g.x + m, g.y);
+            int j = 0;
+            for (; j + 16 <= nb; j += 16) {
+                float2 g[16];
+                float now[16];
+#pragma unroll
+                for (int u = 0; u < 16; ++u) g[u] = gates[j + u];
+#pragma unroll
+                for (int u = 0; u < 16; ++u) { m = fmaxf(g[u].x + m, g[u].y); now[u] = m; }
+#pragma unroll
+                for (int u = 0; u < 16; ++u) after[j + u + 1] = now[u];
+            }
+            for (; j < nb; ++j) {
+                m = fmaxf(gates[j].x + m, gates[j].y);
                 after[j + 1] = m;
             }
         }
