@@ -1293,7 +1293,7 @@ def _lotazen_sizes(width, heads, kv_heads, dim, lin_heads, lin_dim, lin_vdim, ex
                shared=dict(ff=shared_ff, limit=7.0))
     pair = dict(type="parallel", mixer=dict(left=left, right=recurrent, left_scale=0.5, right_scale=0.5), mlp=mlp)
     memory = lambda kind: dict(type=kind, mixer=dict(recurrent, gate_cap=15.0), mlp=mlp)
-    return dict(architecture="Lotazen", vocab=vocab, width=width, norm=dict(eps=1e-6), max_positions=8192, logit_softcap=30.0,
+    return dict(architecture="Lotazen", vocab=vocab, width=width, norm=dict(eps=1e-6), max_positions=8192, logit_softcap=25.0,
                 layers=[pair, memory("mlstm"), pair, memory("mlstm_2")] * 2)
 
 

@@ -50,7 +50,7 @@ def moe(experts, top, ff, limit, shared=None):
 CASE_A = dict(architecture="Lotazen", vocab=173, width=96, norm=dict(eps=1e-5), max_positions=400, logit_softcap=25.0, layers=[
     dict(pair(left(4, 2, 32, 32, 0.2, 10000.0, 16, 24, 4.0), right(3, 24, 16), 0.7, 1.3), mlp=moe(4, 4, 24, 1.2, (40, 0.6))),
     dict(mlstm(3, 20, 28, 6.0), mlp=moe(3, 3, 16, 2.0, (24, 5.0))),
-    dict(mlstm(2, 40, 16, 15.0, kind="mlstm_2"), mlp=None),
+    dict(mlstm(2, 40, 16, 16.0, kind="mlstm_2"), mlp=None),
     dict(pair(left(6, 1, 16, 16, 0.3, 300.0, 16, 7), right(2, 64, 80), 1.0, 0.4), mlp=moe(5, 5, 32, 0.9, (16, 3.0))),
 ])
 # one expert a token and two of five, no shared expert, no cap; windows of one position and longer than every request; one
@@ -72,8 +72,8 @@ CASE_C = dict(architecture="Lotazen", vocab=53, width=70, norm=dict(eps=1e-5), m
 # longer requests over pages of 16: heads of 128 whose whole 128-token tiles take the tensor-memory kernel with a window that is
 # a multiple of neither a page nor a key tile; requests beyond the chunked scan's length
 CASE_D = dict(architecture="Lotazen", vocab=301, width=256, norm=dict(eps=1e-5), max_positions=512, logit_softcap=20.0, layers=[
-    dict(pair(left(4, 2, 128, 128, 0.09, 100000.0, 48, 100, 4.0), right(4, 32, 48), 0.8, 0.9), mlp=moe(4, 4, 40, 1.0, (64, 2.0))),
-    dict(mlstm(4, 32, 64, 15.0), mlp=moe(2, 2, 72, 1.5, (40, 1.0))),
+    dict(pair(left(4, 2, 128, 128, 0.09, 100000.0, 48, 100, 4.0), right(4, 32, 40), 0.85, 0.95), mlp=moe(4, 4, 40, 1.0, (64, 2.0))),
+    dict(mlstm(4, 32, 72, 14.0), mlp=moe(2, 2, 72, 1.4, (40, 0.9))),
     dict(pair(left(2, 2, 64, 64, 0.125, 10000.0, 64, 300), right(2, 128, 64), 1.1, 0.6), mlp=None),
     dict(mlstm(2, 64, 130, 8.0, kind="mlstm_2"), mlp=moe(3, 3, 48, 3.0, (24, 0.7))),
 ])
