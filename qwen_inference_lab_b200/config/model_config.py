@@ -626,3 +626,110 @@ class LotazenConfig:
 
     def __eq__(self, other):
         return isinstance(other, LotazenConfig) and self.to_dict() == other.to_dict()
+
+
+class BugidraConfig:
+    """Bugidra: a decoder whose layers are listed one by one in config.json.
+
+    ``vocab``, ``width``, ``norm.eps``, ``embedding.scale`` (what a token's row is multiplied by) and ``layers``.  A layer is a
+    ``delta`` mixer (the gated delta rule: ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``conv`` taps), a ``parallel`` one
+    (``left`` an attention: ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale``, ``rot``; ``right`` a retention: ``heads``,
+    ``dim``, ``vdim``, ``rot``, ``decay``, one per head) or an ``attention`` one (as ``left``, with an optional ``softcap`` and
+    ``v_mix``: its values are mixed with those of the first such layer), and a feed-forward: ``mlp`` null or ``dense``
+    (``ff``).  ``rot`` has ``base``, ``dims`` and optionally ``scaling`` with ``factor``, ``original``, ``fast`` and ``slow``.
+    The configuration is kept as the dictionary it came in; this class checks it and answers the few questions the engine
+    asks.  ``max_positions`` (not a key of the design; 2**20 unless given) only bounds a request.
+    """
+    architecture = "Bugidra"
+    model_type = "bugidra"
+    MOST_TAPS = 16           # of a short convolution
+
+    def __init__(self, data: dict):
+        self.data = data
+        for key in ("vocab", "width"):
+            if not _positive_int(data.get(key)):
+                raise ConfigError(f"{key} must be a positive integer, got {data.get(key)!r}")
+        eps = (data.get("norm") or {}).get("eps")
+        if not _positive_number(eps):
+            raise ConfigError(f"norm.eps must be a positive number, got {eps!r}")
+        scale = (data.get("embedding") or {}).get("scale", 1.0)
+        if isinstance(scale, bool) or not isinstance(scale, (int, float)):
+            raise ConfigError(f"embedding.scale must be a number, got {scale!r}")
+        layers = data.get("layers")
+        if not isinstance(layers, list) or not layers:
+            raise ConfigError("layers must be a non-empty list")
+        mixed_widths = set()
+        for index, layer in enumerate(layers):
+            where = f"layers[{index}]"
+            kind, mixer = layer.get("type"), layer.get("mixer")
+            if not isinstance(mixer, dict):
+                raise ConfigError(f"{where}.mixer must be an object")
+            if kind == "delta":
+                LarolornConfig._check_sizes(where, mixer, ("heads", "kv_heads", "dim", "vdim", "conv"))
+                self._check_heads(where, mixer)
+                if mixer["conv"] > self.MOST_TAPS:
+                    raise ConfigError(f"{where}.conv: {mixer['conv']} taps are more than {self.MOST_TAPS}")
+            elif kind == "attention":
+                self._check_attention(where, mixer)
+                cap = mixer.get("softcap")
+                if cap is not None and not _positive_number(cap):
+                    raise ConfigError(f"{where}.softcap must be a positive number or absent, got {cap!r}")
+                if mixer.get("v_mix"):
+                    mixed_widths.add(mixer["kv_heads"] * mixer["vdim"])
+            elif kind == "parallel":
+                left, right = mixer.get("left"), mixer.get("right")
+                if not isinstance(left, dict) or not isinstance(right, dict):
+                    raise ConfigError(f"{where}.mixer needs a left and a right mixer")
+                self._check_attention(where + ".left", left)
+                LarolornConfig._check_sizes(where + ".right", right, ("heads", "dim", "vdim"))
+                self._check_rotation(where + ".right", right)
+                decay = right.get("decay")
+                if not isinstance(decay, list) or len(decay) != right["heads"] \
+                        or any(isinstance(v, bool) or not isinstance(v, (int, float)) or not 0 <= v <= 1 for v in decay):
+                    raise ConfigError(f"{where}.right.decay must give one decay in [0, 1] per head")
+            else:
+                raise ConfigError(f"{where}.type {kind!r} is none of delta, parallel, attention")
+            mlp = layer.get("mlp")
+            if mlp is not None and (mlp.get("kind") != "dense" or not _positive_int(mlp.get("ff"))):
+                raise ConfigError(f"{where}.mlp must be null or dense with a positive ff, got {mlp!r}")
+        if len(mixed_widths) > 1:
+            raise ConfigError(f"layers with v_mix have values of different widths: {sorted(mixed_widths)}")
+        self.vocab_size, self.width, self.eps = data["vocab"], data["width"], float(eps)
+        self.embedding_scale, self.layers = float(scale), layers
+        self.max_positions = int(data.get("max_positions", 1 << 20))
+        eos = data.get("eos_token_id")
+        self.eos_token_ids = frozenset() if eos is None else frozenset(eos if isinstance(eos, list) else [eos])
+
+    @staticmethod
+    def _check_heads(where, mixer):
+        if mixer["heads"] % mixer["kv_heads"]:
+            raise ConfigError(f"{where}: {mixer['heads']} heads do not divide into {mixer['kv_heads']} kv heads")
+
+    @classmethod
+    def _check_attention(cls, where, mixer):
+        LarolornConfig._check_sizes(where, mixer, ("heads", "kv_heads", "dim", "vdim"))
+        cls._check_heads(where, mixer)
+        cls._check_rotation(where, mixer)
+        if not _positive_number(mixer.get("scale")):
+            raise ConfigError(f"{where}.scale must be a positive number, got {mixer.get('scale')!r}")
+
+    @staticmethod
+    def _check_rotation(where, mixer):
+        LarolornConfig._check_rotation(where, mixer, mixer["dim"])
+        scaling = mixer["rot"].get("scaling")
+        if scaling is not None and (not all(_positive_number(scaling.get(k)) for k in ("factor", "original", "fast", "slow"))
+                                    or not mixer["rot"]["base"] > 1):
+            raise ConfigError(f"{where}.rot.scaling needs positive factor, original, fast and slow, and a base above one; "
+                              f"got {scaling!r}")
+
+    @classmethod
+    def from_dict(cls, data: dict) -> "BugidraConfig":
+        if data.get("architecture", cls.architecture) != cls.architecture:
+            raise ConfigError(f"architecture {data.get('architecture')!r} is not {cls.architecture}")
+        return cls(json.loads(json.dumps(data)))
+
+    def to_dict(self) -> dict:
+        return json.loads(json.dumps(self.data)) | {"architecture": self.architecture}
+
+    def __eq__(self, other):
+        return isinstance(other, BugidraConfig) and self.to_dict() == other.to_dict()

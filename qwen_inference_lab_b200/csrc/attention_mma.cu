@@ -1,6 +1,7 @@
 // bfloat16 causal grouped-query attention over the paged cache on the tensor
 // cores (mma.sync m16n8k16, float32 accumulation, float32 softmax), compiled for
-// one head size: -DQIL_HEAD_DIM=<multiple of 16, at most 256>.
+// one head size: -DQIL_HEAD_DIM=<multiple of 16, at most 256>, and, where values have a
+// size of their own, -DQIL_V_DIM=<the same>.
 //
 // Two forms, one arithmetic (scores = q k^T * head_dim^-1/2 over keys j <= the
 // token's absolute position and inside the window; softmax; times v;
@@ -21,7 +22,8 @@
 //    many do.
 //
 // Key tiles and spans are aligned to absolute positions.
-// Cache layout of one layer: [page][2 (K,V)][kv_head][slot in page][head_dim].
+// Cache layout of one layer: [page][2 (K,V)][kv_head][slot in page][head_dim]; with a value size of its own a page is its
+// key rows [kv_head][slot][head_dim] followed by its value rows [kv_head][slot][v_dim].
 #include "common.cuh"
 
 #ifndef QIL_HEAD_DIM
@@ -30,6 +32,12 @@
 static_assert(QIL_HEAD_DIM % 16 == 0 && QIL_HEAD_DIM >= 16 && QIL_HEAD_DIM <= 256,
               "the tensor-core attention takes head sizes 16, 32, ..., 256");
 
+#ifndef QIL_V_DIM
+#define QIL_V_DIM QIL_HEAD_DIM
+#endif
+static_assert(QIL_V_DIM % 16 == 0 && QIL_V_DIM >= 16 && QIL_V_DIM <= 256,
+              "the tensor-core attention takes value sizes 16, 32, ..., 256");
+
 QIL_ERROR_STORAGE
 
 #define KV_TILE 64          // key positions per shared-memory tile
@@ -37,7 +45,10 @@ QIL_ERROR_STORAGE
 #define MAX_DECODE_SPAN 8192 // most key positions per block (single tokens)
 
 constexpr int D = QIL_HEAD_DIM;
+constexpr int E = QIL_V_DIM;         // values and outputs
+constexpr bool ONE_SIZE = D == E;
 constexpr int LDS = D + 8;           // shared-memory row stride in elements: rows start 16 bytes apart mod 128
+constexpr int LDV = E + 8;           // of a value row
 constexpr int KSTEPS = D / 16;
 constexpr bool Q_IN_REGS = (D <= 128);
 
@@ -89,7 +100,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 struct AttnParams {
     const bf16* q;            // [N, Hq, D]
     const bf16* kv;           // one layer's pages
-    bf16* out;                // [N, Hq, D]
+    bf16* out;                // [N, Hq, E]
     const int* block_table;
     int table_stride;
     int n_q_heads, n_kv_heads, page_size, num_pages, window;
@@ -97,7 +108,7 @@ struct AttnParams {
     // row per (kv head, slot), which is the key, and whose leading columns are the value: no value row is stored
     // or read, the value tile is the key tile, and the output's trailing columns hold sums the caller ignores
     int planes;
-    // how many leading columns of a value row anyone reads (D, or with shared rows the value's width rounded up to
+    // how many leading columns of a value row anyone reads (E, or with shared rows the value's width rounded up to
     // 16): the weighted sum is not computed for the rest, whose output columns stay zero
     int v_cols;
     float scale_log2;         // head_dim^-1/2 * log2(e)
@@ -149,7 +160,18 @@ __device__ __forceinline__ int kv_row_offset(const AttnParams& p, const int* pag
     if (pos < lo || pos > hi || pos / p.page_size >= p.table_stride) return -1;
     const int page = pages[pos / p.page_size - first_page];
     if (page < 0 || page >= p.num_pages) return -1;
-    return (int)((((size_t)page * p.planes * p.n_kv_heads + kv_head) * p.page_size + (pos % p.page_size)) * (D / 8));
+    const int row = kv_head * p.page_size + pos % p.page_size;
+    if (ONE_SIZE) return (int)(((size_t)page * p.planes * p.n_kv_heads * p.page_size + row) * (D / 8));
+    return (int)((size_t)page * p.n_kv_heads * p.page_size * ((D + E) / 8) + (size_t)row * (D / 8));
+}
+// Where the value row of the key row at `off` starts, in the same units.
+__device__ __forceinline__ int value_row_offset(const AttnParams& p, int off) {
+    if (off < 0) return -1;
+    const int plane = p.n_kv_heads * p.page_size * (D / 8);
+    if (ONE_SIZE) return off + plane;
+    const int page_units = p.n_kv_heads * p.page_size * ((D + E) / 8);
+    const int page = off / page_units, row = (off - page * page_units) / (D / 8);
+    return page * page_units + plane + row * (E / 8);
 }
 
 // Queue the copies of 64 key rows and 64 value rows into shared memory; rows without an offset are
@@ -167,7 +189,16 @@ __device__ __forceinline__ void issue_kv_tile(const AttnParams& p, const int* ro
         const bool valid = off >= 0;
         const bf16* src = p.kv + (size_t)(valid ? off : 0) * 8 + piece * 8;
         cp_async16(sK + row * LDS + piece * 8, src, valid);
-        if (p.planes == 2) cp_async16(sV + row * LDS + piece * 8, src + v_plane, valid);
+        if (ONE_SIZE && p.planes == 2) cp_async16(sV + row * LDS + piece * 8, src + v_plane, valid);
+    }
+    if (ONE_SIZE) return;
+    constexpr int CPV = E / 8;
+#pragma unroll
+    for (int i = 0; i < KV_TILE * CPV / 128; ++i) {
+        const int idx = i * 128 + tid;
+        const int row = idx / CPV, piece = idx % CPV;
+        const int off = value_row_offset(p, row_off[row]);
+        cp_async16(sV + row * LDV + piece * 8, p.kv + (size_t)(off >= 0 ? off : 0) * 8 + piece * 8, off >= 0);
     }
 }
 
@@ -179,8 +210,8 @@ __device__ __forceinline__ void attn_prefill_tile(const AttnParams& p, const int
     // [K stage 0][K stage 1][V stage 0][V stage 1]; when the queries live in registers (head sizes up to
     // 128) their tile borrows K stage 1 until the fragments are loaded, else it has a region of its own
     bf16* sK = reinterpret_cast<bf16*>(smem_raw);      // [2][64][LDS]
-    bf16* sV = p.planes == 2 ? sK + 2 * KV_TILE * LDS : sK;   // [2][64][LDS]; shared rows: the key tiles themselves
-    bf16* sQ = Q_IN_REGS ? sK + KV_TILE * LDS : sV + 2 * KV_TILE * LDS;   // [64][LDS]
+    bf16* sV = p.planes == 2 ? sK + 2 * KV_TILE * LDS : sK;   // [2][64][LDV]; shared rows: the key tiles themselves
+    bf16* sQ = Q_IN_REGS ? sK + KV_TILE * LDS : sV + 2 * KV_TILE * LDV;   // [64][LDS]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int kv_head = head / (p.n_q_heads / p.n_kv_heads);
     // info: (first token in the flat batch, its absolute position, rows in the tile, block-table row)
@@ -224,9 +255,9 @@ __device__ __forceinline__ void attn_prefill_tile(const AttnParams& p, const int
                         sQ + (warp * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDS + ks * 16 + (lane >> 4) * 8);
         __syncthreads();               // K stage 1 is free for the second tile
     }
-    float o[D / 8][4];
+    float o[E / 8][4];
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+    for (int i = 0; i < E / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
     const int row_a = warp * 16 + (lane >> 2), row_b = row_a + 8;
     const int pos_a = pos0 + row_a, pos_b = pos0 + row_b;
@@ -236,7 +267,7 @@ __device__ __forceinline__ void attn_prefill_tile(const AttnParams& p, const int
     for (int tile = first_tile; tile <= last_tile; ++tile) {
         const int buf = (tile - first_tile) & 1;
         if (tile + 1 <= last_tile)
-            issue_kv_tile(p, row_off[buf ^ 1], sK + (buf ^ 1) * KV_TILE * LDS, sV + (buf ^ 1) * KV_TILE * LDS, tid);
+            issue_kv_tile(p, row_off[buf ^ 1], sK + (buf ^ 1) * KV_TILE * LDS, sV + (buf ^ 1) * KV_TILE * LDV, tid);
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
@@ -244,7 +275,7 @@ __device__ __forceinline__ void attn_prefill_tile(const AttnParams& p, const int
         if (tile + 2 <= last_tile && tid < KV_TILE)
             row_off[buf][tid] = kv_row_offset(p, table, 0, kv_head, (tile + 2) * KV_TILE + tid, lo, hi);
         const bf16* tK = sK + buf * KV_TILE * LDS;
-        const bf16* tV = sV + buf * KV_TILE * LDS;
+        const bf16* tV = sV + buf * KV_TILE * LDV;
 
         float s[KV_TILE / 8][4];
 #pragma unroll
@@ -327,7 +358,7 @@ __device__ __forceinline__ void attn_prefill_tile(const AttnParams& p, const int
         l_a = l_a * corr_a + sum_a;
         l_b = l_b * corr_b + sum_b;
 #pragma unroll
-        for (int i = 0; i < D / 8; ++i) { o[i][0] *= corr_a; o[i][1] *= corr_a; o[i][2] *= corr_b; o[i][3] *= corr_b; }
+        for (int i = 0; i < E / 8; ++i) { o[i][0] *= corr_a; o[i][1] *= corr_a; o[i][2] *= corr_b; o[i][3] *= corr_b; }
 #pragma unroll
         for (int kt = 0; kt < KV_TILE / 16; ++kt) {
             unsigned a[4];
@@ -336,11 +367,11 @@ __device__ __forceinline__ void attn_prefill_tile(const AttnParams& p, const int
             a[2] = pack_bf16(s[2 * kt + 1][0], s[2 * kt + 1][1]);
             a[3] = pack_bf16(s[2 * kt + 1][2], s[2 * kt + 1][3]);
 #pragma unroll
-            for (int dp = 0; dp < D / 16; ++dp) {
+            for (int dp = 0; dp < E / 16; ++dp) {
                 if (dp * 16 >= p.v_cols) continue;      // the same for all threads; the loop stays unrolled
                 unsigned b0, b1, b2, b3;
                 ldmatrix_x4_trans(b0, b1, b2, b3,
-                                  tV + (kt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDS + dp * 16 + (lane >> 4) * 8);
+                                  tV + (kt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDV + dp * 16 + (lane >> 4) * 8);
                 mma_bf16(o[2 * dp], a, b0, b1);
                 mma_bf16(o[2 * dp + 1], a, b2, b3);
             }
@@ -355,20 +386,20 @@ __device__ __forceinline__ void attn_prefill_tile(const AttnParams& p, const int
     }
     const float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) {
+    for (int dt = 0; dt < E / 8; ++dt) {
         const int col = dt * 8 + (lane & 3) * 2;
         if (row_a < rows)
-            *reinterpret_cast<unsigned*>(p.out + ((size_t)(n0 + row_a) * p.n_q_heads + head) * D + col) =
+            *reinterpret_cast<unsigned*>(p.out + ((size_t)(n0 + row_a) * p.n_q_heads + head) * E + col) =
                 pack_bf16(o[dt][0] * inv_a, o[dt][1] * inv_a);
         if (row_b < rows)
-            *reinterpret_cast<unsigned*>(p.out + ((size_t)(n0 + row_b) * p.n_q_heads + head) * D + col) =
+            *reinterpret_cast<unsigned*>(p.out + ((size_t)(n0 + row_b) * p.n_q_heads + head) * E + col) =
                 pack_bf16(o[dt][2] * inv_b, o[dt][3] * inv_b);
     }
 }
 
 // Heads vary fastest, so all heads of the longest tile start first (tiles come sorted, longest first).
 template <bool MOD>
-__global__ void __launch_bounds__(128, (QIL_HEAD_DIM <= 128) ? 3 : 1)
+__global__ void __launch_bounds__(128, (QIL_HEAD_DIM <= 128 && QIL_V_DIM <= 128) ? 3 : 1)
 attn_prefill_kernel(AttnParams p, const int4* __restrict__ tile_info) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     attn_prefill_tile<MOD>(p, tile_info[blockIdx.y], (int)blockIdx.x, smem_raw);
@@ -487,7 +518,7 @@ __device__ __forceinline__ void warp_norm_rotate_head(const bf16* __restrict__ s
 __device__ __forceinline__ void merge_spans_of_head(const AttnParams& p, const float* __restrict__ part_o,
                                                     const float* __restrict__ part_ml, int d_idx, int n, int head,
                                                     int n_spans, int s_lo, int s_hi, bool uncovered, int lane) {
-    constexpr int COLS = (D + 31) / 32, BATCH = 16;
+    constexpr int COLS = (E + 31) / 32, BATCH = 16;
     const size_t base = ((size_t)d_idx * p.n_q_heads + head) * n_spans;
     float mx = -INFINITY, sum = 0.f;
     float acc[COLS];
@@ -505,7 +536,7 @@ __device__ __forceinline__ void merge_spans_of_head(const AttnParams& p, const f
 #pragma unroll
             for (int i = 0; i < COLS; ++i) {
                 const int col = lane + i * 32;
-                o_part[j][i] = col < D ? __ldcg(part_o + slot * D + col) : 0.f;
+                o_part[j][i] = col < E ? __ldcg(part_o + slot * E + col) : 0.f;
             }
         }
         float batch_max = m[0];
@@ -531,15 +562,15 @@ __device__ __forceinline__ void merge_spans_of_head(const AttnParams& p, const f
 #pragma unroll
     for (int i = 0; i < COLS; ++i) {
         const int col = lane + i * 32;
-        if (col < D)
-            p.out[((size_t)n * p.n_q_heads + head) * D + col] =
+        if (col < E)
+            p.out[((size_t)n * p.n_q_heads + head) * E + col] =
                 __float2bfloat16_rn(uncovered ? __int_as_float(0x7fc00000) : acc[i] * inv);
     }
 }
 
 // ------------------------------------------------------------------ single tokens: spans
 // decode_info: (token in the flat batch, its absolute position, block-table row, unused) per token.
-// part_o  [n_decode, Hq, n_spans, D] float32, unnormalised; part_ml [n_decode, Hq, n_spans, 2] (max, sum).
+// part_o  [n_decode, Hq, n_spans, E] float32, unnormalised; part_ml [n_decode, Hq, n_spans, 2] (max, sum).
 //
 // The work of one block, as a function of its place in the grid (``block_x`` of ``grid_x``, ``d_idx``, ``span``)
 // so that a kernel that walks several such places in a loop can call it too.  ``wait_for_inputs`` is called once,
@@ -554,8 +585,8 @@ __device__ __forceinline__ void attn_decode_span_block(
     bf16* sQ = reinterpret_cast<bf16*>(smem_raw);      // [16][LDS]
     bf16* sK = sQ + 16 * LDS;                           // [2][64][LDS]
     const bool shared = p.planes == 1;                  // the value rows are the key rows: see AttnParams
-    bf16* sV = shared ? sK : sK + 2 * KV_TILE * LDS;    // [2][64][LDS]
-    int* s_pages = reinterpret_cast<int*>(sV + 2 * KV_TILE * LDS);   // [span_len / page_size + 2]
+    bf16* sV = shared ? sK : sK + 2 * KV_TILE * LDS;    // [2][64][LDV]
+    int* s_pages = reinterpret_cast<int*>(sV + 2 * KV_TILE * LDV);   // [span_len / page_size + 2]
     // Up to qil_wait_for_producer() below only memory that no kernel of this step writes is read:
     // the step's description, the block table, and keys and values of earlier positions.
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -599,7 +630,7 @@ __device__ __forceinline__ void attn_decode_span_block(
     // only warp-level barriers around them, and asks for the rows of tile t + 2 as soon as it is done
     // with the rows of tile t (K after the scores, V after the output), so two tiles are in flight per
     // warp instead of one per block.  cp.async groups of a thread, in order: K0, V0, K1, V1, K2, ...
-    constexpr int CPR = D / 8;                   // 16-byte pieces per row
+    constexpr int CPR = D / 8, CPV = E / 8;      // 16-byte pieces per key row and per value row
     const size_t v_plane = (size_t)p.n_kv_heads * p.page_size * D;
     auto row_offset = [&](int tile) {            // lanes 0..15: where this warp's row `lane` of the tile starts
         return (lane < 16 && tile <= last_tile)
@@ -615,16 +646,27 @@ __device__ __forceinline__ void attn_decode_span_block(
             cp_async16_stream(dst + row * LDS + piece * 8, p.kv + (size_t)(valid ? off : 0) * 8 + piece * 8 + (valid ? plane : 0), valid);
         }
     };
+    auto issue_values = [&](int offset_of_lane, bf16* dst) {       // the values of the rows of issue_rows
+        if (ONE_SIZE) { issue_rows(offset_of_lane, dst, shared ? 0 : v_plane); return; }
+        const int value_of_lane = value_row_offset(p, offset_of_lane);
+#pragma unroll
+        for (int i = 0; i < 16 * CPV / 32; ++i) {
+            const int idx = i * 32 + lane;
+            const int row = idx / CPV, piece = idx % CPV;
+            const int off = __shfl_sync(0xffffffffu, value_of_lane, row);
+            cp_async16_stream(dst + row * LDV + piece * 8, p.kv + (size_t)(off >= 0 ? off : 0) * 8 + piece * 8, off >= 0);
+        }
+    };
     bf16* const my_k = sK + warp * 16 * LDS;    // this warp's rows of buffer 0; buffer 1 lies KV_TILE rows further
-    bf16* const my_v = sV + warp * 16 * LDS;
-    constexpr int BUFFER = KV_TILE * LDS;
+    bf16* const my_v = sV + warp * 16 * LDV;
+    constexpr int BUFFER = KV_TILE * LDS, V_BUFFER = KV_TILE * LDV;
     const int off0 = row_offset(first_tile), off1 = row_offset(first_tile + 1);
     // The first tile starts before the wait unless it holds this step's own position, whose key and
     // value are written below (or by the kernel before this one).
     const bool early = first_tile != hi / KV_TILE;
     if (early) issue_rows(off0, my_k, 0);
     cp_async_commit();
-    if (early && !shared) issue_rows(off0, my_v, v_plane);
+    if (early && !shared) issue_values(off0, my_v);
     cp_async_commit();
     wait_for_inputs();
     if (tail.qkv == nullptr) {   // finished queries: the heads of this kv head, 8 threads per row
@@ -664,18 +706,18 @@ __device__ __forceinline__ void attn_decode_span_block(
         }
         __syncthreads();
     }
-    if (!early) { issue_rows(off0, my_k, 0); if (!shared) issue_rows(off0, my_v, v_plane); }
+    if (!early) { issue_rows(off0, my_k, 0); if (!shared) issue_values(off0, my_v); }
     if (first_tile + 1 <= last_tile) issue_rows(off1, my_k + BUFFER, 0);
     cp_async_commit();
-    if (first_tile + 1 <= last_tile && !shared) issue_rows(off1, my_v + BUFFER, v_plane);
+    if (first_tile + 1 <= last_tile && !shared) issue_values(off1, my_v + V_BUFFER);
     cp_async_commit();
     cp_async_wait<1>();          // the queries and the first tiles' keys; only the second tile's values may be under way
     __syncthreads();             // the query rows are every warp's
 
     unsigned qf[Q_IN_REGS ? KSTEPS : 1][4];
-    float o[D / 8][4];
+    float o[E / 8][4];
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+    for (int i = 0; i < E / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
 
     for (int tile = first_tile; tile <= last_tile; ++tile) {
@@ -693,7 +735,7 @@ __device__ __forceinline__ void attn_decode_span_block(
                             sQ + (((lane >> 3) & 1) * 8 + (lane & 7)) * LDS + ks * 16 + (lane >> 4) * 8);
         }
         const bf16* tK = my_k + buf * BUFFER;   // this warp's 16 keys of the tile
-        const bf16* tV = my_v + buf * BUFFER;
+        const bf16* tV = my_v + buf * V_BUFFER;
         float s[2][4];
         s[0][0] = s[0][1] = s[0][2] = s[0][3] = 0.f;
         s[1][0] = s[1][1] = s[1][2] = s[1][3] = 0.f;
@@ -746,7 +788,7 @@ __device__ __forceinline__ void attn_decode_span_block(
         l_a = l_a * corr_a + (s[0][0] + s[0][1] + s[1][0] + s[1][1]);
         l_b = l_b * corr_b + (s[0][2] + s[0][3] + s[1][2] + s[1][3]);
 #pragma unroll
-        for (int i = 0; i < D / 8; ++i) { o[i][0] *= corr_a; o[i][1] *= corr_a; o[i][2] *= corr_b; o[i][3] *= corr_b; }
+        for (int i = 0; i < E / 8; ++i) { o[i][0] *= corr_a; o[i][1] *= corr_a; o[i][2] *= corr_b; o[i][3] *= corr_b; }
         unsigned a[4];
         a[0] = pack_bf16(s[0][0], s[0][1]);
         a[1] = pack_bf16(s[0][2], s[0][3]);
@@ -755,15 +797,15 @@ __device__ __forceinline__ void attn_decode_span_block(
         cp_async_wait<3>();          // this tile's values: K(t+1), V(t+1), K(t+2) may still be under way
         __syncwarp();
 #pragma unroll
-        for (int dp = 0; dp < D / 16; ++dp) {
+        for (int dp = 0; dp < E / 16; ++dp) {
             if (dp * 16 >= p.v_cols) continue;
             unsigned b0, b1, b2, b3;
-            ldmatrix_x4_trans(b0, b1, b2, b3, tV + (((lane >> 3) & 1) * 8 + (lane & 7)) * LDS + dp * 16 + (lane >> 4) * 8);
+            ldmatrix_x4_trans(b0, b1, b2, b3, tV + (((lane >> 3) & 1) * 8 + (lane & 7)) * LDV + dp * 16 + (lane >> 4) * 8);
             mma_bf16(o[2 * dp], a, b0, b1);
             mma_bf16(o[2 * dp + 1], a, b2, b3);
         }
         __syncwarp();
-        if (tile + 2 <= last_tile) issue_rows(off2, my_v + buf * BUFFER, shared ? 0 : v_plane);
+        if (tile + 2 <= last_tile) issue_values(off2, my_v + buf * V_BUFFER);
         cp_async_commit();
     }
     cp_async_wait<0>();
@@ -774,17 +816,17 @@ __device__ __forceinline__ void attn_decode_span_block(
     // merge the four warps' (max, sum, acc) through shared memory (the tile buffers are free now)
     float* wm = reinterpret_cast<float*>(sK);          // [4][16]
     float* wl = wm + 4 * 16;                            // [4][16]
-    float* wo = wl + 4 * 16;                            // [4][16][D]
+    float* wo = wl + 4 * 16;                            // [4][16][E]
     const int ra = lane >> 2, rb = ra + 8;
     if ((lane & 3) == 0) {
         wm[warp * 16 + ra] = m_a; wm[warp * 16 + rb] = m_b;
         wl[warp * 16 + ra] = l_a; wl[warp * 16 + rb] = l_b;
     }
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) {
+    for (int dt = 0; dt < E / 8; ++dt) {
         const int col = dt * 8 + (lane & 3) * 2;
-        wo[(warp * 16 + ra) * D + col] = o[dt][0]; wo[(warp * 16 + ra) * D + col + 1] = o[dt][1];
-        wo[(warp * 16 + rb) * D + col] = o[dt][2]; wo[(warp * 16 + rb) * D + col + 1] = o[dt][3];
+        wo[(warp * 16 + ra) * E + col] = o[dt][0]; wo[(warp * 16 + ra) * E + col + 1] = o[dt][1];
+        wo[(warp * 16 + rb) * E + col] = o[dt][2]; wo[(warp * 16 + rb) * E + col + 1] = o[dt][3];
     }
     __syncthreads();
     // The spans that hold keys of this token (the others returned at the top).  n_spans * span_len short of the
@@ -795,27 +837,27 @@ __device__ __forceinline__ void attn_decode_span_block(
     const bool uncovered = s_hi >= n_spans;
     if (uncovered) s_hi = n_spans - 1;
     const bool alone = s_lo == s_hi;             // this block holds the whole context: its sums are the result
-    for (int idx = tid; idx < gcount * D; idx += 128) {
-        const int r = idx / D, col = idx - r * D;
+    for (int idx = tid; idx < gcount * E; idx += 128) {
+        const int r = idx / E, col = idx - r * E;
         float mx = fmaxf(fmaxf(wm[r], wm[16 + r]), fmaxf(wm[32 + r], wm[48 + r]));
         const float ms = (mx == -INFINITY) ? 0.f : mx;
         float acc = 0.f, sum = 0.f;
 #pragma unroll
         for (int w = 0; w < 4; ++w) {
             const float f = fast_exp2(wm[w * 16 + r] - ms);
-            acc += f * wo[(w * 16 + r) * D + col];
+            acc += f * wo[(w * 16 + r) * E + col];
             sum += f * wl[w * 16 + r];
         }
         const int head = kv_head * group + g0 + r;
         if (alone) {
             if (p.sink) sum += sink_weight(p, head, mx);
             const float inv = sum > 0.f ? 1.f / sum : 0.f;
-            p.out[((size_t)n * p.n_q_heads + head) * D + col] =
+            p.out[((size_t)n * p.n_q_heads + head) * E + col] =
                 __float2bfloat16_rn(uncovered ? __int_as_float(0x7fc00000) : acc * inv);
             continue;
         }
         const size_t slot = ((size_t)d_idx * p.n_q_heads + head) * n_spans + span;
-        part_o[slot * D + col] = acc;
+        part_o[slot * E + col] = acc;
         if (col == 0) { part_ml[slot * 2] = mx; part_ml[slot * 2 + 1] = sum; }
     }
     if (alone || tickets == nullptr) return;        // no counters: a merge kernel follows
@@ -886,7 +928,7 @@ static int fill_params(AttnParams& p, const void* q, const void* kv, void* out, 
     p.q = (const bf16*)q; p.kv = (const bf16*)kv; p.out = (bf16*)out;
     p.block_table = block_table; p.table_stride = table_stride;
     p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads; p.page_size = page_size; p.num_pages = num_pages;
-    p.window = window; p.planes = 2; p.v_cols = D;
+    p.window = window; p.planes = 2; p.v_cols = E;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.slopes_log2 = nullptr;
     p.scale = scale; p.softcap = 0.f; p.tanh_arg = p.cap_log2 = 0.f; p.dist_bias = nullptr; p.dist_len = 0; p.chunk = 0; p.sink = 0; p.sink_log2 = nullptr;
@@ -915,7 +957,7 @@ static bool has_options(const AttnParams& p) {
 // Shared memory of the span kernel: query rows, two stages of key and value tiles (reused for the
 // merge of the four warps), and the span's page ids.
 static int decode_smem_bytes(int span_len, int page_size, int planes = 2) {
-    const int tile_bytes = (16 + 2 * planes * KV_TILE) * LDS * (int)sizeof(bf16);
+    const int tile_bytes = ((16 + 2 * KV_TILE) * LDS + (planes - 1) * 2 * KV_TILE * LDV) * (int)sizeof(bf16);
     return tile_bytes + (span_len / page_size + 3) * (int)sizeof(int);
 }
 
@@ -947,6 +989,7 @@ static int check_decode_span(int span_len, int n_spans) {
 }
 
 extern "C" int qil_attn_head_dim() { return D; }
+extern "C" int qil_attn_v_dim() { return E; }
 extern "C" int qil_attn_max_decode_span() { return MAX_DECODE_SPAN; }
 
 // tile_info: int32 [n_tiles, 4] = (first token, its absolute position, rows <= 64, block-table row).
@@ -961,15 +1004,16 @@ static int launch_prefill(const void* q, const void* kv, void* out, const int* t
     if (fill_params(p, q, kv, out, block_table, table_stride, n_q_heads, n_kv_heads, page_size, num_pages,
                     window, scale)) return -1;
     if (planes != 1 && planes != 2) QIL_REFUSE("attention: a page holds 1 or 2 rows per position, not %d", planes);
-    if (v_cols < 0 || v_cols > D) QIL_REFUSE("attention: %d value columns of %d", v_cols, D);
+    if (v_cols < 0 || v_cols > E) QIL_REFUSE("attention: %d value columns of %d", v_cols, E);
+    if (planes == 1 && !ONE_SIZE) QIL_REFUSE("attention: shared rows have values as wide as keys");
     p.planes = planes;
     if (v_cols > 0) p.v_cols = (v_cols + 15) / 16 * 16;
     p.slopes_log2 = slopes_log2;
     if (fill_options(p, softcap, dist_bias, dist_len, chunk, sink, sink_log2)) return -1;
     if (n_tiles > 65535) QIL_REFUSE("attention: %d query tiles in one launch; at most 65535", n_tiles);
     if ((uintptr_t)tile_info & 15) QIL_REFUSE("attention: tile_info must be 16-byte aligned");
-    const int full = ((Q_IN_REGS ? 0 : Q_TILE) + 4 * KV_TILE) * LDS * (int)sizeof(bf16);
-    const int smem = ((Q_IN_REGS ? 0 : Q_TILE) + 2 * planes * KV_TILE) * LDS * (int)sizeof(bf16);
+    const int keys = ((Q_IN_REGS ? 0 : Q_TILE) + 2 * KV_TILE) * LDS * (int)sizeof(bf16), values = 2 * KV_TILE * LDV * (int)sizeof(bf16);
+    const int full = keys + values, smem = keys + (planes - 1) * values;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, full);
@@ -1030,7 +1074,7 @@ extern "C" int qil_attn_prefill(const void* q, const void* kv, void* out, const 
 }
 
 // decode_info: int32 [n_decode, 4] = (token, its absolute position, block-table row, 0).
-// Scratch: part_o needs n_decode * Hq * n_spans * D floats, part_ml n_decode * Hq * n_spans * 2 floats, tickets
+// Scratch: part_o needs n_decode * Hq * n_spans * E floats, part_ml n_decode * Hq * n_spans * 2 floats, tickets
 // n_decode * n_kv_heads * ceil(Hq / n_kv_heads / 16) unsigned ints that are zero before the first launch (every
 // launch leaves them zero again), or null: then a second kernel merges the spans (what many tokens want: a
 // ticket costs every block a fence and an atomic at its end, a merge kernel costs one launch).
@@ -1050,8 +1094,10 @@ static int launch_decode(const void* q, const void* kv, void* out, const int* de
     if (fill_params(p, q, kv, out, block_table, table_stride, n_q_heads, n_kv_heads, page_size, num_pages,
                     window, scale)) return -1;
     if (planes != 1 && planes != 2) QIL_REFUSE("attention: a page holds 1 or 2 rows per position, not %d", planes);
+    if (!ONE_SIZE && tail.qkv != nullptr) QIL_REFUSE("attention: the projection's tail has values as wide as keys");
     if (planes == 1 && tail.qkv != nullptr) QIL_REFUSE("attention: the projection's tail writes value rows; shared rows have none");
-    if (v_cols < 0 || v_cols > D) QIL_REFUSE("attention: %d value columns of %d", v_cols, D);
+    if (v_cols < 0 || v_cols > E) QIL_REFUSE("attention: %d value columns of %d", v_cols, E);
+    if (planes == 1 && !ONE_SIZE) QIL_REFUSE("attention: shared rows have values as wide as keys");
     p.planes = planes;
     if (v_cols > 0) p.v_cols = (v_cols + 15) / 16 * 16;
     p.slopes_log2 = slopes_log2;

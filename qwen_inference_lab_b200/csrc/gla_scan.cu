@@ -52,6 +52,7 @@
 // columns (o over max(|n . q|, floor) + 1e-6, over its own root mean square, times a weight per element of all heads and
 // sigmoid of a gate); else mlstm_finish does, from the raw outputs.
 #include "common.cuh"
+#include "head_norm_gate.cuh"
 
 #define GLA_TB 8
 
@@ -88,28 +89,6 @@ gla_decay_kernel(const T* __restrict__ low, int ld, const W* __restrict__ a2, co
         const W* a2_row = a2 + (size_t)c * rank;
         for (int j = 0; j < rank; ++j) z = fmaf(to_f32<W>(a2_row[j]), s_low[j], z);
         alpha[token * channels + c] = decay_from_logit(z, inv_tau);
-    }
-}
-
-template <typename T, typename W>
-__device__ __forceinline__ void gla_norm_gate_rows(const float* o_rows, int o_stride, int nb, size_t first_token,
-                                                   const T* g, int ld, const W* norm_w, float eps, int n_heads,
-                                                   int head, int e, T* out, int lane, int warp, int warps) {
-    for (int tb = warp; tb < nb; tb += warps) {
-        const float* o = o_rows + (size_t)tb * o_stride;
-        float ss = 0.f;
-        for (int c = lane; c < e; c += 32) ss = fmaf(o[c], o[c], ss);
-        ss = warp_sum(ss);
-        const float scale = 1.0f / sqrtf(ss / (float)e + eps);
-        const size_t token = first_token + tb;
-        for (int c = lane; c < e; c += 32) {
-            float y = o[c] * scale * to_f32<W>(norm_w[c]);
-            if (g != nullptr) {
-                const float gate = to_f32<T>(g[token * ld + head * e + c]);
-                y *= gate / (1.f + expf(-gate));
-            }
-            out[(token * n_heads + head) * e + c] = from_f32<T>(y);
-        }
     }
 }
 
@@ -309,7 +288,7 @@ gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __res
         }
         if (FUSE == GLA_NORM && MODE != GLA_OWN_STATE) {
             __syncthreads();
-            gla_norm_gate_rows<T, W>(so, tile_cols, nb, (size_t)(first + t0), g, ld, norm_w, eps, n_heads, head, e, out,
+            head_norm_gate_rows<T, W>(so, tile_cols, nb, (size_t)(first + t0), g, ld, norm_w, eps, n_heads, head, e, out,
                                      lane, warp, warps);
         }
         if (FUSE == GLA_MEMORY && MODE != GLA_OWN_STATE) {
@@ -380,7 +359,7 @@ gla_norm_gate_kernel(const float* __restrict__ o_raw, const T* __restrict__ g, i
     const size_t token = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int head = warp; head < n_heads; head += 8)
-        gla_norm_gate_rows<T, W>(o_raw + (token * n_heads + head) * e, 0, 1, token, g, ld, norm_w, eps, n_heads, head, e,
+        head_norm_gate_rows<T, W>(o_raw + (token * n_heads + head) * e, 0, 1, token, g, ld, norm_w, eps, n_heads, head, e,
                                  out, lane, 0, 1);
 }
 

@@ -387,16 +387,30 @@ extern "C" int qil_norm_join(void* x, int x_dtype, const float* a, const void* w
 
 // Several branches of one layer join the stream at once (a layer whose sublayers read the same normed row), and the
 // norm of whoever reads the stream next rides along:
-//   x += sum_k scale_k * b_k + sum_s y[row * top + s],   rows = norm(x; next_w)   (rows optional; without next_w: x rounded)
-// b_k: up to four float32 branches [N, width]; y (optional): float32 rows of a token's `top` routed experts.  norm as in
-// norm_join.  float32 arithmetic; every sum in the order of the arguments, every reduction a fixed tree over one row.
+//   x += sum_k scale_k * b_k + sum_s y[row * top + s],   rows = norm(x; next)   (rows optional; without next.w: x rounded)
+// b_k: up to four float32 branches [N, width]; a branch with a weight w_k (float32 [width]) is first divided by its root mean
+// square and multiplied by it, b_k / sqrt(mean(b_k^2) + eps) * w_k.  y (optional): float32 rows of a token's `top` routed
+// experts.  norm as in norm_join, or the one without statistics (below).  float32 arithmetic; every sum in the order of the
+// arguments, every reduction a fixed tree over one row.
 #define JOIN_MOST 4
+#define JOIN_MOST_NORMED 2       // of the branches, that the register form takes
 struct JoinBranches {
     const float* b[JOIN_MOST];
+    const float* w[JOIN_MOST];       // null: the branch as it is
     float scale[JOIN_MOST];
     int n;
+    float eps;
     const float* y;
     int top;
+};
+#define JOIN_RMS 0
+#define JOIN_LAYER 1
+#define JOIN_TANH 2
+struct JoinNext {
+    const void* w;       // [width]; null: no norm
+    const void* b;       // [width], of w's type (JOIN_TANH)
+    float eps, alpha;
+    int kind;
 };
 
 template <typename T> __device__ __forceinline__ float4 join_load4(const T* p);
@@ -417,27 +431,44 @@ __device__ __forceinline__ void join_store4(bf16* p, float4 v) {
 }
 
 // Rows of up to 1024 * V4 values, a multiple of four, held in registers: 16 bytes a load.
-template <typename TX, typename W, typename TO, int V4>
+template <typename TX, typename W, typename TO, int V4, bool NORMED>
 __global__ void __launch_bounds__(256)
-branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, const W* __restrict__ next_w, float next_eps,
-                        int next_center, TO* __restrict__ rows) {
+branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext next, TO* __restrict__ rows) {
     __shared__ float scratch[32];
     qil_wait_for_producer();
     qil_release_consumer();
     const size_t row = blockIdx.x;
     TX* dst = x + row * width;
-    float4 v[V4];
-    float sum = 0.f;
+    float4 v[V4], stream[V4];
+    float4 held[NORMED ? JOIN_MOST_NORMED : 1][NORMED ? V4 : 1];      // the normed branches' rows
+    float ss[JOIN_MOST_NORMED] = {0.f, 0.f};
 #pragma unroll
     for (int c = 0; c < V4; ++c) {
         const int col = (threadIdx.x + c * 256) * 4;
-        v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        v[c] = stream[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (NORMED) {
+#pragma unroll
+            for (int m = 0; m < JOIN_MOST_NORMED; ++m) held[m][c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
         if (col >= width) continue;
+        stream[c] = join_load4<TX>(dst + col);
         float4 add = make_float4(0.f, 0.f, 0.f, 0.f);
+        int normed = 0;
 #pragma unroll
         for (int k = 0; k < JOIN_MOST; ++k) {
             if (k >= in.n) break;
             const float4 b = *reinterpret_cast<const float4*>(in.b[k] + row * width + col);
+            if (NORMED && in.w[k] != nullptr) {
+#pragma unroll
+                for (int m = 0; m < JOIN_MOST_NORMED; ++m)
+                    if (m == normed) {
+                        held[m][c] = b;
+                        ss[m] = fmaf(b.x, b.x, ss[m]); ss[m] = fmaf(b.y, b.y, ss[m]);
+                        ss[m] = fmaf(b.z, b.z, ss[m]); ss[m] = fmaf(b.w, b.w, ss[m]);
+                    }
+                ++normed;
+                continue;
+            }
             add.x = fmaf(in.scale[k], b.x, add.x); add.y = fmaf(in.scale[k], b.y, add.y);
             add.z = fmaf(in.scale[k], b.z, add.z); add.w = fmaf(in.scale[k], b.w, add.w);
         }
@@ -446,8 +477,36 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, const W*
                 const float4 b = *reinterpret_cast<const float4*>(in.y + (row * in.top + t) * width + col);
                 add.x += b.x; add.y += b.y; add.z += b.z; add.w += b.w;
             }
-        float4 now = join_load4<TX>(dst + col);
-        now.x += add.x; now.y += add.y; now.z += add.z; now.w += add.w;
+        v[c] = add;
+    }
+    if (NORMED) {
+        int normed = 0;
+#pragma unroll
+        for (int k = 0; k < JOIN_MOST; ++k) {
+            if (k >= in.n) break;
+            if (in.w[k] == nullptr) continue;
+#pragma unroll
+            for (int m = 0; m < JOIN_MOST_NORMED; ++m)
+                if (m == normed) {
+                    const float r = 1.0f / sqrtf(block_sum(ss[m], scratch) / (float)width + in.eps);
+#pragma unroll
+                    for (int c = 0; c < V4; ++c) {
+                        const int col = (threadIdx.x + c * 256) * 4;
+                        if (col >= width) continue;
+                        const float4 w = join_load4<float>(in.w[k] + col);
+                        v[c].x = fmaf(in.scale[k], held[m][c].x * r * w.x, v[c].x); v[c].y = fmaf(in.scale[k], held[m][c].y * r * w.y, v[c].y);
+                        v[c].z = fmaf(in.scale[k], held[m][c].z * r * w.z, v[c].z); v[c].w = fmaf(in.scale[k], held[m][c].w * r * w.w, v[c].w);
+                    }
+                }
+            ++normed;
+        }
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int c = 0; c < V4; ++c) {
+        const int col = (threadIdx.x + c * 256) * 4;
+        if (col >= width) continue;
+        float4 now = make_float4(stream[c].x + v[c].x, stream[c].y + v[c].y, stream[c].z + v[c].z, stream[c].w + v[c].w);
         now.x = round_to<TX>(now.x); now.y = round_to<TX>(now.y); now.z = round_to<TX>(now.z); now.w = round_to<TX>(now.w);
         join_store4(dst + col, now);
         v[c] = now;
@@ -455,6 +514,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, const W*
     }
     if (rows == nullptr) return;
     TO* out = rows + row * width;
+    const W* next_w = reinterpret_cast<const W*>(next.w);
     if (next_w == nullptr) {
 #pragma unroll
         for (int c = 0; c < V4; ++c) {
@@ -463,8 +523,20 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, const W*
         }
         return;
     }
+    if (next.kind == JOIN_TANH) {
+        const W* next_b = reinterpret_cast<const W*>(next.b);
+#pragma unroll
+        for (int c = 0; c < V4; ++c) {
+            const int col = (threadIdx.x + c * 256) * 4;
+            if (col >= width) continue;
+            const float4 w = join_load4<W>(next_w + col), b = join_load4<W>(next_b + col);
+            join_store4(out + col, make_float4(fmaf(tanhf(next.alpha * v[c].x), w.x, b.x), fmaf(tanhf(next.alpha * v[c].y), w.y, b.y),
+                                               fmaf(tanhf(next.alpha * v[c].z), w.z, b.z), fmaf(tanhf(next.alpha * v[c].w), w.w, b.w)));
+        }
+        return;
+    }
     float mean = 0.f;
-    if (next_center) mean = block_sum(sum, scratch) / (float)width;
+    if (next.kind == JOIN_LAYER) mean = block_sum(sum, scratch) / (float)width;
     float sq = 0.f;
 #pragma unroll
     for (int c = 0; c < V4; ++c) {
@@ -474,7 +546,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, const W*
         sq = fmaf(v[c].z, v[c].z, sq); sq = fmaf(v[c].w, v[c].w, sq);
     }
     sq = block_sum(sq, scratch);
-    const float scale = 1.0f / sqrtf(sq / (float)width + next_eps);
+    const float scale = 1.0f / sqrtf(sq / (float)width + next.eps);
 #pragma unroll
     for (int c = 0; c < V4; ++c) {
         const int col = (threadIdx.x + c * 256) * 4;
@@ -484,66 +556,99 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, const W*
     }
 }
 
-// Any width: the stream's row is read back by the threads that wrote it.
+// Any width and number of normed branches: the stream's row is read back by the threads that wrote it.
 template <typename TX, typename W, typename TO>
 __global__ void __launch_bounds__(256)
-branch_join_kernel(TX* __restrict__ x, JoinBranches in, int width, const W* __restrict__ next_w, float next_eps,
-                   int next_center, TO* __restrict__ rows) {
+branch_join_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext next, TO* __restrict__ rows) {
     __shared__ float scratch[32];
     qil_wait_for_producer();
     qil_release_consumer();
     const size_t row = blockIdx.x;
     TX* dst = x + row * width;
+    float r[JOIN_MOST];
+#pragma unroll
+    for (int k = 0; k < JOIN_MOST; ++k) {
+        r[k] = 1.f;
+        if (k >= in.n || in.w[k] == nullptr) continue;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < width; i += 256) { const float v = in.b[k][row * width + i]; ss = fmaf(v, v, ss); }
+        r[k] = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + in.eps);
+    }
     float sum = 0.f;
     for (int i = threadIdx.x; i < width; i += 256) {
         float add = 0.f;
-        for (int k = 0; k < in.n; ++k) add = fmaf(in.scale[k], in.b[k][row * width + i], add);
+#pragma unroll
+        for (int k = 0; k < JOIN_MOST; ++k)
+            if (k < in.n && in.w[k] == nullptr) add = fmaf(in.scale[k], in.b[k][row * width + i], add);
         if (in.y != nullptr)
             for (int t = 0; t < in.top; ++t) add += in.y[(row * in.top + t) * width + i];
-        const TX next = from_f32<TX>(to_f32<TX>(dst[i]) + add);
-        dst[i] = next;
-        sum += to_f32<TX>(next);
+#pragma unroll
+        for (int k = 0; k < JOIN_MOST; ++k)
+            if (k < in.n && in.w[k] != nullptr) add = fmaf(in.scale[k], in.b[k][row * width + i] * r[k] * in.w[k][i], add);
+        const TX now = from_f32<TX>(to_f32<TX>(dst[i]) + add);
+        dst[i] = now;
+        sum += to_f32<TX>(now);
     }
     if (rows == nullptr) return;
     TO* out = rows + row * width;
+    const W* next_w = reinterpret_cast<const W*>(next.w);
     if (next_w == nullptr) {
         for (int i = threadIdx.x; i < width; i += 256) out[i] = from_f32<TO>(to_f32<TX>(dst[i]));
         return;
     }
+    if (next.kind == JOIN_TANH) {
+        const W* next_b = reinterpret_cast<const W*>(next.b);
+        for (int i = threadIdx.x; i < width; i += 256)
+            out[i] = from_f32<TO>(fmaf(tanhf(next.alpha * to_f32<TX>(dst[i])), to_f32<W>(next_w[i]), to_f32<W>(next_b[i])));
+        return;
+    }
     float mean = 0.f;
-    if (next_center) mean = block_sum(sum, scratch) / (float)width;
+    if (next.kind == JOIN_LAYER) mean = block_sum(sum, scratch) / (float)width;
     float sq = 0.f;
     for (int i = threadIdx.x; i < width; i += 256) {
         const float v = to_f32<TX>(dst[i]) - mean;
         sq = fmaf(v, v, sq);
     }
     sq = block_sum(sq, scratch);
-    const float scale = 1.0f / sqrtf(sq / (float)width + next_eps);
+    const float scale = 1.0f / sqrtf(sq / (float)width + next.eps);
     for (int i = threadIdx.x; i < width; i += 256)
         out[i] = from_f32<TO>((to_f32<TX>(dst[i]) - mean) * scale * to_f32<W>(next_w[i]));
 }
 
-// branches: host array of n device pointers; scales: host array of n.
-extern "C" int qil_branch_join(void* x, int x_dtype, const float* const* branches, const float* scales, int n_branches,
-                               const float* y, int top, int n_rows, int width, const void* next_w, int weight_dtype,
-                               float next_eps, int next_center, void* rows, int rows_dtype, cudaStream_t stream) {
+// branches, weights (entries may be null): host arrays of n device pointers; scales: host array of n.
+extern "C" int qil_branch_join(void* x, int x_dtype, const float* const* branches, const float* const* weights, const float* scales,
+                               int n_branches, float branch_eps, const float* y, int top, int n_rows, int width,
+                               const void* next_w, const void* next_b, int weight_dtype, float next_eps, float next_alpha,
+                               int next_kind, void* rows, int rows_dtype, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     if (width <= 0 || n_branches < 0 || n_branches > JOIN_MOST || (y != nullptr && top < 1))
         QIL_REFUSE("branch_join: width %d, %d branches (at most %d), %d experts a token", width, n_branches, JOIN_MOST, top);
     if (next_w != nullptr && rows == nullptr) QIL_REFUSE("branch_join: the next norm needs rows to write");
+    if (next_kind < 0 || next_kind > JOIN_TANH || (next_w != nullptr && next_kind == JOIN_TANH && next_b == nullptr))
+        QIL_REFUSE("branch_join: next norm %d", next_kind);
     JoinBranches in = {};
-    uintptr_t bits = (uintptr_t)x | (uintptr_t)y | (uintptr_t)next_w | (uintptr_t)rows;
-    for (int k = 0; k < n_branches; ++k) { in.b[k] = branches[k]; in.scale[k] = scales[k]; bits |= (uintptr_t)branches[k]; }
-    in.n = n_branches; in.y = y; in.top = top;
-    const bool wide = width % 4 == 0 && (bits & 15) == 0;
-#define QIL_JOIN_ARGS(TX, WT, TO) \
-    dim3(n_rows), dim3(256), 0, stream, (TX*)x, in, width, (const WT*)next_w, next_eps, next_center, (TO*)rows
-#define QIL_JOIN_GO(TX, WT, TO)                                                                                       \
-    do {                                                                                                              \
-        if (wide && width <= 1024) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 1>, QIL_JOIN_ARGS(TX, WT, TO));      \
-        else if (wide && width <= 2048) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 2>, QIL_JOIN_ARGS(TX, WT, TO)); \
-        else if (wide && width <= 4096) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 4>, QIL_JOIN_ARGS(TX, WT, TO)); \
-        else qil_launch_chained(branch_join_kernel<TX, WT, TO>, QIL_JOIN_ARGS(TX, WT, TO));                           \
+    uintptr_t bits = (uintptr_t)x | (uintptr_t)y | (uintptr_t)next_w | (uintptr_t)next_b | (uintptr_t)rows;
+    int normed = 0;
+    for (int k = 0; k < n_branches; ++k) {
+        in.b[k] = branches[k]; in.scale[k] = scales[k]; in.w[k] = weights != nullptr ? weights[k] : nullptr;
+        bits |= (uintptr_t)branches[k] | (uintptr_t)in.w[k];
+        if (in.w[k] != nullptr) ++normed;
+    }
+    in.n = n_branches; in.eps = branch_eps; in.y = y; in.top = top;
+    const JoinNext next = {next_w, next_b, next_eps, next_alpha, next_kind};
+    const bool wide = width % 4 == 0 && (bits & 15) == 0 && normed <= JOIN_MOST_NORMED;
+#define QIL_JOIN_ARGS(TX, TO) dim3(n_rows), dim3(256), 0, stream, (TX*)x, in, width, next, (TO*)rows
+#define QIL_JOIN_SIZE(TX, WT, TO, N)                                                                                           \
+    do {                                                                                                                       \
+        if (width <= 1024) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 1, N>, QIL_JOIN_ARGS(TX, TO));               \
+        else if (width <= 2048) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 2, N>, QIL_JOIN_ARGS(TX, TO));          \
+        else qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 4, N>, QIL_JOIN_ARGS(TX, TO));                             \
+    } while (0)
+#define QIL_JOIN_GO(TX, WT, TO)                                                                                                \
+    do {                                                                                                                       \
+        if (!wide || width > 4096) qil_launch_chained(branch_join_kernel<TX, WT, TO>, QIL_JOIN_ARGS(TX, TO));                  \
+        else if (normed) QIL_JOIN_SIZE(TX, WT, TO, true);                                                                      \
+        else QIL_JOIN_SIZE(TX, WT, TO, false);                                                                                 \
     } while (0)
 #define QIL_JOIN_O(TX, WT)                                                                                            \
     do { if (rows_dtype == QIL_F32) QIL_JOIN_GO(TX, WT, float); else QIL_JOIN_GO(TX, WT, bf16); } while (0)
@@ -557,6 +662,44 @@ extern "C" int qil_branch_join(void* x, int x_dtype, const float* const* branche
 #undef QIL_JOIN_W
 #undef QIL_JOIN_O
 #undef QIL_JOIN_GO
+#undef QIL_JOIN_SIZE
 #undef QIL_JOIN_ARGS
+    QIL_CHECK_LAUNCH();
+}
+
+// The norm without statistics (Dynamic Tanh): y = tanh(alpha x) * w + b, float32 arithmetic, one rounding.
+template <typename TI, typename TO, typename W>
+__global__ void __launch_bounds__(256)
+tanh_norm_kernel(const TI* __restrict__ x, const W* __restrict__ weight, const W* __restrict__ bias, float alpha,
+                 const int* __restrict__ rows, TO* __restrict__ out, int width) {
+    qil_wait_for_producer();
+    qil_release_consumer();
+    const int r = blockIdx.x;
+    const TI* src = x + (size_t)(rows ? rows[r] : r) * width;
+    TO* dst = out + (size_t)r * width;
+    for (int i = threadIdx.x; i < width; i += 256)
+        dst[i] = from_f32<TO>(fmaf(tanhf(alpha * to_f32<TI>(src[i])), to_f32<W>(weight[i]), to_f32<W>(bias[i])));
+}
+
+extern "C" int qil_tanh_norm(const void* x, int x_dtype, const void* weight, const void* bias, int weight_dtype, float alpha,
+                             const int* rows, void* out, int out_dtype, int n_rows, int width, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (width <= 0) QIL_REFUSE("tanh_norm: width %d", width);
+    if (weight_dtype != QIL_F32 && weight_dtype != QIL_BF16) QIL_REFUSE("tanh_norm: weight dtype %d", weight_dtype);
+#define QIL_TANH_GO(TI, TO)                                                                                                  \
+    do {                                                                                                                     \
+        if (weight_dtype == QIL_F32)                                                                                         \
+            qil_launch_chained(tanh_norm_kernel<TI, TO, float>, dim3(n_rows), dim3(256), 0, stream, (const TI*)x,            \
+                               (const float*)weight, (const float*)bias, alpha, rows, (TO*)out, width);                      \
+        else                                                                                                                 \
+            qil_launch_chained(tanh_norm_kernel<TI, TO, bf16>, dim3(n_rows), dim3(256), 0, stream, (const TI*)x,             \
+                               (const bf16*)weight, (const bf16*)bias, alpha, rows, (TO*)out, width);                        \
+    } while (0)
+    if (x_dtype == QIL_F32 && out_dtype == QIL_F32) QIL_TANH_GO(float, float);
+    else if (x_dtype == QIL_F32 && out_dtype == QIL_BF16) QIL_TANH_GO(float, bf16);
+    else if (x_dtype == QIL_BF16 && out_dtype == QIL_BF16) QIL_TANH_GO(bf16, bf16);
+    else if (x_dtype == QIL_BF16 && out_dtype == QIL_F32) QIL_TANH_GO(bf16, float);
+    else QIL_REFUSE("tanh_norm: dtypes %d -> %d", x_dtype, out_dtype);
+#undef QIL_TANH_GO
     QIL_CHECK_LAUNCH();
 }

@@ -5,16 +5,20 @@
 // (u cos a - v sin a, v cos a + u sin a).  Two layouts of the rot_dims rotated dimensions of a vector:
 //   layout 0 (halves)       dimension i pairs with dimension i + rot_dims / 2
 //   layout 1 (interleaved)  dimension 2 i pairs with dimension 2 i + 1
-// Dimensions from rot_dims on pass unchanged.
+// Dimensions from rot_dims on pass unchanged.  A gain may multiply cosines and sines (scaled frequencies of long contexts).
 //
 // qk_rotate_store: q [Hq * d], k [Hkv * d], v [Hkv * e] are column ranges of one row-major buffer (a stacked
 // projection).  Optionally q and k are first divided by their root mean square over the WHOLE projection (all
 // heads at once) and multiplied by a weight per element (float32 arithmetic), or (per_head) every head by its own
 // root mean square over its d dimensions, with one weight of d that all heads share (per_head 2: without a weight, in
 // which case it makes no difference whether a head is normed before or after it is turned: a rotation keeps the sum
-// of squares); then every head is rotated;
+// of squares; with a gain the norm is the turned head's, the rotated dimensions' squares counting gain^2 times); then every
+// head is rotated;
 // queries go to q_out, keys and values into the request's page (a page holds its key rows
-// [kv_head][slot][d] followed by its value rows [kv_head][slot][e]).
+// [kv_head][slot][d] followed by its value rows [kv_head][slot][e]).  Values may be mixed with another layer's of the same
+// tokens on their way: (1 - share) v + share first, float32 arithmetic, one rounding.
+//
+// rotate_rows turns the heads of a column range into float32 rows, some of them times a factor (what enters a recurrence).
 //
 // latent_prepare: the tail of a latent attention's projection.  The projection holds per token the queries
 // [H][d plain, r rotated] and one row [c latent, r rotated key part].  The latent is divided by its root mean
@@ -27,11 +31,38 @@
 // the projection from qn_col on, divided by their root mean square, times qn_w, to qn_out [N][qn_width].
 #include "common.cuh"
 
-// The token's angles, once a block: table[i] = cos(pos * freq[i]), table[half + i] = sin(pos * freq[i]), i < half.
+// The token's angles, once a block: table[i] = gain cos(pos * freq[i]), table[half + i] = gain sin(pos * freq[i]), i < half.
 // The caller puts a barrier between this and the first rotated_element.
-__device__ __forceinline__ void angle_table(float* __restrict__ table, int rot_dims, int pos, const float* __restrict__ freq) {
+__device__ __forceinline__ void angle_table(float* __restrict__ table, int rot_dims, int pos, const float* __restrict__ freq,
+                                            float gain = 1.f) {
     const int half = rot_dims >> 1;
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * freq[i], &table[half + i], &table[i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float s, c;
+        sincosf((float)pos * freq[i], &s, &c);
+        table[i] = gain * c;
+        table[half + i] = gain * s;
+    }
+}
+
+// Another layer's values of the same tokens, and their share of this layer's.
+struct ValueMix {
+    const void* first;      // T [tokens, ld]; null: none
+    long long ld;
+    float share;
+};
+
+// 16 bytes of values, mixed.
+template <typename T>
+__device__ __forceinline__ uint4 mixed_values16(const uint4 mine, const T* first, float share) {
+    constexpr int V = 16 / (int)sizeof(T);
+    const uint4 other = *reinterpret_cast<const uint4*>(first);
+    const T* a = reinterpret_cast<const T*>(&mine);
+    const T* b = reinterpret_cast<const T*>(&other);
+    uint4 packed;
+    T* out = reinterpret_cast<T*>(&packed);
+#pragma unroll
+    for (int k = 0; k < V; ++k) out[k] = from_f32<T>((1.f - share) * to_f32<T>(a[k]) + share * to_f32<T>(b[k]));
+    return packed;
 }
 
 __device__ __forceinline__ float rotated_element(const float* __restrict__ vec, int j, int rot_dims, int layout,
@@ -66,7 +97,8 @@ qk_rotate_store_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col,
                        T* __restrict__ pages, const W* __restrict__ q_norm_w, const W* __restrict__ k_norm_w, float eps,
                        const float* __restrict__ freq, int rot_dims, int layout, const int* __restrict__ positions,
                        const int* __restrict__ token_row, const int* __restrict__ block_table, int table_stride,
-                       int n_q_heads, int n_kv_heads, int d, int e, int page_size, int num_pages, int wide, int per_head) {
+                       int n_q_heads, int n_kv_heads, int d, int e, int page_size, int num_pages, int wide, int per_head, float gain,
+                       ValueMix mix) {
     constexpr int V = 16 / (int)sizeof(T);
     extern __shared__ __align__(16) float vals[];   // [Hq * d + Hkv * d]: q then k, normed, float32;  then [rot_dims]: the angles
     __shared__ float scratch[32];
@@ -77,7 +109,7 @@ qk_rotate_store_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col,
     const int q_width = n_q_heads * d, k_width = n_kv_heads * d, v_width = n_kv_heads * e;
     const T* row = proj + (size_t)token * ld;
     const float* table = vals + q_width + k_width;
-    angle_table(vals + q_width + k_width, rot_dims, pos, freq);
+    angle_table(vals + q_width + k_width, rot_dims, pos, freq, gain);
     float sq = 0.f, sk = 0.f;
     if (wide) {
         auto load = [&](int column, int width, float* dst, float& sum) {
@@ -102,7 +134,10 @@ qk_rotate_store_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col,
             float* v = vals + head * d;
             const W* w = head < n_q_heads ? q_norm_w : k_norm_w;
             float ss = 0.f;
-            for (int j = lane; j < d; j += 32) ss = fmaf(v[j], v[j], ss);
+            for (int j = lane; j < d; j += 32) {
+                const float x = (per_head == 2 && j < rot_dims) ? v[j] * gain : v[j];
+                ss = fmaf(x, x, ss);
+            }
             ss = warp_sum(ss);
             const float r = 1.0f / sqrtf(ss / (float)d + eps);
             for (int j = lane; j < d; j += 32) v[j] = per_head == 2 ? v[j] * r : v[j] * r * to_f32<W>(w[j]);
@@ -143,8 +178,10 @@ qk_rotate_store_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col,
         T* values = page_base + (size_t)n_kv_heads * page_size * d;
         for (int c = tid; c < v_width / V; c += 256) {
             const int head = c * V / e, j = c * V - head * e;
-            *reinterpret_cast<uint4*>(values + ((size_t)head * page_size + slot) * e + j) =
-                *reinterpret_cast<const uint4*>(row + v_col + c * V);
+            uint4 v = *reinterpret_cast<const uint4*>(row + v_col + c * V);
+            if (mix.first != nullptr)
+                v = mixed_values16<T>(v, reinterpret_cast<const T*>(mix.first) + (size_t)token * mix.ld + c * V, mix.share);
+            *reinterpret_cast<uint4*>(values + ((size_t)head * page_size + slot) * e + j) = v;
         }
         return;
     }
@@ -156,26 +193,33 @@ qk_rotate_store_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col,
     T* v_base = page_base + (size_t)n_kv_heads * page_size * d;
     for (int i = tid; i < v_width; i += 256) {
         const int head = i / e, j = i - head * e;
-        v_base[((size_t)head * page_size + slot) * e + j] = row[v_col + i];
+        T v = row[v_col + i];
+        if (mix.first != nullptr)
+            v = from_f32<T>((1.f - mix.share) * to_f32<T>(v)
+                            + mix.share * to_f32<T>(reinterpret_cast<const T*>(mix.first)[(size_t)token * mix.ld + i]));
+        v_base[((size_t)head * page_size + slot) * e + j] = v;
     }
 }
 
-// The same for pairs of neighbours and norms per head (or none), 16 bytes a lane: a head is d / V lanes (a power of two),
-// which hold their values in registers, sum their squares by shuffles and turn their own pairs, so that nothing but the
-// token's angles goes through shared memory.  Every head of the token is asked for before the angles are made.
+// The same, 16 bytes a lane: a head is d / V lanes (a power of two), which hold their values in registers, sum their squares
+// by shuffles (the norm over the whole projection: over the block) and turn their own pairs: of neighbours within a lane, of
+// halves with the lane rot_dims / 2 dimensions away, so that nothing but the token's angles goes through shared memory.
+// Every head of the token is asked for before the angles are made.
 #define ROTATE_PIECES 4      // pieces of a token's q and k that a thread may hold
-template <typename T, typename W>
+template <typename T, typename W, int LAYOUT>
 __global__ void __launch_bounds__(256)
 qk_rotate_store_lanes_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col, int v_col, T* __restrict__ q_out,
                              T* __restrict__ pages, const W* __restrict__ q_norm_w, const W* __restrict__ k_norm_w, float eps,
                              const float* __restrict__ freq, int rot_dims, const int* __restrict__ positions,
                              const int* __restrict__ token_row, const int* __restrict__ block_table, int table_stride,
-                             int n_q_heads, int n_kv_heads, int d, int e, int page_size, int num_pages, int per_head) {
+                             int n_q_heads, int n_kv_heads, int d, int e, int page_size, int num_pages, int per_head, float gain,
+                             ValueMix mix) {
     constexpr int V = 16 / (int)sizeof(T);
     extern __shared__ __align__(16) float angles[];        // [rot_dims]: cosines, then sines
+    __shared__ float scratch[32];
     qil_wait_for_producer();
     qil_release_consumer();
-    const int token = blockIdx.x, tid = threadIdx.x;
+    const int token = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
     const int pos = positions[token];
     const T* row = proj + (size_t)token * ld;
     const int lanes = d / V;                                // of a head
@@ -190,7 +234,23 @@ qk_rotate_store_lanes_kernel(const T* __restrict__ proj, int ld, int q_col, int 
     const int index = pos / page_size;
     int page = (n_kv_heads > 0 && pos >= 0 && index < table_stride) ? block_table[(size_t)token_row[token] * table_stride + index] : -1;
     if (page >= num_pages) page = -1;                       // never write outside the pool
-    angle_table(angles, rot_dims, pos, freq);
+    angle_table(angles, rot_dims, pos, freq, gain);
+    float whole_q = 0.f, whole_k = 0.f;                     // one over the root mean square of the whole projections
+    const bool whole = !per_head && q_norm_w != nullptr;
+    if (whole) {
+#pragma unroll
+        for (int u = 0; u < ROTATE_PIECES; ++u) {
+            const int c = tid + u * 256;
+            const T* x = reinterpret_cast<const T*>(&raw[u]);
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < V; ++i) { const float f = to_f32<T>(x[i]); ss = fmaf(f, f, ss); }
+            if (c < q_pieces) whole_q += ss; else whole_k += ss;
+        }
+        whole_q = 1.0f / sqrtf(block_sum(whole_q, scratch) / (float)(n_q_heads * d) + eps);
+        whole_k = block_sum(whole_k, scratch);
+        whole_k = n_kv_heads > 0 ? 1.0f / sqrtf(whole_k / (float)(n_kv_heads * d) + eps) : 0.f;
+    }
     __syncthreads();
     const int half = rot_dims >> 1, slot = pos % page_size;
     T* page_base = pages + (size_t)(page < 0 ? 0 : page) * n_kv_heads * page_size * (d + e);
@@ -201,26 +261,48 @@ qk_rotate_store_lanes_kernel(const T* __restrict__ proj, int ld, int q_col, int 
         const T* x = reinterpret_cast<const T*>(&raw[u]);
         const bool is_q = c < q_pieces;
         const int piece = is_q ? c : c - q_pieces, head = piece / lanes, j0 = (piece - head * lanes) * V;
+        const W* w = is_q ? q_norm_w : k_norm_w;
         float v[V];
 #pragma unroll
         for (int i = 0; i < V; ++i) v[i] = to_f32<T>(x[i]);
         if (per_head) {
             float ss = 0.f;
 #pragma unroll
-            for (int i = 0; i < V; ++i) ss = fmaf(v[i], v[i], ss);
+            for (int i = 0; i < V; ++i) {
+                const float y = (per_head == 2 && j0 + i < rot_dims) ? v[i] * gain : v[i];
+                ss = fmaf(y, y, ss);
+            }
             for (int step = 1; step < lanes; step <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, step);
             const float r = 1.0f / sqrtf(ss / (float)d + eps);
-            const W* w = is_q ? q_norm_w : k_norm_w;
 #pragma unroll
             for (int i = 0; i < V; ++i) v[i] = (per_head == 2 || c >= pieces) ? v[i] * r : v[i] * r * to_f32<W>(w[j0 + i]);
-        }
+        } else if (whole && c < pieces) {
+            const float r = is_q ? whole_q : whole_k;
 #pragma unroll
-        for (int i = 0; i < V; i += 2) {
-            if (j0 + i >= rot_dims) continue;
-            const float cos_a = angles[(j0 + i) >> 1], sin_a = angles[half + ((j0 + i) >> 1)];
-            const float first = v[i], second = v[i + 1];
-            v[i] = first * cos_a - second * sin_a;
-            v[i + 1] = second * cos_a + first * sin_a;
+            for (int i = 0; i < V; ++i) v[i] = v[i] * r * to_f32<W>(w[piece * V + i]);
+        }
+        if (LAYOUT == 1) {
+#pragma unroll
+            for (int i = 0; i < V; i += 2) {
+                if (j0 + i >= rot_dims) continue;
+                const float cos_a = angles[(j0 + i) >> 1], sin_a = angles[half + ((j0 + i) >> 1)];
+                const float first = v[i], second = v[i + 1];
+                v[i] = first * cos_a - second * sin_a;
+                v[i + 1] = second * cos_a + first * sin_a;
+            }
+        } else {
+            // rot_dims / 2 is a multiple of V: a lane's dimensions all lie in the first half, in the second, or behind
+            const int away = half / V;
+            const bool low = j0 < half, turned = j0 < rot_dims;
+            const int from = turned ? (low ? lane + away : lane - away) : lane;
+            const int at = low ? j0 : j0 - half;
+#pragma unroll
+            for (int i = 0; i < V; ++i) {
+                const float other = __shfl_sync(0xffffffffu, v[i], from);
+                if (!turned) continue;
+                const float cos_a = angles[at + i], sin_a = angles[half + at + i];
+                v[i] = low ? v[i] * cos_a - other * sin_a : v[i] * cos_a + other * sin_a;
+            }
         }
         uint4 packed;
         T* o = reinterpret_cast<T*>(&packed);
@@ -234,7 +316,10 @@ qk_rotate_store_lanes_kernel(const T* __restrict__ proj, int ld, int q_col, int 
     T* values = page_base + (size_t)n_kv_heads * page_size * d;
     for (int c = tid; c < n_kv_heads * e / V; c += 256) {
         const int head = c * V / e, j = c * V - head * e;
-        *reinterpret_cast<uint4*>(values + ((size_t)head * page_size + slot) * e + j) = *reinterpret_cast<const uint4*>(row + v_col + c * V);
+        uint4 v = *reinterpret_cast<const uint4*>(row + v_col + c * V);
+        if (mix.first != nullptr)
+            v = mixed_values16<T>(v, reinterpret_cast<const T*>(mix.first) + (size_t)token * mix.ld + c * V, mix.share);
+        *reinterpret_cast<uint4*>(values + ((size_t)head * page_size + slot) * e + j) = v;
     }
 }
 
@@ -242,8 +327,8 @@ extern "C" int qil_qk_rotate_store(const void* proj, int ld, int q_col, int k_co
                                    const void* q_norm_w, const void* k_norm_w, int norm_dtype, float eps, const float* freq,
                                    int rot_dims, int layout, const int* positions, const int* token_row,
                                    const int* block_table, int table_stride, int n_tokens, int n_q_heads, int n_kv_heads,
-                                   int d, int e, int page_size, int num_pages, int act_dtype, int per_head,
-                                   cudaStream_t stream) {
+                                   int d, int e, int page_size, int num_pages, int act_dtype, int per_head, float gain,
+                                   const void* mix_first, long long mix_ld, float mix_share, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (n_q_heads <= 0 || n_kv_heads < 0 || d <= 0 || e <= 0 || page_size <= 0)
         QIL_REFUSE("qk_rotate_store: heads %d/%d sizes %d/%d page %d", n_q_heads, n_kv_heads, d, e, page_size);
@@ -251,20 +336,26 @@ extern "C" int qil_qk_rotate_store(const void* proj, int ld, int q_col, int k_co
         QIL_REFUSE("qk_rotate_store: %d rotated dimensions of %d, layout %d", rot_dims, d, layout);
     if ((q_norm_w == nullptr) != (k_norm_w == nullptr) && n_kv_heads > 0)
         QIL_REFUSE("qk_rotate_store: give both norm weights or neither");
+    if (mix_first != nullptr && mix_ld < (long long)n_kv_heads * e) QIL_REFUSE("qk_rotate_store: rows of %lld for %d values", mix_ld, n_kv_heads * e);
+    const ValueMix mix = {mix_first, mix_ld, mix_share};
     const size_t smem = ((size_t)(n_q_heads + n_kv_heads) * d + rot_dims) * sizeof(float);
     if (smem > 160 * 1024) QIL_REFUSE("qk_rotate_store: %d values of q and k per token are too many", (n_q_heads + n_kv_heads) * d);
+#define QIL_LANES_GO(LAYOUT)                                                                      \
+    qil_launch_chained(qk_rotate_store_lanes_kernel<T, W, LAYOUT>, dim3(n_tokens), dim3(256),                     \
+                       (size_t)rot_dims * sizeof(float), stream, (const T*)proj, ld, q_col, k_col, v_col,         \
+                       (T*)q_out, (T*)pages, (const W*)q_norm_w, (const W*)k_norm_w, eps, freq, rot_dims,         \
+                       positions, token_row, block_table, table_stride, n_q_heads, n_kv_heads, d, e, page_size,   \
+                       num_pages, per_head, gain, mix)
     cudaError_t err = cudaSuccess;
     QIL_DISPATCH_2(act_dtype, norm_dtype, {
         constexpr int V = 16 / (int)sizeof(T);
         const int wide = (d % V == 0 && e % V == 0 && ld % V == 0 && q_col % V == 0 && k_col % V == 0 && v_col % V == 0 &&
-                          (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)pages) & 15) == 0) ? 1 : 0;
+                          mix_ld % V == 0 &&
+                          (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)pages | (uintptr_t)mix_first) & 15) == 0) ? 1 : 0;
         const int lanes = d / V;
-        if (wide && layout == 1 && (per_head || q_norm_w == nullptr) && lanes <= 32 && (lanes & (lanes - 1)) == 0
+        if (wide && (layout == 1 || rot_dims % (2 * V) == 0) && lanes <= 32 && (lanes & (lanes - 1)) == 0
             && (n_q_heads + n_kv_heads) * lanes <= 256 * ROTATE_PIECES) {
-            qil_launch_chained(qk_rotate_store_lanes_kernel<T, W>, dim3(n_tokens), dim3(256), (size_t)rot_dims * sizeof(float), stream,
-                               (const T*)proj, ld, q_col, k_col, v_col, (T*)q_out, (T*)pages, (const W*)q_norm_w,
-                               (const W*)k_norm_w, eps, freq, rot_dims, positions, token_row, block_table, table_stride,
-                               n_q_heads, n_kv_heads, d, e, page_size, num_pages, per_head);
+            if (layout == 1) QIL_LANES_GO(1); else QIL_LANES_GO(0);
             QIL_CHECK_LAUNCH();
         }
         if (smem > 48 * 1024)
@@ -273,9 +364,52 @@ extern "C" int qil_qk_rotate_store(const void* proj, int ld, int q_col, int k_co
             qil_launch_chained(qk_rotate_store_kernel<T, W>, dim3(n_tokens), dim3(256), smem, stream,
                                (const T*)proj, ld, q_col, k_col, v_col, (T*)q_out, (T*)pages, (const W*)q_norm_w,
                                (const W*)k_norm_w, eps, freq, rot_dims, layout, positions, token_row, block_table,
-                               table_stride, n_q_heads, n_kv_heads, d, e, page_size, num_pages, wide, per_head);
+                               table_stride, n_q_heads, n_kv_heads, d, e, page_size, num_pages, wide, per_head, gain, mix);
     });
+#undef QIL_LANES_GO
     if (err != cudaSuccess) { snprintf(qil_error_text, sizeof(qil_error_text), "%s", cudaGetErrorString(err)); return (int)err; }
+    QIL_CHECK_LAUNCH();
+}
+
+// Heads of d dimensions, side by side from column `col` of the projection on, turned into float32 rows out [tokens, heads * d];
+// heads from `scaled_from` on are multiplied by `scale`.  A thread takes a pair.
+template <typename T>
+__global__ void __launch_bounds__(256)
+rotate_rows_kernel(const T* __restrict__ proj, long long ld, int col, int n_heads, int d, const float* __restrict__ freq,
+                   int rot_dims, int layout, float gain, const int* __restrict__ positions, int scaled_from, float scale,
+                   float* __restrict__ out) {
+    extern __shared__ __align__(16) float angles[];        // [rot_dims]: cosines, then sines
+    qil_wait_for_producer();
+    qil_release_consumer();
+    const int token = blockIdx.x, half = rot_dims >> 1, rest = d - rot_dims;
+    angle_table(angles, rot_dims, positions[token], freq, gain);
+    __syncthreads();
+    const T* row = proj + (size_t)token * ld + col;
+    float* dst = out + (size_t)token * n_heads * d;
+    for (int i = threadIdx.x; i < n_heads * half; i += 256) {
+        const int head = i / half, p = i - head * half;
+        const int first = head * d + (layout == 0 ? p : 2 * p), second = layout == 0 ? first + half : first + 1;
+        const float by = head >= scaled_from ? scale : 1.f;
+        const float u = to_f32<T>(row[first]), v = to_f32<T>(row[second]), c = angles[p], s = angles[half + p];
+        dst[first] = (u * c - v * s) * by;
+        dst[second] = (v * c + u * s) * by;
+    }
+    for (int i = threadIdx.x; i < n_heads * rest; i += 256) {
+        const int head = i / rest, at = head * d + rot_dims + i - head * rest;
+        dst[at] = to_f32<T>(row[at]) * (head >= scaled_from ? scale : 1.f);
+    }
+}
+
+extern "C" int qil_rotate_rows(const void* proj, long long ld, int col, int n_heads, int d, const float* freq, int rot_dims,
+                               int layout, float gain, const int* positions, int scaled_from, float scale, int n_tokens,
+                               float* out, int act_dtype, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (n_heads <= 0 || d <= 0 || col < 0 || ld < col + (long long)n_heads * d) QIL_REFUSE("rotate_rows: %d heads of %d from column %d", n_heads, d, col);
+    if (rot_dims < 0 || rot_dims > d || (rot_dims & 1) || (rot_dims > 0 && freq == nullptr) || (layout != 0 && layout != 1))
+        QIL_REFUSE("rotate_rows: %d rotated dimensions of %d, layout %d", rot_dims, d, layout);
+    QIL_DISPATCH_1(act_dtype,
+        qil_launch_chained(rotate_rows_kernel<T>, dim3(n_tokens), dim3(256), (size_t)rot_dims * sizeof(float), stream, (const T*)proj,
+                           ld, col, n_heads, d, freq, rot_dims, layout, gain, positions, scaled_from, scale, out));
     QIL_CHECK_LAUNCH();
 }
 
@@ -444,14 +578,30 @@ extern "C" int qil_head_product(const void* x, long long x_row, int x_head, cons
 }
 
 // y[n, h * width + j] *= sigmoid(gate[n, h]): a gate per token and head on rows laid out head by head (float32 math,
-// one rounding).  For steps whose per-head products ran as one batched library product.
+// one rounding).  For steps whose per-head products ran as one batched library product, and for attention whose output is
+// gated; width 1: a gate per element, 16 bytes a load where the rows allow it.
 template <typename T>
 __global__ void __launch_bounds__(256)
-head_gate_kernel(T* __restrict__ y, long long y_row, int width, const T* __restrict__ gate, long long gate_row, int n_heads) {
+head_gate_kernel(T* __restrict__ y, long long y_row, int width, const T* __restrict__ gate, long long gate_row, int n_heads,
+                 int wide) {
+    constexpr int V = 16 / (int)sizeof(T);
     qil_wait_for_producer();
     qil_release_consumer();
     const size_t token = blockIdx.x;
     const int per_row = n_heads * width;
+    if (wide) {
+        for (int i = threadIdx.x; i < per_row / V; i += 256) {
+            uint4* at = reinterpret_cast<uint4*>(y + token * y_row + i * V);
+            uint4 mine = *at;
+            const uint4 g4 = *reinterpret_cast<const uint4*>(gate + token * gate_row + i * V);
+            T* x = reinterpret_cast<T*>(&mine);
+            const T* g = reinterpret_cast<const T*>(&g4);
+#pragma unroll
+            for (int k = 0; k < V; ++k) x[k] = from_f32<T>(to_f32<T>(x[k]) / (1.f + expf(-to_f32<T>(g[k]))));
+            *at = mine;
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < per_row; i += 256) {
         const float g = to_f32<T>(gate[token * gate_row + i / width]);
         T* at = y + token * y_row + i;
@@ -464,8 +614,11 @@ extern "C" int qil_head_gate(void* y, long long y_row, int width, const void* ga
     if (n_tokens <= 0) return 0;
     if (n_heads <= 0 || width <= 0) QIL_REFUSE("head_gate: %d heads of %d", n_heads, width);
     QIL_DISPATCH_1(act_dtype, {
+        constexpr int V = 16 / (int)sizeof(T);
+        const int wide = (width == 1 && n_heads % V == 0 && y_row % V == 0 && gate_row % V == 0 &&
+                          (((uintptr_t)y | (uintptr_t)gate) & 15) == 0) ? 1 : 0;
         qil_launch_chained(head_gate_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, (T*)y, y_row, width, (const T*)gate,
-                           gate_row, n_heads);
+                           gate_row, n_heads, wide);
     });
     QIL_CHECK_LAUNCH();
 }

@@ -184,7 +184,7 @@ short_conv_store_vec8_kernel(const bf16* __restrict__ u, const bf16* __restrict_
 // The state after a segment of more than one token: the last taps - 1 rows of u that the request has seen.
 template <typename T>
 __global__ void __launch_bounds__(256)
-short_conv_state_kernel(const T* __restrict__ u, float* __restrict__ state, const int* __restrict__ seg_row,
+short_conv_state_kernel(const T* __restrict__ u, long long ld, float* __restrict__ state, const int* __restrict__ seg_row,
                         const int* __restrict__ seg_start, const int* __restrict__ seg_len, int taps, int channels) {
     qil_wait_for_producer();
     qil_release_consumer();
@@ -201,7 +201,7 @@ short_conv_state_kernel(const T* __restrict__ u, float* __restrict__ state, cons
         const int at = len - (taps - 1) + i;          // index into the segment; negative: before it
         rows[i] = 0.f;
         if (i < taps - 1)
-            rows[i] = at >= 0 ? to_f32<T>(u[(size_t)(first + at) * channels + c]) : slot[(size_t)(len + i) * channels + c];
+            rows[i] = at >= 0 ? to_f32<T>(u[(size_t)(first + at) * ld + c]) : slot[(size_t)(len + i) * channels + c];
     }
 #pragma unroll
     for (int i = 0; i < CONV_MAX_TAPS - 1; ++i)
@@ -233,14 +233,15 @@ extern "C" int qil_short_conv_store(const void* u, const void* taps_w, float* st
     QIL_CHECK_LAUNCH();
 }
 
-extern "C" int qil_short_conv_state(const void* u, float* state, const int* seg_row, const int* seg_start,
+// ld: row stride of u (its `channels` columns may be the head of a wider row).
+extern "C" int qil_short_conv_state(const void* u, long long ld, float* state, const int* seg_row, const int* seg_start,
                                     const int* seg_len, int n_segments, int taps, int channels, int act_dtype,
                                     cudaStream_t stream) {
     if (n_segments <= 0 || taps <= 1) return 0;
-    if (taps > CONV_MAX_TAPS || channels <= 0) QIL_REFUSE("short_conv_state: %d taps, %d channels", taps, channels);
+    if (taps > CONV_MAX_TAPS || channels <= 0 || ld < channels) QIL_REFUSE("short_conv_state: %d taps, %d channels", taps, channels);
     dim3 grid(n_segments, (channels + 255) / 256);
     QIL_DISPATCH_1(act_dtype,
-        qil_launch_chained(short_conv_state_kernel<T>, grid, dim3(256), 0, stream, (const T*)u, state, seg_row,
+        qil_launch_chained(short_conv_state_kernel<T>, grid, dim3(256), 0, stream, (const T*)u, ld, state, seg_row,
                            seg_start, seg_len, taps, channels));
     QIL_CHECK_LAUNCH();
 }

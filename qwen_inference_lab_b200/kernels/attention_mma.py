@@ -74,33 +74,44 @@ def step_plan(ctx):
     return view.array, view.count
 
 
-def supports(head_dim, n_q_heads, n_kv_heads) -> bool:
-    return head_dim % 16 == 0 and 16 <= head_dim <= 256 and n_q_heads % n_kv_heads == 0
+def supports(head_dim, n_q_heads, n_kv_heads, v_dim=None) -> bool:
+    fits = lambda size: size % 16 == 0 and 16 <= size <= 256
+    return fits(head_dim) and fits(head_dim if v_dim is None else v_dim) and n_q_heads % n_kv_heads == 0
 
 
-def library(head_dim):
-    lib = _libs.get(head_dim)
+def library_name(head_dim, v_dim=None):
+    """(name, defines) of the library for heads of ``head_dim`` whose values have ``v_dim`` columns (None: as many)."""
+    if v_dim is None or v_dim == head_dim:
+        return f"qil_attn_d{head_dim}", {"QIL_HEAD_DIM": head_dim}
+    return f"qil_attn_d{head_dim}_v{v_dim}", {"QIL_HEAD_DIM": head_dim, "QIL_V_DIM": v_dim}
+
+
+def library(head_dim, v_dim=None):
+    v_dim = head_dim if v_dim is None else v_dim
+    lib = _libs.get((head_dim, v_dim))
     if lib is None:
-        if not supports(head_dim, 1, 1):
-            raise KernelError(f"the tensor-core attention takes head sizes 16, 32, ..., 256, not {head_dim}")
-        lib = build.load(f"qil_attn_d{head_dim}", ["attention_mma.cu"], {"QIL_HEAD_DIM": head_dim})
-        if lib.qil_attn_head_dim() != head_dim or lib.qil_attn_max_decode_span() != MAX_DECODE_SPAN:
+        if not supports(head_dim, 1, 1, v_dim):
+            raise KernelError(f"the tensor-core attention takes head sizes 16, 32, ..., 256, not {head_dim} (values of {v_dim})")
+        name, defines = library_name(head_dim, v_dim)
+        lib = build.load(name, ["attention_mma.cu"], defines)
+        if lib.qil_attn_head_dim() != head_dim or lib.qil_attn_v_dim() != v_dim or lib.qil_attn_max_decode_span() != MAX_DECODE_SPAN:
             raise KernelError("attention library was built for other constants")
-        _libs[head_dim] = lib
+        _libs[(head_dim, v_dim)] = lib
     return lib
 
 
 _sm_count = None
 
 
-def _slots(head_dim, planes=2) -> int:
+def _slots(head_dim, planes=2, v_dim=None) -> int:
     """Blocks of the span kernel that run at a time: SMs x blocks per SM (shared memory decides; ``planes`` = 1:
     pages of one row per position, half the tiles)."""
     global _sm_count
     if _sm_count is None:
         _sm_count = torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count \
             if torch.cuda.is_available() else 148
-    block_smem = (16 + 2 * planes * KV_TILE) * (head_dim + 8) * 2 + 2048
+    values = (planes - 1) * 2 * KV_TILE * ((head_dim if v_dim is None else v_dim) + 8)
+    block_smem = ((16 + 2 * KV_TILE) * (head_dim + 8) + values) * 2 + 2048
     return _sm_count * max(1, min(3, (227 * 1024) // block_smem))
 
 
@@ -227,13 +238,14 @@ class ScoreOptions:
 
 
 def prefill(q, pages, out, tile_info, n_tiles, block_table, n_q_heads, n_kv_heads, head_dim, page_size, window,
-            scale, slopes_log2=None, options=None, shared_rows=False, value_cols=0):
+            scale, slopes_log2=None, options=None, shared_rows=False, value_cols=0, v_dim=None):
     """tile_info int32 [n_tiles * 4]: (first token, its position, rows <= 64, block-table row) per tile.
     ``slopes_log2`` float32 [Hq]: slope_h * log2(e) of a bias slope_h * (query position - key position) that is
     taken off the scaled score.  ``options``: a :class:`ScoreOptions` (no window then).  ``shared_rows``: a page
     holds one row per position, the key, whose leading ``value_cols`` columns (0: all) are the value (no slopes
-    then; options go with it); the output's columns past those are zero."""
-    lib = library(head_dim)
+    then; options go with it); the output's columns past those are zero.  ``v_dim``: the size of a value head where it
+    is not ``head_dim``."""
+    lib = library(head_dim, v_dim)
     _check_slopes(slopes_log2, n_q_heads)
     if shared_rows and options:
         options.check(n_q_heads)
@@ -269,13 +281,13 @@ def prefill(q, pages, out, tile_info, n_tiles, block_table, n_q_heads, n_kv_head
 
 def decode(q, pages, out, decode_info, n_decode, part_o, part_ml, n_spans, span_len, block_table,
            n_q_heads, n_kv_heads, head_dim, page_size, window, scale, tickets=None, slopes_log2=None, options=None,
-           shared_rows=False, value_cols=0):
+           shared_rows=False, value_cols=0, v_dim=None):
     """decode_info int32 [n_decode * 4]: (token, its position, block-table row, the step's longest context)
     per single token.  A negative ``span_len``: the kernels cut the step's longest context into ``n_spans``
     equal spans of at most ``-span_len`` positions (see ``plan_spans``).  ``tickets``: int32 zeros, one per
     (token, query head) or more (``decode_scratch``): the last block of a token's spans merges them; None: a
-    second kernel does.  ``shared_rows``: see ``prefill``."""
-    lib = library(head_dim)
+    second kernel does.  ``shared_rows``, ``v_dim``: see ``prefill``."""
+    lib = library(head_dim, v_dim)
     _check_slopes(slopes_log2, n_q_heads)
     if shared_rows and options:
         options.check(n_q_heads)
@@ -357,19 +369,24 @@ def attend_projection(ctx, qkv, cache, out, n_q_heads, n_kv_heads, own_kv_heads,
 
 
 def attend(ctx, q, cache, out, n_q_heads, n_kv_heads, head_dim, window, scale, slopes_log2=None, options=None,
-           shared_rows=False, value_cols=0):
-    """q, out bfloat16 [N, Hq*D]; cache a KVCacheView whose pages already hold this step's keys and values.
-    ``slopes_log2``, ``options``, ``shared_rows``, ``value_cols``: see ``prefill``."""
+           shared_rows=False, value_cols=0, v_dim=None):
+    """q bfloat16 [N, Hq*D], out [N, Hq*v_dim]; cache a KVCacheView whose pages already hold this step's keys and values.
+    ``slopes_log2``, ``options``, ``shared_rows``, ``value_cols``, ``v_dim``: see ``prefill``."""
     if q.dtype != torch.bfloat16 or cache.pages.dtype != torch.bfloat16:
         raise KernelError("the tensor-core attention takes bfloat16 queries and pages")
     planes = 1 if shared_rows else 2
-    if tuple(cache.pages.shape[1:]) != (planes, n_kv_heads, cache.page_size, head_dim):
+    v_dim = head_dim if v_dim is None else int(v_dim)
+    layout = (planes, n_kv_heads, cache.page_size, head_dim) if v_dim == head_dim \
+        else (n_kv_heads * cache.page_size * (head_dim + v_dim),)
+    if tuple(cache.pages.shape[1:]) != layout or (shared_rows and v_dim != head_dim):
         raise KernelError(f"attention: cache layout {tuple(cache.pages.shape)}")
+    if q.shape[1] != n_q_heads * head_dim or out.shape != (q.shape[0], n_q_heads * v_dim):
+        raise KernelError(f"attention: queries {tuple(q.shape)}, output {tuple(out.shape)}")
     arrays, counts = step_plan(ctx)
     n_tiles, n_big, n_rest, n_decode = (counts[name] // 4 for name in
                                         ("tile_info", "big_tile_info", "rest_tile_info", "decode_info"))
     if n_big and (not options or attention_tc.takes(options)) and not shared_rows \
-            and attention_tc.supports(head_dim, cache.page_size, window):
+            and v_dim == head_dim and attention_tc.supports(head_dim, cache.page_size, window):
         # whole 128-token tiles on tcgen05 with the accumulators in tensor memory, the leftovers below
         if options:
             options.check(n_q_heads)
@@ -379,17 +396,17 @@ def attend(ctx, q, cache, out, n_q_heads, n_kv_heads, head_dim, window, scale, s
                              softcap=options.softcap if options else 0.0, window=window)
         if n_rest:
             prefill(q, cache.pages, out, arrays["rest_tile_info"], n_rest, cache.block_table, n_q_heads,
-                    n_kv_heads, head_dim, cache.page_size, window, scale, slopes_log2, options)
+                    n_kv_heads, head_dim, cache.page_size, window, scale, slopes_log2, options, v_dim=v_dim)
     elif n_tiles:
         prefill(q, cache.pages, out, arrays["tile_info"], n_tiles, cache.block_table, n_q_heads, n_kv_heads,
-                head_dim, cache.page_size, window, scale, slopes_log2, options, shared_rows, value_cols)
+                head_dim, cache.page_size, window, scale, slopes_log2, options, shared_rows, value_cols, v_dim)
     if n_decode:
         n_spans, longest_span = plan_spans(n_decode, n_q_heads, n_kv_heads, ctx.max_context, head_dim,
                                            getattr(ctx, "min_context", 0) or None,
-                                           slots=_slots(head_dim, planes) if shared_rows else None)
-        part_o, part_ml, tickets = decode_scratch(ctx, n_decode, n_q_heads, n_spans, head_dim)
+                                           slots=_slots(head_dim, planes, v_dim) if shared_rows or v_dim != head_dim else None)
+        part_o, part_ml, tickets = decode_scratch(ctx, n_decode, n_q_heads, n_spans, v_dim)
         if not merge_in_kernel(n_decode, n_q_heads, n_kv_heads, head_dim):
             tickets = None
         decode(q, cache.pages, out, arrays["decode_info"], n_decode, part_o, part_ml, n_spans, -longest_span,
                cache.block_table, n_q_heads, n_kv_heads, head_dim, cache.page_size, window, scale, tickets, slopes_log2,
-               options, shared_rows, value_cols)
+               options, shared_rows, value_cols, v_dim)

@@ -18,7 +18,7 @@ _CODES = {torch.float32: F32, torch.bfloat16: BF16}
 
 CORE_SOURCES = ["elementwise.cu", "rope_kv.cu", "gemm_f32.cu", "gemm_small_m.cu", "attention_generic.cu",
                 "sampling.cu", "norm_exact.cu", "gated_activation.cu", "qkv_store.cu", "gla_scan.cu", "moe.cu",
-                "short_conv.cu", "rotary_freq.cu"]
+                "short_conv.cu", "rotary_freq.cu", "matrix_state.cu"]
 SMALL_M_MAX_ROWS = min(16, tuning.SMALL_M_MAX_ROWS)      # the kernel takes 16 at most
 
 _core = None
@@ -578,12 +578,22 @@ def short_conv_store(u, taps_weight, state, q_out, kv_cache, positions, token_ro
         c_int(num_pages), c_int(dtype_code(u.dtype)), c_int(dtype_code(taps_weight.dtype)), _stream()),
         "short_conv_store")
     if taps > 1 and n_segments < n:      # some request brought more than one token: its state moves on here
-        for t in (seg_row, seg_start, seg_len):
-            _need(t, "segments", torch.int32, 1)
-        _check(lib, lib.qil_short_conv_state(_p(u), _p(state), _p(seg_row), _p(seg_start), _p(seg_len), c_int(n_segments),
-                                             c_int(taps), c_int(channels), c_int(dtype_code(u.dtype)), _stream()),
-               "short_conv_state")
+        short_conv_state(u, channels, state, seg_row, seg_start, seg_len, n_segments)
     return q_out
+
+
+def short_conv_state(u, channels, state, seg_row, seg_start, seg_len, n_segments):
+    """Move the convolution slots of the requests that brought more than one token on to their last rows of ``u`` [N, width]
+    (its first ``channels`` columns).  ``state`` float32 [slots, taps - 1, channels]."""
+    _need(u, "u", ndim=2); _need(state, "state", torch.float32, 3)
+    for t in (seg_row, seg_start, seg_len):
+        _need(t, "segments", torch.int32, 1)
+    if state.shape[2] != channels or channels > u.shape[1]:
+        raise KernelError(f"short_conv_state: {channels} channels of rows of {u.shape[1]}, state {tuple(state.shape)}")
+    lib = core()
+    _check(lib, lib.qil_short_conv_state(_p(u), c_longlong(u.shape[1]), _p(state), _p(seg_row), _p(seg_start), _p(seg_len),
+                                         c_int(n_segments), c_int(state.shape[1] + 1), c_int(channels),
+                                         c_int(dtype_code(u.dtype)), _stream()), "short_conv_state")
 
 
 def gated_activation(gate_up, kind, *, limit=0.0, alpha=1.0, pairs8=False, out=None, column=0, width=None):
@@ -780,7 +790,7 @@ def gla_carry(chunk_state, decay_product, slots, carry, n_carries):
 
 
 def gla_norm_gate(scratch, projected, gate_column, norm_weight, eps, n_heads, e, out):
-    """out = rmsnorm over each head's e values of ``scratch`` (weight ``norm_weight``) * silu(gate), the gate
+    """out = rmsnorm over each head's e values of ``scratch`` (weight ``norm_weight``, or None) * silu(gate), the gate
     being the columns of ``projected`` from ``gate_column`` on (None: no gate)."""
     _need(scratch, "scratch", torch.float32); _need(projected, "projected", ndim=2); _need(out, "out", projected.dtype, 2)
     n = projected.shape[0]
@@ -791,7 +801,8 @@ def gla_norm_gate(scratch, projected, gate_column, norm_weight, eps, n_heads, e,
     _check(lib, lib.qil_gla_norm_gate(_p(scratch), c_void_p(gate),
                                       c_int(projected.shape[1]), _p(norm_weight), c_float(eps), c_int(n), c_int(n_heads),
                                       c_int(e), _p(out), c_int(dtype_code(projected.dtype)),
-                                      c_int(dtype_code(norm_weight.dtype)), _stream()), "gla_norm_gate")
+                                      c_int(dtype_code(norm_weight.dtype) if norm_weight is not None else F32), _stream()),
+           "gla_norm_gate")
     return out
 
 
@@ -888,7 +899,10 @@ def softcap_inplace(x, cap):
     return x
 
 
-NORM_KINDS = {"rms": 0, "layer": 1}     # root mean square; mean taken off first (a layer norm without a bias)
+# root mean square; mean taken off first (a layer norm without a bias); tanh(alpha x) * w + b, which has no statistics and
+# which only branch_join knows
+NORM_KINDS = {"rms": 0, "layer": 1, "tanh": 2}
+JOINED_NORM_KINDS = ("rms", "layer")
 
 
 def norm_join(x, branch, weight, eps, kind="rms", *, next_weight=None, next_eps=None, next_kind=None, rows=None):
@@ -900,8 +914,8 @@ def norm_join(x, branch, weight, eps, kind="rms", *, next_weight=None, next_eps=
     _need(x, "x", ndim=2); _need(branch, "branch", torch.float32, 2); _need(weight, "weight", ndim=1)
     if branch.shape != x.shape or weight.shape[0] != x.shape[1]:
         raise KernelError("norm_join: shapes differ")
-    if kind not in NORM_KINDS or (next_kind or kind) not in NORM_KINDS:
-        raise KernelError(f"norm_join: a norm is one of {sorted(NORM_KINDS)}")
+    if kind not in JOINED_NORM_KINDS or (next_kind or kind) not in JOINED_NORM_KINDS:
+        raise KernelError(f"norm_join: a norm is one of {sorted(JOINED_NORM_KINDS)}")
     if rows is not None:
         _need(rows, "rows", ndim=2)
         if rows.shape != x.shape:
@@ -922,18 +936,26 @@ def norm_join(x, branch, weight, eps, kind="rms", *, next_weight=None, next_eps=
 JOIN_MOST_BRANCHES = 4
 
 
-def branch_join(x, branches, *, routed=None, next_weight=None, next_eps=0.0, next_kind="rms", rows=None):
-    """x += sum of scale * branch over ``branches`` (pairs of a float32 [N, width] and a number, at most four) + the sum
-    of each row's routed experts (``routed`` float32 [N, top, width]), row by row in float32; x [N, width] is the stream
-    (float32 or bfloat16), updated in place.  ``rows`` and ``next_weight``: as in :func:`norm_join`."""
+def branch_join(x, branches, *, routed=None, next_weight=None, next_eps=0.0, next_kind="rms", next_bias=None, next_alpha=0.0,
+                rows=None, branch_eps=0.0):
+    """x += sum of scale * branch over ``branches`` (a float32 [N, width] and a number each, at most four) + the sum of each
+    row's routed experts (``routed`` float32 [N, top, width]), row by row in float32; x [N, width] is the stream (float32 or
+    bfloat16), updated in place.  A branch with a third entry, a weight float32 [width], is divided by its root mean square
+    (with ``branch_eps``) and multiplied by it on the way.  ``rows`` and ``next_weight``: as in :func:`norm_join`;
+    ``next_kind`` ``"tanh"`` takes ``next_bias`` [width] and ``next_alpha``."""
     _need(x, "x", ndim=2)
     n, width = x.shape
     if len(branches) > JOIN_MOST_BRANCHES:
         raise KernelError(f"branch_join: {len(branches)} branches are more than {JOIN_MOST_BRANCHES}")
-    for branch, _ in branches:
+    weights = [branch[2] if len(branch) > 2 else None for branch in branches]
+    for branch, weight in zip((b[0] for b in branches), weights):
         _need(branch, "branch", torch.float32, 2)
         if branch.shape != x.shape:
             raise KernelError("branch_join: shapes differ")
+        if weight is not None:
+            _need(weight, "a branch's weight", torch.float32, 1)
+            if weight.shape[0] != width:
+                raise KernelError("branch_join: a branch's weight has one value per column")
     top = 0
     if routed is not None:
         _need(routed, "routed", torch.float32, 3)
@@ -950,15 +972,42 @@ def branch_join(x, branches, *, routed=None, next_weight=None, next_eps=0.0, nex
         _need(next_weight, "next_weight", ndim=1)
         if rows is None or next_weight.shape[0] != width:
             raise KernelError("branch_join: the next norm needs rows to write and a weight of the stream's width")
-    pointers = (c_void_p * JOIN_MOST_BRANCHES)(*(branch.data_ptr() for branch, _ in branches))
-    scales = (c_float * JOIN_MOST_BRANCHES)(*(float(scale) for _, scale in branches))
+        if next_kind == "tanh":
+            _need(next_bias, "next_bias", next_weight.dtype, 1)
+            if next_bias.shape[0] != width:
+                raise KernelError("branch_join: the next norm's bias has another size")
+    pointers = (c_void_p * JOIN_MOST_BRANCHES)(*(branch[0].data_ptr() for branch in branches))
+    weight_pointers = (c_void_p * JOIN_MOST_BRANCHES)(*(w.data_ptr() if w is not None else 0 for w in weights))
+    scales = (c_float * JOIN_MOST_BRANCHES)(*(float(branch[1]) for branch in branches))
     lib = core()
-    _check(lib, lib.qil_branch_join(_p(x), c_int(dtype_code(x.dtype)), pointers, scales, c_int(len(branches)), _p(routed),
-                                    c_int(top), c_int(n), c_int(width), _p(next_weight),
-                                    c_int(dtype_code(next_weight.dtype) if next_weight is not None else F32),
-                                    c_float(next_eps), c_int(NORM_KINDS[next_kind]), _p(rows),
+    _check(lib, lib.qil_branch_join(_p(x), c_int(dtype_code(x.dtype)), pointers, weight_pointers, scales, c_int(len(branches)),
+                                    c_float(branch_eps), _p(routed), c_int(top), c_int(n), c_int(width), _p(next_weight),
+                                    _p(next_bias), c_int(dtype_code(next_weight.dtype) if next_weight is not None else F32),
+                                    c_float(next_eps), c_float(next_alpha), c_int(NORM_KINDS[next_kind]), _p(rows),
                                     c_int(dtype_code(rows.dtype) if rows is not None else F32), _stream()), "branch_join")
     return x
+
+
+def tanh_norm(x, weight, bias, alpha, out_dtype=None, rows=None, out=None):
+    """y = tanh(alpha x) * weight + bias with float32 arithmetic and one rounding.  ``x`` float32 or bfloat16 [N, width]; the
+    result has ``out_dtype`` (default: x's); with ``rows`` (int32) only those rows, in that order."""
+    _need(x, "x", ndim=2); _need(weight, "weight", ndim=1); _need(bias, "bias", weight.dtype, 1)
+    width = x.shape[1]
+    if weight.shape[0] != width or bias.shape[0] != width:
+        raise KernelError(f"tanh_norm: weight of {weight.shape[0]} (or the bias) for width {width}")
+    if rows is not None:
+        _need(rows, "rows", torch.int32, 1)
+    n_rows = x.shape[0] if rows is None else rows.shape[0]
+    if out is None:
+        out = torch.empty((n_rows, width), dtype=out_dtype or x.dtype, device=x.device)
+    _need(out, "out", ndim=2)
+    if out.shape != (n_rows, width):
+        raise KernelError("tanh_norm: out has the wrong shape")
+    lib = core()
+    _check(lib, lib.qil_tanh_norm(_p(x), c_int(dtype_code(x.dtype)), _p(weight), _p(bias), c_int(dtype_code(weight.dtype)),
+                                  c_float(alpha), _p(rows), _p(out), c_int(dtype_code(out.dtype)), c_int(n_rows), c_int(width),
+                                  _stream()), "tanh_norm")
+    return out
 
 
 def scale_inplace(x, factor):
@@ -983,15 +1032,18 @@ def _check_rotation(freq, rot_dims, layout, most, what):
 
 def qk_rotate_store(proj, columns, q_out, kv_cache, q_norm_w, k_norm_w, eps, freq, rot_dims, layout, positions,
                     token_row, block_table, n_q_heads, n_kv_heads, head_dim, v_dim, page_size, per_head=False,
-                    unit_heads=False):
+                    unit_heads=False, gain=1.0, mix=None):
     """The tail of a q/k/v projection with rotation from frequencies (float32 angles position * freq[i]).
 
     ``proj`` [N, width] holds q, k, v from the columns ``columns`` = (q, k, v) on.  With ``q_norm_w`` [Hq * d] and
     ``k_norm_w`` [Hkv * d], q and k are first divided by their root mean square over the whole projection (all heads
     at once) and multiplied by the weight; with ``per_head`` every head is normed by itself over its d dimensions and
     the weights are [d], one for all query heads and one for all key heads.  ``unit_heads`` (no weights): every head is
-    divided by its own root mean square and that is all, which a rotation before or after does not change.  The values are copied as projected from
-    column v on: giving the keys' column there stores the keys as projected, before norm and rotation, as values.
+    divided by its own root mean square and that is all, which a rotation before or after does not change.  ``gain``
+    multiplies cosines and sines; heads of unit size are then those of the turned heads.  The values are copied as projected from
+    column v on: giving the keys' column there stores the keys as projected, before norm and rotation, as values.  ``mix`` =
+    (rows, column, share): the values become (1 - share) v + share first, ``first`` being n_kv_heads * v_dim columns of
+    ``rows`` [N, width] from ``column`` on.
     Then the first ``rot_dims`` dimensions of every head are rotated
     (``layout``: ``ROTARY_HALVES`` or ``ROTARY_INTERLEAVED``); queries go to ``q_out`` [N, Hq * d], keys and values
     into the pages."""
@@ -1003,6 +1055,13 @@ def qk_rotate_store(proj, columns, q_out, kv_cache, q_norm_w, k_norm_w, eps, fre
         raise KernelError("qk_rotate_store: shapes do not match the head counts")
     _check_rotation(freq, rot_dims, layout, head_dim, "qk_rotate_store")
     norm_code = F32
+    mix_ptr, mix_ld, share = c_void_p(0), 0, 0.0
+    if mix is not None:
+        first, column, share = mix
+        _need(first, "the values to mix in", proj.dtype, 2)
+        if first.shape[0] != n or column < 0 or column + n_kv_heads * v_dim > first.shape[1]:
+            raise KernelError("qk_rotate_store: the values to mix in do not fit")
+        mix_ptr, mix_ld = c_void_p(first.data_ptr() + column * first.element_size()), first.shape[1]
     if unit_heads and (q_norm_w is not None or k_norm_w is not None):
         raise KernelError("qk_rotate_store: heads of unit size have no norm weights")
     if q_norm_w is not None:
@@ -1027,9 +1086,158 @@ def qk_rotate_store(proj, columns, q_out, kv_cache, q_norm_w, k_norm_w, eps, fre
         _p(q_norm_w), _p(k_norm_w), c_int(norm_code), c_float(eps), _p(freq), c_int(rot_dims), c_int(layout),
         _p(positions), _p(token_row), _p(block_table if n_kv_heads else None),
         c_int(block_table.shape[1] if n_kv_heads else 0), c_int(n), c_int(n_q_heads), c_int(n_kv_heads), c_int(head_dim),
-        c_int(v_dim), c_int(page_size), c_int(num_pages), c_int(dtype_code(proj.dtype)), 
-        c_int(2 if unit_heads else 1 if per_head else 0), _stream()), "qk_rotate_store")
+        c_int(v_dim), c_int(page_size), c_int(num_pages), c_int(dtype_code(proj.dtype)),
+        c_int(2 if unit_heads else 1 if per_head else 0), c_float(gain), mix_ptr, c_longlong(mix_ld), c_float(share), _stream()),
+        "qk_rotate_store")
     return q_out
+
+
+def rotate_rows(proj, column, n_heads, head_dim, freq, rot_dims, layout, positions, *, gain=1.0, scaled_from=None, scale=1.0):
+    """float32 [N, n_heads * head_dim]: that many heads of ``proj`` from ``column`` on, the first ``rot_dims`` dimensions of each
+    turned as in :func:`qk_rotate_store`; heads from number ``scaled_from`` on times ``scale``."""
+    _need(proj, "proj", ndim=2); _need(positions, "positions", torch.int32, 1)
+    n, ld = proj.shape
+    if column < 0 or column + n_heads * head_dim > ld or positions.shape[0] != n:
+        raise KernelError("rotate_rows: shapes do not fit together")
+    _check_rotation(freq, rot_dims, layout, head_dim, "rotate_rows")
+    out = torch.empty((n, n_heads * head_dim), dtype=torch.float32, device=proj.device)
+    lib = core()
+    _check(lib, lib.qil_rotate_rows(_p(proj), c_longlong(ld), c_int(column), c_int(n_heads), c_int(head_dim), _p(freq),
+                                    c_int(rot_dims), c_int(layout), c_float(gain), _p(positions),
+                                    c_int(n_heads if scaled_from is None else scaled_from), c_float(scale), c_int(n), _p(out),
+                                    c_int(dtype_code(proj.dtype)), _stream()), "rotate_rows")
+    return out
+
+
+def state_scan_needs_scratch(d, e) -> bool:
+    """Do a head's ``e`` value columns take more than one block of :func:`state_scan`?"""
+    code = core().qil_state_scan_needs_scratch(c_int(d), c_int(e))
+    if code < 0:
+        raise KernelError(f"state_scan: {d} key channels per head are too many")
+    return bool(code)
+
+
+def state_chunk_most_d() -> int:
+    """The most key channels per head that :func:`state_chunks` takes."""
+    return core().qil_state_chunk_most_d()
+
+
+class StateRows:
+    """What enters a recurrence with a state matrix per head (csrc/matrix_state.cu): ``qk`` float32 [N, 2 * kv_heads * d] (all
+    q heads, then all k heads), ``values`` = (rows [N, width], column of the first of heads * e values), decays ``log_decay``
+    float32 [N, heads] or ``head_decay`` float32 [heads], and with the delta rule's correction ``beta`` float32 [N, heads]."""
+
+    def __init__(self, qk, values, n_heads, n_kv_heads, d, e, *, log_decay=None, head_decay=None, beta=None):
+        rows, column = values
+        _need(qk, "qk", torch.float32, 2); _need(rows, "values", ndim=2)
+        n = rows.shape[0]
+        if qk.shape != (n, 2 * n_kv_heads * d) or n_heads % n_kv_heads or column < 0 or column + n_heads * e > rows.shape[1]:
+            raise KernelError(f"state rows: q/k {tuple(qk.shape)}, values {tuple(rows.shape)} for {n_heads} heads of {d}/{e}")
+        if (log_decay is None) == (head_decay is None):
+            raise KernelError("state rows: decays per token or per head")
+        for t, name in ((log_decay, "log_decay"), (beta, "beta")):
+            if t is not None:
+                _need(t, name, torch.float32, 2)
+                if t.shape != (n, n_heads):
+                    raise KernelError(f"state rows: one {name} per token and head")
+        if head_decay is not None:
+            _need(head_decay, "head_decay", torch.float32, 1)
+            if head_decay.shape[0] != n_heads:
+                raise KernelError("state rows: one decay per head")
+        self.n, self.n_heads, self.d, self.e, self.delta = n, n_heads, d, e, beta is not None
+        self.dtype = rows.dtype
+        self._keep = (qk, rows, log_decay, head_decay, beta)
+        self.arguments = (c_void_p(qk.data_ptr()), c_void_p(qk.data_ptr() + n_kv_heads * d * 4), c_longlong(qk.shape[1]),
+                          c_int(n_heads // n_kv_heads), c_void_p(rows.data_ptr() + column * rows.element_size()),
+                          c_longlong(rows.shape[1]), _p(log_decay), _p(head_decay), _p(beta))
+
+
+def state_scan(inputs, gate, norm_weight, eps, slots, seg_start, seg_len, seg_row, n_segments, *, out=None, raw=None):
+    """The recurrence of ``inputs`` (a :class:`StateRows`) over segments, token by token from the slots ``seg_row`` names (``slots``
+    float32 [slots, heads, d, e], read and written).  ``out`` [N, heads * e]: every head divided by its root mean square, times
+    ``norm_weight`` (float32 [e], or None) and silu of ``gate`` = (rows, column) (or None); or ``raw`` float32 [N, heads * e]:
+    the outputs as they are."""
+    _need(slots, "slots", torch.float32, 4)
+    heads, d, e = inputs.n_heads, inputs.d, inputs.e
+    if tuple(slots.shape[1:]) != (heads, d, e):
+        raise KernelError(f"state_scan: slots {tuple(slots.shape)} for {heads} heads of {d}/{e}")
+    for t in (seg_start, seg_len, seg_row):
+        _need(t, "segments", torch.int32, 1)
+        if t.shape[0] < n_segments:
+            raise KernelError("state_scan: fewer segment entries than segments")
+    gate_ptr, gate_ld = c_void_p(0), 0
+    if raw is not None:
+        _need(raw, "raw", torch.float32, 2)
+    else:
+        _need(out, "out", inputs.dtype, 2)
+        if norm_weight is not None:
+            _need(norm_weight, "norm_weight", torch.float32, 1)
+        if gate is not None:
+            rows, column = gate
+            _need(rows, "gate", inputs.dtype, 2)
+            if rows.shape[0] != inputs.n or column < 0 or column + heads * e > rows.shape[1]:
+                raise KernelError("state_scan: the gate's columns lie outside its buffer")
+            gate_ptr, gate_ld = c_void_p(rows.data_ptr() + column * rows.element_size()), rows.shape[1]
+    target = raw if raw is not None else out
+    if target.shape != (inputs.n, heads * e) or (raw is None and norm_weight is not None and norm_weight.shape[0] != e):
+        raise KernelError("state_scan: the outputs or the norm's weight have another shape")
+    lib = core()
+    _check(lib, lib.qil_state_scan(*inputs.arguments, gate_ptr, c_longlong(gate_ld), _p(norm_weight), c_float(eps), _p(slots),
+                                   _p(seg_start), _p(seg_len), _p(seg_row), c_int(n_segments), c_int(heads), c_int(d), c_int(e),
+                                   _p(raw), _p(out if raw is None else None), c_int(dtype_code(inputs.dtype)), _stream()),
+           "state_scan")
+
+
+def state_chunks(inputs, slots, chunk_start, chunk_len, n_chunks, carry, n_carries, raw):
+    """The recurrence of ``inputs`` over the chunks of a step's long portions (``parts.linear_attention.ScanPlanner``), as matrix
+    products: ``raw`` float32 [N, heads * e] receives the outputs of the chunks' tokens as they are, ``slots`` move on.
+    ``carry`` int32 [n_carries * 3] = (slot, first chunk, chunks)."""
+    heads, d, e = inputs.n_heads, inputs.d, inputs.e
+    _need(slots, "slots", torch.float32, 4); _need(raw, "raw", torch.float32, 2)
+    for t, count in ((chunk_start, n_chunks), (chunk_len, n_chunks), (carry, 3 * n_carries)):
+        _need(t, "chunks", torch.int32, 1)
+        if t.shape[0] < count:
+            raise KernelError("state_chunks: fewer entries than chunks")
+    if tuple(slots.shape[1:]) != (heads, d, e) or raw.shape != (inputs.n, heads * e):
+        raise KernelError("state_chunks: shapes do not fit together")
+    lib = core()
+    chunk = lib.qil_state_chunk()
+    empty = lambda *shape: torch.empty(shape, dtype=torch.float32, device=slots.device)
+    y, w = (empty(n_chunks, heads, chunk, e), empty(n_chunks, heads, chunk, d)) if inputs.delta else (None, None)
+    states = empty(n_chunks, heads, d, e)
+    _check(lib, lib.qil_state_chunks(*inputs.arguments, _p(chunk_start), _p(chunk_len), c_int(n_chunks), _p(carry),
+                                     c_int(n_carries), c_int(heads), c_int(d), c_int(e), _p(y), _p(w), _p(states), _p(slots),
+                                     _p(raw), c_int(dtype_code(inputs.dtype)), _stream()), "state_chunks",
+           kernels=3 if inputs.delta else 2)
+
+
+def delta_prepare(proj, columns, taps_weight, state, a_log, dt_bias, q_scale, positions, token_row, heads, kv_heads, d, e):
+    """What a gated delta rule reads, from its projection's rows ``proj`` [N, width], whose first columns are q and k
+    [kv_heads * d] and v [heads * e]: (qk float32 [N, 2 * kv_heads * d], v [N, heads * e], beta, log_decay float32 [N, heads]).
+    q, k, v pass the convolution ``taps_weight`` float32 [taps, channels] over time (``state`` float32 [slots, taps - 1,
+    channels], None without earlier taps) and silu; q and k become unit vectors per head, q times ``q_scale``;
+    beta = sigmoid(b), log_decay = -exp(a_log) softplus(a + dt_bias), ``columns`` = (b, a): the first of each one's columns."""
+    _need(proj, "proj", ndim=2); _need(taps_weight, "taps_weight", torch.float32, 2)
+    _need(a_log, "a_log", torch.float32, 1); _need(dt_bias, "dt_bias", torch.float32, 1)
+    _need(positions, "positions", torch.int32, 1); _need(token_row, "token_row", torch.int32, 1)
+    n, ld = proj.shape
+    taps, channels = taps_weight.shape
+    if channels != 2 * kv_heads * d + heads * e or channels > ld or any(c < 0 or c + heads > ld for c in columns) \
+            or a_log.shape[0] != heads or dt_bias.shape[0] != heads:
+        raise KernelError("delta_prepare: shapes do not fit together")
+    if taps > 1:
+        _need(state, "state", torch.float32, 3)
+        if tuple(state.shape[1:]) != (taps - 1, channels):
+            raise KernelError(f"delta_prepare: state {tuple(state.shape)} for {taps} taps and {channels} channels")
+    f32 = lambda width: torch.empty((n, width), dtype=torch.float32, device=proj.device)
+    qk, beta, log_decay = f32(2 * kv_heads * d), f32(heads), f32(heads)
+    v = torch.empty((n, heads * e), dtype=proj.dtype, device=proj.device)
+    lib = core()
+    _check(lib, lib.qil_delta_prepare(_p(proj), c_longlong(ld), c_int(columns[0]), c_int(columns[1]), _p(taps_weight), c_int(taps),
+                                      _p(state if taps > 1 else None), _p(a_log), _p(dt_bias), c_float(q_scale), _p(positions),
+                                      _p(token_row), c_int(n), c_int(heads), c_int(kv_heads), c_int(d), c_int(e), _p(qk), _p(v),
+                                      _p(beta), _p(log_decay), c_int(dtype_code(proj.dtype)), _stream()), "delta_prepare")
+    return qk, v, beta, log_decay
 
 
 def latent_prepare(proj, q_column, kv_column, q_att, kv_cache, norm_w, eps, freq, rot_dims, layout, positions, token_row,

@@ -5,3 +5,4 @@ from . import debisun  # noqa: F401
 from . import larolorn  # noqa: F401
 from . import gogotar  # noqa: F401
 from . import lotazen  # noqa: F401
+from . import bugidra  # noqa: F401

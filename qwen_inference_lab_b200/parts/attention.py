@@ -32,10 +32,14 @@ their root mean square over the whole projection, all heads at once, and multipl
 the short convolution and the query temperature.  With such a rotation ``qk_norm_eps`` norms every head by itself
 (one weight of head_dim for all query heads, one for all key heads) in the same kernel.  ``values_from_keys``: there
 is no value projection; a position's value is its key as projected, before norm and rotation.  ``unit_qk_norm_eps``
-divides every q and k head by its own root mean square without a weight (after the rotation or before it, which is
-the same: a rotation keeps the sum of squares); such a layer may have a sliding window.  ``head_gate``: the
+divides every q and k head by its own root mean square without a weight (after the rotation; before it is
+the same where no gain comes with it: a rotation keeps the sum of squares); such a layer may have a sliding window.  ``head_gate``: the
 name of a [query heads, hidden] matrix G; head h's output is multiplied by sigmoid(G x)_h before the output
-projection (G's rows ride behind the keys' in the stacked projection).
+projection (G's rows ride behind the keys' in the stacked projection).  ``element_gate``: the name of a
+[query heads * v_head_dim, hidden] matrix: a gate per element instead.  ``value_mix`` = (name, first): values mixed with those
+that the first such layer of the model projected for the same token (``first`` says whether this is that layer, which
+only hands its values on, through ``ctx.shared``): v <- (1 - s) v + s v_first with the learned number s = ``name``; the pages
+hold the mixed values.
 """
 from __future__ import annotations
 
@@ -96,7 +100,7 @@ class GroupedQueryAttention(Mixer):
                  v_head_dim=None, distance_slopes=None, q_temperature=None, out_bias=None,
                  suffixes=(".weight", ".bias"), conv_taps=0, conv_suffix=".conv", softcap=0.0, distance_bias=None,
                  chunk=0, sink=False, whole_qk_norm_eps=None, norm_suffix=".weight", values_from_keys=False,
-                 head_gate=None, unit_qk_norm_eps=None):
+                 head_gate=None, unit_qk_norm_eps=None, element_gate=None, value_mix=None):
         if n_q_heads % n_kv_heads:
             raise ValueError(f"{n_q_heads} query heads do not divide into {n_kv_heads} kv heads")
         self.hidden_size, self.head_dim = int(hidden_size), int(head_dim)
@@ -128,8 +132,11 @@ class GroupedQueryAttention(Mixer):
             raise ValueError("rotation from frequencies and the norm over the whole projection go without a rotary "
                              "table, a short convolution or a query temperature, and with one kind of q/k norm")
         self.values_from_keys, self.head_gate = bool(values_from_keys), head_gate
-        if (self.values_from_keys or head_gate) and not self.frequency_tail:
-            raise ValueError("keys as values and a gate per head go with the rotation from frequencies")
+        self.element_gate, self.mixes_values, self.first_values = element_gate, value_mix is not None, bool(value_mix and value_mix[1])
+        if (self.values_from_keys or head_gate or element_gate or value_mix) and not self.frequency_tail:
+            raise ValueError("keys as values, mixed values and output gates go with the rotation from frequencies")
+        if (head_gate and element_gate) or (value_mix and (self.values_from_keys or reads_shared_cache)):
+            raise ValueError("one kind of output gate, and mixed values are projected ones")
         if self.values_from_keys and (reads_shared_cache or (v_head_dim and int(v_head_dim) != int(head_dim))):
             raise ValueError("keys as values need keys of the layer's own, and values as large as keys")
         if isinstance(position, RotaryFrequencies) and position.rotary_dim > self.head_dim:
@@ -155,10 +162,16 @@ class GroupedQueryAttention(Mixer):
                 pieces += [(names["v"], n_kv_heads * self.v_head_dim)]
         if head_gate:
             pieces += [(head_gate, n_q_heads)]
+        if element_gate:
+            pieces += [(element_gate, n_q_heads * self.v_head_dim)]
         self.qkv = StackedLinear(hidden_size, pieces, bias=bias, suffixes=suffixes)
         self.out = Linear(n_q_heads * self.v_head_dim, hidden_size, name=names["o"],
                           bias=bias if out_bias is None else out_bias, suffixes=suffixes)
         self._extra = {}
+        self.value_share, self._share = None, 0.0
+        if value_mix is not None:
+            self.value_share = Param((), std=0.5, optional=self.first_values)
+            self._extra[value_mix[0]] = self.value_share
         self.conv = None
         if self.conv_taps:
             self.conv = [Param((rows, self.conv_taps), std=0.5) for _, rows in pieces]
@@ -203,6 +216,8 @@ class GroupedQueryAttention(Mixer):
         super().finalize(device, dtype)
         if self.q_norm is not None and self.q_norm.data.dtype != self.k_norm.data.dtype:
             self.q_norm.data, self.k_norm.data = self.q_norm.data.float(), self.k_norm.data.float()
+        if self.value_share is not None and self.value_share.data is not None:
+            self._share = float(self.value_share.data)
         if self.distance_slopes is not None:
             self._slopes = torch.tensor(self.distance_slopes, dtype=torch.float32, device=device)
             self._slopes_log2 = (self._slopes.double() * 1.4426950408889634).float().contiguous()
@@ -269,6 +284,11 @@ class GroupedQueryAttention(Mixer):
             k_weight = self.k_norm if per_head else self.whole_k_norm
             # keys as values: the value rows are copied from the keys' columns, as projected
             v_column = q_width if self.values_from_keys else q_width + k_width
+            mix = None
+            if self.first_values:
+                ctx.shared["first_values"] = (qkv, at + v_column)
+            elif self.mixes_values:
+                mix = (*ctx.shared["first_values"], self._share)
             ops.qk_rotate_store(qkv, (at, at + q_width, at + v_column), q, cache.pages,
                                 q_weight.data if q_weight is not None else None,
                                 k_weight.data if k_weight is not None else None,
@@ -277,11 +297,14 @@ class GroupedQueryAttention(Mixer):
                                 rotation.rotary_dim if rotation is not None else 0,
                                 rotation.layout if rotation is not None else 0, ctx.positions, ctx.token_row,
                                 cache.block_table, self.n_q_heads, n_kv, self.head_dim, self.v_head_dim, cache.page_size,
-                                per_head=per_head, unit_heads=self.unit_qk_norm_eps is not None)
+                                per_head=per_head, unit_heads=self.unit_qk_norm_eps is not None,
+                                gain=rotation.gain if rotation is not None else 1.0, mix=mix)
             attended = ctx.empty((n, self.n_q_heads * self.v_head_dim))
             self._attend(ctx, q, cache, attended)
             if self.head_gate:
                 ops.head_gate(attended, self.v_head_dim, qkv, at + self.qkv.out_features - self.n_q_heads)
+            if self.element_gate:
+                ops.head_gate(attended, 1, qkv, at + self.qkv.out_features - attended.shape[1])
             return self.out.forward(ctx, attended, residual=residual, out_scale=out_scale, out_float32=out_float32)
         if out_float32:
             raise ValueError("a float32 result is given by the layers that rotate by frequencies only")
@@ -340,11 +363,11 @@ class GroupedQueryAttention(Mixer):
         return self.out.forward(ctx, attended, residual=residual)
 
     def _attend(self, ctx, q, cache, out):
-        tensor_cores = q.dtype == torch.bfloat16 and self.v_head_dim == self.head_dim \
-            and attention_mma.supports(self.head_dim, self.n_q_heads, self.n_kv_heads)
+        tensor_cores = q.dtype == torch.bfloat16 \
+            and attention_mma.supports(self.head_dim, self.n_q_heads, self.n_kv_heads, self.v_head_dim)
         if self.modified_scores and tensor_cores:
             attention_mma.attend(ctx, q, cache, out, self.n_q_heads, self.n_kv_heads, self.head_dim, 0, self.scale,
-                                 self._slopes_log2, self._options)
+                                 self._slopes_log2, self._options, v_dim=self.v_head_dim)
             return
         if self.modified_scores:
             ops.attention_generic(q, cache.pages, out, ctx.positions, ctx.token_row, cache.block_table,
@@ -353,10 +376,9 @@ class GroupedQueryAttention(Mixer):
                                   softcap=self.softcap, distance_bias=self._bias_by_distance, chunk=self.chunk,
                                   sink=self.sink, sink_logits=self._sinks)
             return
-        if q.dtype == torch.bfloat16 and self.v_head_dim == self.head_dim \
-                and attention_mma.supports(self.head_dim, self.n_q_heads, self.n_kv_heads):
+        if tensor_cores:
             attention_mma.attend(ctx, q, cache, out, self.n_q_heads, self.n_kv_heads, self.head_dim,
-                                 self.window, self.scale, self._slopes_log2)
+                                 self.window, self.scale, self._slopes_log2, v_dim=self.v_head_dim)
             return
         ops.attention_generic(q, cache.pages, out, ctx.positions, ctx.token_row, cache.block_table,
                               self.n_q_heads, self.n_kv_heads, self.head_dim, cache.page_size,

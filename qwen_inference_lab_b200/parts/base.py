@@ -140,8 +140,9 @@ class Norm(Part):
         return None
 
     def as_join(self):
-        """(weight [width], eps, kind) if this norm is one that the kernels which join branches to the stream can
-        apply to the new stream (``kernels.ops.NORM_KINDS``), else None."""
+        """If this norm is one that the kernels which join branches to the stream can apply to the new stream
+        (``kernels.ops.NORM_KINDS``): ``kernels.ops.branch_join``'s arguments for it, next_weight [width], next_kind and what
+        that kind takes; else None."""
         return None
 
 
@@ -244,6 +245,8 @@ class StepContext:
     h_seg_pos0: object = None
     # the runner's own dict, the same one every step: parts keep scratch buffers here under their own keys
     extras: dict = field(default_factory=dict)
+    # what parts of this step leave to later parts of the same step, by their own keys (values that a later layer mixes in)
+    shared: dict = field(default_factory=dict)
     # dtype of the residual stream when it differs from the activations' (a model that keeps it in float32)
     stream_dtype: torch.dtype | None = None
 

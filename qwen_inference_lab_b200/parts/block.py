@@ -15,6 +15,7 @@ of the block's.  And parts that run on the stream after the feed-forward (``afte
 sublayer's output, x <- x + m * norm1(mixer(x)), x <- x + m * norm2(ff(x)) with a fixed multiplier m.
 :class:`ParallelBlock` has one norm whose output both sublayers read: x <- x + mixer(h) + ff(h), h = norm(x).
 :class:`SandwichNormBlock` norms on both sides of each sublayer: x <- x + post1(mixer(pre1 x)), x <- x + post2(ff(pre2 x)).
+:class:`DeferredPreNormBlock` is the pre-norm order whose sums and norms are one kernel per sublayer.
 """
 from __future__ import annotations
 
@@ -257,20 +258,10 @@ class ParallelBlock(Part):
     def forward(self, ctx, x, cache):
         """x [N, width] is the residual stream; updated in place (by the next reader of the stream) and returned."""
         pending = ctx.extras.pop("pending_join", None)
-        how = self.norm.as_join()
-        if isinstance(pending, PendingBranches) and pending.stream is x and how is not None:
-            rows = ctx.empty(x.shape)
-            pending.settle(next_weight=how[0], next_eps=how[1], next_kind=how[2], rows=rows)
-        else:
-            if pending is not None:
-                pending.settle()
-            rows = self.norm.forward(ctx, x)
+        rows = _settled_rows(ctx, x, pending, self.norm)
         joint = self.input.forward_joint(ctx, rows)
         options = {} if joint is None else dict(joint=joint)
-        if hasattr(self.mixer, "branches"):
-            branches = list(self.mixer.branches(ctx, rows, cache, **options))
-        else:
-            branches = [(self.mixer.forward(ctx, rows, cache, out_float32=True, **options), 1.0)]
+        branches = _mixer_branches(ctx, self.mixer, rows, cache, options)
         routed = None
         if self.feed_forward is not None:
             if hasattr(self.feed_forward, "branches"):
@@ -278,24 +269,87 @@ class ParallelBlock(Part):
                 branches += more
             else:
                 branches.append((self.feed_forward.forward(ctx, rows, out_float32=True, **options), 1.0))
-        ctx.extras["pending_join"] = PendingBranches(x, branches, routed)
+        ctx.extras["pending_join"] = PendingBranches(x, branches, routed, _branch_eps(self.mixer))
         return x
 
 
-class PendingBranches:
-    """Branches that have not joined their stream yet: stream += sum of scale * branch + the experts' rows."""
-    __slots__ = ("stream", "branches", "routed")
+class DeferredPreNormBlock(Part):
+    """The pre-norm order, x <- x + mixer(norm1 x), then x <- x + ff(norm2 x), for a float32 stream: a sublayer gives its
+    branch unsummed (two mixers side by side: both, with the weights of their norms), and ``ops.branch_join`` adds it to the
+    stream and norms the new stream for the sublayer that reads it next, in one kernel.  That also holds from block to block:
+    a block leaves its last branch in ``ctx.extras["pending_join"]`` and the next block of this kind joins it together with
+    its own first norm; the decoder settles what is left before anyone else reads the stream.  The mixer's first products run
+    as one where it has several (:class:`JointProjection`).  ``feed_forward`` may be None; a second norm given all the same
+    only claims its tensors."""
+    takes_pending_join = True
+    graph_safe = True
 
-    def __init__(self, stream, branches, routed):
-        self.stream, self.branches, self.routed = stream, branches, routed
+    def __init__(self, mixer_norm, mixer, ff_norm, feed_forward):
+        self.mixer_norm, self.mixer = mixer_norm, mixer
+        self.ff_norm, self.feed_forward = ff_norm, feed_forward
+        self.input = JointProjection(mixer.input_projections() if hasattr(mixer, "input_projections") else [])
+
+    def children(self):
+        return [part for part in (self.mixer_norm, self.mixer, self.ff_norm, self.feed_forward) if part is not None]
+
+    def finalize(self, device, dtype):
+        super().finalize(device, dtype)
+        self.input.join()
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def forward(self, ctx, x, cache):
+        """x [N, width] is the residual stream; updated in place (by the next reader of the stream) and returned."""
+        rows = _settled_rows(ctx, x, ctx.extras.pop("pending_join", None), self.mixer_norm)
+        joint = self.input.forward_joint(ctx, rows)
+        branches = _mixer_branches(ctx, self.mixer, rows, cache, {} if joint is None else dict(joint=joint))
+        pending = PendingBranches(x, branches, None, _branch_eps(self.mixer))
+        if self.feed_forward is not None:
+            rows = _settled_rows(ctx, x, pending, self.ff_norm)
+            pending = PendingBranches(x, [(self.feed_forward.forward(ctx, rows, out_float32=True), 1.0)], None)
+        ctx.extras["pending_join"] = pending
+        return x
+
+
+def _branch_eps(mixer):
+    """eps of the norms that a mixer's branches still want (``ParallelMixers.branches``)."""
+    return getattr(mixer, "norm_eps", 0.0)
+
+
+def _mixer_branches(ctx, mixer, rows, cache, options):
+    if hasattr(mixer, "branches"):
+        return list(mixer.branches(ctx, rows, cache, **options))
+    return [(mixer.forward(ctx, rows, cache, out_float32=True, **options), 1.0)]
+
+
+def _settled_rows(ctx, x, pending, norm):
+    """norm(x) after what is pending has joined the stream x, in one kernel where norm and branches allow it."""
+    how = norm.as_join()
+    if isinstance(pending, PendingBranches) and pending.stream is x and how is not None:
+        rows = ctx.empty(x.shape)
+        pending.settle(rows=rows, **how)
+        return rows
+    if pending is not None:
+        pending.settle()
+    return norm.forward(ctx, x)
+
+
+class PendingBranches:
+    """Branches that have not joined their stream yet: stream += sum of scale * branch (normed with its weight and ``eps``, where
+    it has one) + the experts' rows."""
+    __slots__ = ("stream", "branches", "routed", "eps")
+
+    def __init__(self, stream, branches, routed, eps=0.0):
+        self.stream, self.branches, self.routed, self.eps = stream, branches, routed, eps
 
     def settle(self, **norm):
-        ops.branch_join(self.stream, self.branches, routed=self.routed, **norm)
+        ops.branch_join(self.stream, self.branches, routed=self.routed, branch_eps=self.eps, **norm)
 
 
 def settle_stream(ctx):
-    """Join what a block left unjoined (see :class:`SandwichNormBlock`, :class:`ParallelBlock`); for whoever reads the
-    stream next."""
+    """Join what a block left unjoined (see :class:`SandwichNormBlock`, :class:`ParallelBlock`,
+    :class:`DeferredPreNormBlock`); for whoever reads the stream next."""
     pending = ctx.extras.pop("pending_join", None)
     if pending is not None:
         pending.settle()

@@ -1,4 +1,4 @@
-"""Norms over the last dimension: root-mean-square norms and a layer norm.
+"""Norms over the last dimension: root-mean-square norms, a layer norm and Dynamic Tanh, which has no statistics.
 
 ``y = cast(x32 * rsqrt(mean(x32^2) + eps)) * w``: statistics and scaling in float32,
 rounded to the activation dtype, then multiplied by the weight (no ``1 + w``), as the
@@ -49,7 +49,7 @@ class ExactRMSNorm(Norm):
         return ops.rmsnorm_exact(x, self.weight.data, self.eps, self.offset, out_dtype=ctx.dtype, rows=rows)
 
     def as_join(self):
-        return (self.weight.data, self.eps, "rms") if self.offset == 0.0 else None
+        return dict(next_weight=self.weight.data, next_eps=self.eps, next_kind="rms") if self.offset == 0.0 else None
 
 
 class ScalarRMSNorm(Norm):
@@ -73,7 +73,7 @@ class ScalarRMSNorm(Norm):
         return ops.rmsnorm_exact(x, self._row, self.eps, 0.0, out_dtype=ctx.dtype, rows=rows)
 
     def as_join(self):
-        return self._row, self.eps, "rms"
+        return dict(next_weight=self._row, next_eps=self.eps, next_kind="rms")
 
 
 class LayerNorm(Norm):
@@ -103,4 +103,33 @@ class LayerNorm(Norm):
                                    out_dtype=ctx.dtype, rows=rows)
 
     def as_join(self):
-        return (self.weight.data, self.eps, "layer") if self.bias is None else None
+        return dict(next_weight=self.weight.data, next_eps=self.eps, next_kind="layer") if self.bias is None else None
+
+
+class TanhNorm(Norm):
+    """Dynamic Tanh: ``y = tanh(alpha x) * w + b`` with one learned number alpha (a tensor without dimensions): no mean, no
+    variance, float32 arithmetic and a single rounding.  ``suffixes``: what the checkpoint appends to ``name`` for the
+    weight, the bias and alpha."""
+    graph_safe = True
+
+    def __init__(self, width, *, name, suffixes=(".weight", ".bias", ".alpha"), optional=False):
+        self.width, self.name, self.suffixes = int(width), name, tuple(suffixes)
+        self.weight = Param((width,), init="norm", std=0.05, optional=optional)
+        self.bias = Param((width,), init="normal", std=0.05, optional=optional)
+        self.alpha = Param((), init="norm", std=0.05, optional=optional)
+        self._alpha = None
+
+    def named_params(self):
+        return {self.name + suffix: param for suffix, param in zip(self.suffixes, (self.weight, self.bias, self.alpha))}
+
+    def finalize(self, device, dtype):
+        if self.weight.data is None:
+            return
+        self.bias.data = self.bias.data.to(self.weight.data.dtype)       # the kernels read both as one dtype
+        self._alpha = float(self.alpha.data)
+
+    def forward(self, ctx, x, rows=None):
+        return ops.tanh_norm(x, self.weight.data, self.bias.data, self._alpha, out_dtype=ctx.dtype, rows=rows)
+
+    def as_join(self):
+        return dict(next_weight=self.weight.data, next_kind="tanh", next_bias=self.bias.data, next_alpha=self._alpha)

@@ -6,7 +6,7 @@ its own, and the mixer's result is a weighted sum of the two (half the sum, by d
 The two keep their own caches: the mixer's cache spec is the tuple of theirs, its view the tuple of their views.
 A pair of scales in place of ``norm_eps``, weights and share (``scales`` = (left, right)) gives the plain weighted sum
 y = left_scale * left(h) + right_scale * right(h); a block that joins several branches at once takes the two unsummed
-(``branches``).
+(``branches``), of either kind of pair: the kernel that joins them norms them on the way.
 Inside a block that norms its branches on the way into the stream (:class:`PostNormBlock`) the two norms, the sum,
 the block's own norm and the residual sum are one kernel (``kernels.ops.rms_join``), so the mixer joins the stream
 itself (``joins_stream``); ``forward`` without a stream returns y in float32.
@@ -47,6 +47,8 @@ class ParallelMixers(Mixer):
         super().finalize(device, dtype)
         if self.scales is None and self.left_weight.data.dtype != self.right_weight.data.dtype:
             self.left_weight.data, self.right_weight.data = self.left_weight.data.float(), self.right_weight.data.float()
+        if self.scales is None:        # the kernel that joins branches reads their weights as float32
+            self._branch_weights = tuple(w.data.float().contiguous() for w in (self.left_weight, self.right_weight))
 
     def cache_spec(self):
         flat = []
@@ -66,11 +68,14 @@ class ParallelMixers(Mixer):
         return found
 
     def branches(self, ctx, x, cache, joint=None):
-        """[(left's float32 rows, its scale), (right's, its scale)], of a pair that is summed by scales."""
+        """[(left's float32 rows, its scale), (right's, its scale)]; with a third entry each, the weight of the norm that the
+        rows still want (``norm_eps``), of a pair that is summed through norms."""
         views = self._views(cache)
         how = {} if joint is None else dict(joint=joint)
-        return [(part.forward(ctx, x, view, out_float32=True, **how), scale)
-                for part, view, scale in zip((self.left, self.right), views, self.scales)]
+        found = [part.forward(ctx, x, view, out_float32=True, **how) for part, view in zip((self.left, self.right), views)]
+        if self.scales is not None:
+            return list(zip(found, self.scales))
+        return [(rows, self.share, weight) for rows, weight in zip(found, self._branch_weights)]
 
     def forward(self, ctx, x, cache, stream=None, norm_weight=None, mult=1.0, out_float32=True, rows=None):
         """x [N, hidden] -> y float32 [N, hidden]; with ``stream`` (the residual stream, updated in place and

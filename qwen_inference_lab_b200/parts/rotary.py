@@ -50,11 +50,14 @@ class RotaryFrequencies(PositionEncoding):
     wavelength l = 2 pi / freq, a frequency stays when l < original / high, becomes freq / factor when
     l > original / low, and between the two is (1 - s) freq / factor + s freq with
     s = (original / l - low) / (high - low).  ``stretch`` divides every frequency, whatever its wavelength (linear
-    scaling of the positions)."""
+    scaling of the positions).  ``ramp`` = (factor, original, fast, slow) is YaRN's scaling: with
+    pair(t) = dims ln(original / (2 pi t)) / (2 ln base), the number of the pair that makes t turns over ``original``
+    positions, pairs up to max(floor(pair(fast)), 0) keep their frequency, pairs from min(ceil(pair(slow)), dims - 1) on are
+    divided by factor, those between are mixed linearly; ``gain`` = 1 + ln(factor) / 10 then multiplies cosines and sines."""
     graph_safe = True
     LAYOUTS = {"halves": 0, "interleaved": 1}
 
-    def __init__(self, dims, base, layout="halves", scaling=None, stretch=1.0):
+    def __init__(self, dims, base, layout="halves", scaling=None, stretch=1.0, ramp=None):
         if dims % 2 or dims <= 0:
             raise ValueError(f"the number of rotated dimensions must be positive and even, got {dims}")
         if layout not in self.LAYOUTS:
@@ -67,11 +70,30 @@ class RotaryFrequencies(PositionEncoding):
         if self.scaling is not None and (len(self.scaling) != 4 or self.scaling[0] <= 0 or self.scaling[3] <= 0
                                          or not 0 < self.scaling[1] < self.scaling[2]):
             raise ValueError(f"frequency scaling wants (factor, low, high, original) with 0 < low < high, got {scaling}")
+        self.ramp = None if ramp is None else tuple(float(v) for v in ramp)
+        self.gain = 1.0
+        if self.ramp is not None:
+            if len(self.ramp) != 4 or any(not v > 0 for v in self.ramp) or self.scaling is not None or self.stretch != 1.0 \
+                    or not self.base > 1:
+                raise ValueError(f"a ramp wants positive (factor, original, fast, slow), a base above one and no other scaling; got {ramp}")
+            self.gain = 0.1 * math.log(self.ramp[0]) + 1.0
         self.freq = None
+
+    def _ramped(self, values) -> list:
+        factor, original, fast, slow = self.ramp
+        pair = lambda turns: self.rotary_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+        first, last = max(math.floor(pair(fast)), 0), min(math.ceil(pair(slow)), self.rotary_dim - 1)
+        mixed = []
+        for i, f in enumerate(values):
+            slowed = min(max((i - first) / max(last - first, 0.001), 0.0), 1.0)
+            mixed.append(f / factor * slowed + f * (1.0 - slowed))
+        return mixed
 
     def frequencies(self) -> list:
         """The frequency of every rotated pair as Python floats (float64)."""
         values = [self.base ** (-2.0 * i / self.rotary_dim) / self.stretch for i in range(self.rotary_dim // 2)]
+        if self.ramp is not None:
+            return self._ramped(values)
         if self.scaling is None:
             return values
         factor, low, high, original = self.scaling
