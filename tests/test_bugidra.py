@@ -98,7 +98,7 @@ def test_a_configuration_comes_back_as_it_was():
     assert BugidraConfig.from_dict(bare).embedding_scale == 1.0
 
 
-ROTATIONS = [cases.rot(10000.0, 64, (2.0, 1024, 32.0, 1.0)), cases.rot(500.0, 8, (4.0, 64, 8.0, 1.0)), cases.rot(100.0, 2, (16.0, 500, 64.0, 3.0)),
+ROTATIONS = [cases.rot(20000.0, 48, (2.5, 900, 24.0, 1.5)), cases.rot(500.0, 8, (4.0, 64, 8.0, 1.0)), cases.rot(100.0, 2, (16.0, 500, 64.0, 3.0)),
              cases.rot(2.0, 16, (3.0, 10, 100.0, 50.0)), cases.rot(1e6, 32), cases.rot(1e6, 96, (1.0, 4096, 4.0, 4.0))]
 
 
