@@ -1459,6 +1459,207 @@ def run_lotazen(args):
         torch.cuda.empty_cache()
 
 
+# --------------------------------------------------------------------------- Bugidra beside Virulix
+BUGIDRA_SHAPES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, lin_heads=8, lin_dim=128, lin_vdim=128, ff=6144, vocab=32768),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, lin_heads=16, lin_dim=128, lin_vdim=128, ff=12288, vocab=32768),
+}
+
+
+def _bugidra_sizes(width, heads, kv_heads, dim, lin_heads, lin_dim, lin_vdim, ff, vocab):
+    """Eight layers: the gated delta rule, attention beside retention, gated attention, attention beside retention, twice."""
+    attention = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5)
+    left = dict(attention, rot=dict(base=500000.0, dims=dim, scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0)))
+    right = dict(heads=lin_heads, dim=lin_dim, vdim=lin_vdim, rot=dict(base=10000.0, dims=lin_dim),
+                 decay=[1.0 - 2.0 ** -(5 + i % 6) for i in range(lin_heads)])
+    mlp = dict(kind="dense", ff=ff)
+    pair = dict(type="parallel", mixer=dict(left=left, right=right), mlp=mlp)
+    gated = dict(type="attention", mixer=dict(attention, rot=dict(base=500000.0, dims=dim // 2), softcap=30.0, v_mix=True), mlp=mlp)
+    delta = dict(type="delta", mixer=dict(heads=lin_heads, kv_heads=lin_heads, dim=lin_dim, vdim=lin_vdim, conv=4), mlp=mlp)
+    return dict(architecture="Bugidra", vocab=vocab, width=width, norm=dict(eps=1e-6), embedding=dict(scale=1.0),
+                layers=[delta, pair, gated, pair] * 2)
+
+
+def _bugidra_kernels(torch, bugidra, virulix, sizes, pk, tokens_n, batch, context, flush):
+    """The kernels of Bugidra's mechanisms alone, each beside the like kernel of Virulix (the short convolution: of Debisun, the
+    join: of Gogotar), with what the roofline allows."""
+    from qwen_inference_lab_b200.kernels import ops
+    from qwen_inference_lab_b200.parts import GroupedQueryAttention
+    bench = _PartKernels(torch, pk, tokens_n, batch, context, flush)
+    H, G, d, W = sizes["heads"], sizes["kv_heads"], sizes["dim"], sizes["width"]
+    delta, pair, gated = (bugidra.layers[i].mixer for i in (0, 1, 6))
+    left, right = pair.left, pair.right
+    theirs = next(l.mixer for l in virulix.layers if hasattr(l.mixer, "plain_tail"))
+    their_gla = next(l.mixer for l in virulix.layers if hasattr(l.mixer, "decay_rank"))
+    pairs_all = tokens_n * (tokens_n + 1) // 2
+
+    # ---- attention itself
+    def attention(mixer):
+        def kernel(ctx, x, view):
+            q = x[:, :H * d].contiguous()
+            out = torch.empty((x.shape[0], H * mixer.v_head_dim), dtype=x.dtype, device=x.device)
+            bench.timed(lambda: mixer._attend(ctx, q, view, out))
+            return out
+        return kernel
+    narrow = GroupedQueryAttention(W, H, G, d, names=dict(q="q", k="k", v="v", o="o"), v_head_dim=d // 2, unit_qk_norm_eps=1e-6,
+                                   position=left.position)
+    for param in narrow.all_named_params().values():
+        param.data = torch.zeros(param.shape, dtype=torch.bfloat16, device="cuda")
+    narrow.finalize(torch.device("cuda"), torch.bfloat16)
+    for label, mixer in (("bugidra attention of unit heads", left), ("bugidra capped attention", gated),
+                         ("bugidra attention, values half as wide as keys", narrow), ("virulix attention (distance slopes)", theirs)):
+        widths = d + mixer.v_head_dim
+        bench.measure(label, mixer, H * d, attention(mixer), (2.0 * H * widths * pairs_all, None), batch * (context + 1) * G * widths * 2)
+
+    # ---- what stands between the projection and the attention, and behind it
+    channels = (H + 2 * G) * d
+    moved = lambda n, width: 2 * n * width * 2          # every row read once and written once
+    def rotate_store(mixer, mix):
+        whole = mixer.whole_q_norm is not None
+        def kernel(ctx, x, view):
+            qkv = x[:, :channels].contiguous()
+            first = x[:, channels:channels + G * d].contiguous()
+            q = torch.empty((x.shape[0], H * d), dtype=x.dtype, device=x.device)
+            bench.timed(lambda: ops.qk_rotate_store(
+                qkv, (0, H * d, (H + G) * d), q, view.pages, mixer.whole_q_norm.data if whole else None,
+                mixer.whole_k_norm.data if whole else None, 1e-6, mixer.position.freq, mixer.position.rotary_dim,
+                mixer.position.layout, ctx.positions, ctx.token_row, view.block_table, H, G, d, d, view.page_size,
+                unit_heads=not whole, gain=mixer.position.gain, mix=(first, 0, 0.25) if mix else None))
+            return q
+        return kernel
+    def plain_store(ctx, x, view):
+        qkv = x[:, :channels].contiguous()
+        q = torch.empty((x.shape[0], H * d), dtype=x.dtype, device=x.device)
+        bench.timed(lambda: ops.qkv_store(qkv, q, view.pages, ctx.positions, ctx.token_row, view.block_table, H, G, d, d,
+                                          view.page_size, 0.1, 256))
+        return q
+    bench.measure("bugidra unit heads + rotation by halves + page write", left, channels, rotate_store(left, False),
+                  (None, moved(tokens_n, channels)), moved(batch, channels))
+    mixed_bytes = lambda n: moved(n, channels) + n * G * d * 2
+    bench.measure("bugidra norm over q and k + rotation + mixed values + page write", gated, channels + G * d, rotate_store(gated, True),
+                  (None, mixed_bytes(tokens_n)), mixed_bytes(batch))
+    bench.measure("virulix query temperature + page write", theirs, channels, plain_store, (None, moved(tokens_n, channels)),
+                  moved(batch, channels))
+    gate_bytes = lambda n: 3 * n * H * d * 2
+    def element_gate(ctx, x, view):
+        attended, gates = x[:, :H * d].contiguous(), x[:, H * d:2 * H * d].contiguous()
+        return bench.timed(lambda: ops.head_gate(attended, 1, gates, 0))
+    bench.measure("bugidra gate per element", gated, 2 * H * d, element_gate, (None, gate_bytes(tokens_n)), gate_bytes(batch))
+
+    # ---- the recurrences: float32 on the CUDA cores by both designs, so the prompt's bound is the float32 FMA rate
+    fma = (148 * 128 * 2 * 1.9e9, "of the float32 FMA rate (72 TFLOP/s nominal)")
+    def scan(part, name, work):
+        width = part.projection.out_features
+        def kernel(ctx, x, view):
+            projected = x[:, :width].contiguous()
+            return bench.timed(lambda: part.scan(ctx, projected, 0, view))
+        state = part.n_heads * part.key_dim * part.value_dim
+        bench.measure(name, part, width, kernel, (work * state * tokens_n, None), batch * state * 4 * 2, prompt_of=fma)
+    scan(right, "bugidra retention (rotation, recurrence, norm and gate)", 5.0)
+    scan(delta, "bugidra gated delta rule (convolution, unit vectors, gates, recurrence, norm and gate)", 7.0)
+    gh, gd, ge = their_gla.n_heads, their_gla.key_dim, their_gla.value_dim
+    their_width = their_gla.projection.out_features
+    def gla_scan(ctx, x, view):
+        projected = x[:, :their_width].contiguous()
+        mixed = torch.empty((x.shape[0], gh * ge), dtype=x.dtype, device=x.device)
+        bench.timed(lambda: their_gla.scan(ctx, projected, view, mixed))
+        return mixed
+    bench.measure("virulix gated linear attention scan (decays, norm and gate with it)", their_gla, their_width, gla_scan,
+                  (5.0 * gh * gd * ge * tokens_n, None), batch * gh * gd * ge * 4 * 2, prompt_of=fma)
+    lin = delta.projection.out_features
+    def prepare(ctx, x, view):
+        projected = x[:, :lin].contiguous()
+        return bench.timed(lambda: ops.delta_prepare(projected, (delta.columns["b"], delta.columns["a"]), delta._taps, view[1].slots,
+                                                     delta.a_log.data, delta.dt_bias.data, delta.q_scale, ctx.positions,
+                                                     ctx.token_row, delta.n_heads, delta.n_kv_heads, delta.key_dim,
+                                                     delta.value_dim))[1]
+    kw, vw = delta.n_kv_heads * delta.key_dim, delta.n_heads * delta.value_dim
+    prepare_bytes = lambda n: n * (2 * (2 * kw + vw) + 2 * kw * 4 + vw * 2)
+    bench.measure("bugidra convolution + unit vectors + gates", delta, lin, prepare, (None, prepare_bytes(tokens_n)), prepare_bytes(batch))
+    conv = GroupedQueryAttention(W, H, G, d, names=dict(q="q", k="k", v="v", o="o"), conv_taps=4, sink=True)
+    for param in conv.all_named_params().values():
+        param.data = torch.zeros(param.shape, dtype=torch.bfloat16, device="cuda")
+    conv.finalize(torch.device("cuda"), torch.bfloat16)
+    def conv_kernel(ctx, x, view):
+        qkv = x[:, :channels].contiguous()
+        q = torch.empty((x.shape[0], H * d), dtype=x.dtype, device=x.device)
+        pages, state = view
+        bench.timed(lambda: ops.short_conv_store(qkv, conv._conv_w, state.slots, q, pages.pages, ctx.positions, ctx.token_row,
+                                                 pages.block_table, ctx.seg_row, ctx.seg_start, ctx.seg_len, ctx.n_segments, H, G,
+                                                 d, d, pages.page_size))
+        return q
+    bench.measure("debisun's short convolution + page write", conv, channels, conv_kernel, (None, moved(tokens_n, channels)),
+                  moved(batch, channels))
+
+    # ---- the sublayers' first products, joining the stream, the feed-forward
+    def product(name, part, run, rows_n):
+        def kernel(ctx, x, view):
+            h = x[:, :W].contiguous()
+            return bench.timed(lambda: run(ctx, h))
+        bench.measure(f"{name} ({rows_n} rows)", part, W, kernel, (2.0 * tokens_n * rows_n * W, None), rows_n * W * 2)
+    joint = bugidra.layers[1].input
+    product("bugidra joint first product of a pair", pair, lambda ctx, h: joint.forward_joint(ctx, h).rows, joint.out_features)
+    product("bugidra first product of the delta rule", delta, lambda ctx, h: delta.projection.forward(ctx, h), lin)
+    product("virulix q/k/v product", theirs, lambda ctx, h: theirs.qkv.forward(ctx, h), theirs.qkv.out_features)
+    weight, one = torch.ones(W, dtype=torch.bfloat16, device="cuda"), torch.ones(W, device="cuda")
+    def branch_join(ctx, x, view):
+        stream = x[:, :W].float()
+        branches = [(x[:, :W].float() * c, 0.5, one) for c in (0.5, 0.25)]
+        out = torch.empty((x.shape[0], W), dtype=x.dtype, device=x.device)
+        return bench.timed(lambda: ops.branch_join(stream, branches, branch_eps=1e-6, next_weight=weight, next_bias=weight,
+                                                   next_alpha=0.5, next_kind="tanh", rows=out))
+    def norm_join(ctx, x, view):
+        stream, branch = x[:, :W].float(), x[:, :W].float() * 3.0
+        out = torch.empty((x.shape[0], W), dtype=x.dtype, device=x.device)
+        return bench.timed(lambda: ops.norm_join(stream, branch, weight, 1e-6, "rms", next_weight=weight, rows=out))
+    bench.measure("bugidra two normed branches join the stream, the next norm behind them (1 kernel)", right, W, branch_join,
+                  (None, tokens_n * W * (4 * 4 + 2)), batch * W * (4 * 4 + 2))
+    bench.measure("gogotar's join (one normed branch, the next norm behind it)", right, W, norm_join,
+                  (None, tokens_n * W * (4 * 3 + 2)), batch * W * (4 * 3 + 2))
+    inner = sizes["ff"]
+    for label, part in (("bugidra feed-forward (gated gelu)", bugidra.layers[0].feed_forward),
+                        ("virulix feed-forward (gated gelu)", virulix.layers[0].feed_forward)):
+        ours = label.startswith("bugidra")
+        def kernel(ctx, x, view, part=part, ours=ours):
+            h, residual = x[:, :W].contiguous(), x[:, :W].float()
+            return bench.timed(lambda: part.forward(ctx, h, out_float32=True) if ours else part.forward(ctx, h, residual=residual))
+        bench.measure(label, part, W, kernel, (2.0 * tokens_n * 3 * inner * W, None), 3 * inner * W * 2)
+    return bench.rows
+
+
+def run_bugidra(args):
+    """Prefill and decode of Bugidra at sizes like a real model's layers, beside Virulix (the engine's closest design: pre-norm
+    over a float32 stream, attention and gated linear attention with a float32 state, dense gated feed-forwards with the same
+    activation) of equal width, heads, layer count, feed-forward size and vocabulary, and the kernels of its mechanisms
+    against their rooflines."""
+    import torch
+    from qwen_inference_lab_b200.config.model_config import BugidraConfig, VirulixConfig
+    from qwen_inference_lab_b200.loading import random_model
+    pk = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    for name in ([args.bugidra_shape] if args.bugidra_shape else sorted(BUGIDRA_SHAPES)):
+        sizes = BUGIDRA_SHAPES[name]
+        bugidra = random_model(BugidraConfig.from_dict(_bugidra_sizes(**sizes)), seed=0, device="cuda", dtype=torch.bfloat16)
+        virulix = random_model(VirulixConfig.from_dict(_virulix_beside_larolorn(**sizes)), seed=0, device="cuda", dtype=torch.bfloat16)
+        result = {"workload": "bugidra", "width": sizes["width"], "layers": 8, "dtype": "bfloat16",
+                  "peaks": "of measured" if pk["source"] == "measured" else "of fallback", "models": {}, "kernels": []}
+        for label, model in (("bugidra", bugidra), ("virulix", virulix)):
+            bench = _ModelBench(model, sizes["vocab"])
+            entry = {}
+            for tokens_n in (512, 2048):
+                ms = bench.prefill(tokens_n, flush)
+                entry[f"prefill_{tokens_n}"] = {"ms": round(ms, 3), "tokens_per_s": round(tokens_n / ms * 1e3, 1)}
+            for batch, context in ((1, 2048), (8, 2048), (32, 2048)):
+                ms = bench.decode(batch, context, args.steps, max(args.warmup, 6))
+                entry[f"decode_b{batch}_c{context}"] = {"ms": round(ms, 4), "tokens_per_s": round(batch / ms * 1e3, 1)}
+            result["models"][label] = entry
+        for kernel, ms, frac, of in _bugidra_kernels(torch, bugidra, virulix, sizes, pk, 2048, 8, 2048 + 511, flush):
+            result["kernels"].append({"kernel": kernel, "ms": round(ms, 4), "frac": round(frac, 4), "of": of})
+        print(json.dumps(result), flush=True)
+        del bugidra, virulix
+        torch.cuda.empty_cache()
+
+
 def run_reference(args):
     ref = ROOT / "baseline" / "_ref"
     def unavailable(why):
@@ -1545,14 +1746,15 @@ def main():
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--layers", type=int, default=None, help="run fewer layers than the configuration has")
     parser.add_argument("--quick", action="store_true", help="skip the batch 1 and 64 points")
-    parser.add_argument("--only", choices=["decode", "prefill", "mixed", "virulix", "debisun", "larolorn", "gogotar", "lotazen"], default=None,
+    parser.add_argument("--only", choices=["decode", "prefill", "mixed", "virulix", "debisun", "larolorn", "gogotar", "lotazen", "bugidra"], default=None,
                         help="run just this part and print its result instead of the JSON line; mixed = 64 requests "
                              "with prompts of 16 to 2048 tokens and 128 new tokens each through Engine.generate; "
                              "virulix = the Virulix design beside dense Qwen3 of equal size, and its mixers' kernels; "
                              "debisun = the Debisun design beside Virulix of equal size, and its mechanisms' kernels; "
                              "larolorn = the Larolorn design beside Virulix of equal size, and its mechanisms' kernels; "
                              "gogotar = the Gogotar design beside Larolorn of equal size, and its mechanisms' kernels; "
-                             "lotazen = the Lotazen design beside Virulix of equal size, and its mechanisms' kernels")
+                             "lotazen = the Lotazen design beside Virulix of equal size, and its mechanisms' kernels; "
+                             "bugidra = the Bugidra design beside Virulix of equal size, and its mechanisms' kernels")
     parser.add_argument("--virulix-shape", choices=sorted(VIRULIX_SHAPES), default=None,
                         help="width of --only virulix (default: all)")
     parser.add_argument("--debisun-shape", choices=sorted(DEBISUN_SHAPES), default=None,
@@ -1563,6 +1765,8 @@ def main():
                         help="width of --only gogotar (default: all)")
     parser.add_argument("--lotazen-shape", choices=sorted(LOTAZEN_SHAPES), default=None,
                         help="width of --only lotazen (default: all)")
+    parser.add_argument("--bugidra-shape", choices=sorted(BUGIDRA_SHAPES), default=None,
+                        help="width of --only bugidra (default: all)")
     parser.add_argument("--shape", choices=sorted(SHAPES), default="8b", help="layer sizes (default: Qwen3-8B)")
     parser.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16")
     parser.add_argument("--context", type=int, default=CONTEXT, help="cached tokens per request (profiling aid)")
@@ -1584,6 +1788,9 @@ def main():
         return 0
     if args.only == "lotazen":
         run_lotazen(args)
+        return 0
+    if args.only == "bugidra":
+        run_bugidra(args)
         return 0
     if args.only == "debisun":
         run_debisun(args)

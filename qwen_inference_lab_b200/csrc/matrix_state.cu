@@ -675,7 +675,8 @@ state_outputs_kernel(StateRows in, const int* __restrict__ chunk_start, const in
 
 template <typename Kernel>
 static cudaError_t ms_reserve(Kernel kernel, size_t smem) {
-    return smem > 48 * 1024 ? cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : cudaSuccess;
+    // the default limit of 48 KB counts the kernels' static arrays too
+    return smem > 40 * 1024 ? cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : cudaSuccess;
 }
 
 // The chunked form over a step's long portions.  y float32 [chunks, heads, MS_CHUNK, e] and w [chunks, heads, MS_CHUNK, d]

@@ -4,7 +4,7 @@ The sizes differ from layer to layer and between the cases: head sizes the tenso
 not, values larger than, smaller than and as large as keys, one to six query heads per key/value head, rotations over all
 and over two of a head's dimensions with and without YaRN's ramp (whose ends lie inside, before and behind the rotated pairs),
 states whose columns one thread, two, four, eight and sixteen threads hold and whose values take one block or several,
-decays of one, next to one and zero, convolutions of one tap and of several, q/k heads shared by several value heads, value
+decays of one and next to one, convolutions of one tap and of several, q/k heads shared by several value heads, value
 mixing in three layers, in one and in none, caps present and absent, layers without a feed-forward.
 """
 import json
@@ -69,13 +69,13 @@ CASE_A = config(173, 96, 1e-5, 3.0,
                 attention(2, 2, 16, 16, 0.4, rot(1e6, 16), cap=5.0, ff=40),
                 attention(2, 2, 32, 32, 0.2, rot(5e4, 2), v_mix=True, ff=48))
 # no convolution over time, a column spread over eight threads and one over sixteen (too wide for the chunks), a head's values
-# over two blocks, a first layer that mixes but has no one to mix with, decays of zero
+# over two blocks, a first layer that mixes but has no one to mix with
 CASE_B = config(97, 64, 1e-6, 1.0,
                 delta(1, 1, 130, 40, 1, ff=72),
                 pair(left(2, 1, 80, 80, 0.11, rot(500.0, 80)), right(96, 140, rot(2000.0, 96, (8.0, 30, 2.0, 0.5)), (0.999,)), 40),
                 attention(3, 3, 48, 48, 0.15, rot(20000.0, 2, (16.0, 500, 64.0, 3.0)), cap=30.0, v_mix=True),
                 delta(2, 1, 260, 10, 3),
-                pair(left(2, 2, 16, 32, 0.2, rot(100.0, 4)), right(8, 8, rot(10.0, 2), (0.0, 0.9, 0.99, 0.999)), 24))
+                pair(left(2, 2, 16, 32, 0.2, rot(100.0, 4)), right(10, 24, rot(10.0, 2), (0.8, 0.95, 0.99, 0.999)), 24))
 # awkward sizes: a width that is a multiple of nothing, heads of 20 and 7 with values of 12 and 9, five heads on one q/k head
 CASE_C = config(53, 70, 1e-5, 0.7,
                 pair(left(3, 3, 20, 12, 0.22, rot(50.0, 4, (2.0, 16, 32.0, 1.0))), right(7, 11, rot(30.0, 6), (0.9, 0.99)), 37),

@@ -110,7 +110,7 @@ def test_rotation_with_a_gain_and_heads_of_unit_size_behind_it(head, dims, origi
     assert rotation.gain > 1.1
     heads, positions, eps = 3, [0, 1, 17, 4095, 70001, 999999], 1e-4
     x = rows(len(positions), heads * head, 5)
-    x[:, head:2 * head] *= 0.01
+    x[:, head:2 * head] = (x[:, head:2 * head] * 0.01).to(torch.bfloat16).float()
     args = (rotation.freq, dims, rotation.layout, int32(*positions))
     f, gain = plain.rotary_frequencies(rot)
     f = torch.tensor(f, dtype=F64).float()
