@@ -18,10 +18,11 @@
 // so with A the strictly lower matrix of those coefficients, U = (I + A)^-1 diag(beta) V and
 // W = (I + A)^-1 diag(beta e^L) K (delta_solve, all chunks at once: forward substitution, a thread per column),
 //
-//   Y = U - W S            (plain: Y = V)                                    state_walk: the chunks of a portion in order,
-//   S' = e^(L_C) S + sum_j e^(L_C - L_j) k_j y_j^T                           a block per (head, 16 value columns)
+//   Y = U - W S            (plain: Y = V)                                    delta_walk: the chunks of a portion in order,
+//   S' = e^(L_C) S + sum_j e^(L_C - L_j) k_j y_j^T                           a block per (head, a few value columns)
 //   o_i = e^(L_i) S^T q_i + sum_{j <= i} e^(L_i - L_j) (q_i . k_j) y_j       state_outputs: all chunks at once
 //
+// Without the correction the sums of S' need no S: state_own makes them for all chunks at once and gla_carry walks them.
 // Every exponential is of a difference of sums kept in double precision and is at most one.  Chunks round differently from
 // the walk by token, in the last bits.
 #include "common.cuh"
@@ -296,7 +297,6 @@ __device__ __forceinline__ void ms_load_rows(float* dst, int stride, const float
 }
 
 __host__ __device__ __forceinline__ int ms_padded(int d) { return (d + 15) / 16 * 16; }
-__host__ __device__ __forceinline__ int ms_walk_stride(int dp) { return dp % 32 == 16 ? dp : dp + 16; }    // 16 banks from row to row
 
 // The 16 x 16 threads of a block hold X Y^T of two tiles of MS_CHUNK rows: element (ty + 16 a, tx + 16 b) in acc[a][b], b <= a
 // only (what lies above the diagonal is not asked for).
@@ -324,19 +324,72 @@ __device__ __forceinline__ void ms_lower_products(const float* x, const float* y
 }
 
 #define MS_A_STRIDE 68
-// One block per (head, chunk): U [MS_CHUNK, e] and W [MS_CHUNK, d] of the chunk (see the top), rows past its end zero.
+#define MS_DECAY_STRIDE 68       // of a (chunk, head): MS_CHUNK decays to the chunk's end, then the whole chunk's
+
+// The decays of a chunk from every token to its end, and over all of it (one warp; sums as chunk_log_sums leaves them).
+__device__ __forceinline__ void chunk_tail_decays(const double* sums, float* dst, int lane) {
+    const double last = sums[MS_CHUNK - 1];
+    for (int i = lane; i < MS_CHUNK; i += 32) dst[i] = expf((float)(last - sums[i]));
+    if (lane == 0) dst[MS_CHUNK] = expf((float)last);
+}
+
+// (I + A)^-1 of a strictly lower A [MS_CHUNK][MS_A_STRIDE] into t (lower, zero above): the diagonal blocks of 16 by forward
+// substitution, a thread per column, then blocks of 32 and of 64 from their halves, [X 0; Y Z]^-1 = [X' 0; -Z' Y X' Z'].
+// tmp holds a third such tile.  All 256 threads; barriers inside and at the end.
+__device__ __forceinline__ void invert_unit_lower(const float* a, float* t, float* tmp, int tid) {
+    for (int i = tid; i < MS_CHUNK * MS_A_STRIDE; i += 256) t[i] = 0.f;
+    __syncthreads();
+    if (tid < MS_CHUNK) {
+        const int base = tid / 16 * 16, col = tid % 16;
+        float x[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            float s = i == col ? 1.f : 0.f;
+#pragma unroll
+            for (int j = 0; j < i; ++j) s = fmaf(-a[(base + i) * MS_A_STRIDE + base + j], x[j], s);
+            x[i] = s;
+            t[(base + i) * MS_A_STRIDE + base + col] = s;
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int half = 16; half < MS_CHUNK; half *= 2) {
+        const int each = half * half;
+        for (int step = 0; step < 2; ++step) {                  // tmp = Y X', then -Z' tmp
+            for (int o = tid; o < MS_CHUNK / (2 * half) * each; o += 256) {
+                const int base = o / each * 2 * half, i = o % each / half, j = o % half;
+                const float* left = step == 0 ? a + (base + half + i) * MS_A_STRIDE + base : t + (base + half + i) * MS_A_STRIDE + base + half;
+                const float* right = step == 0 ? t + base * MS_A_STRIDE + base + j : tmp + (base + half) * MS_A_STRIDE + base + j;
+                float s0 = 0.f, s1 = 0.f;
+                for (int c = 0; c < half; c += 2) {
+                    s0 = fmaf(left[c], right[c * MS_A_STRIDE], s0);
+                    s1 = fmaf(left[c + 1], right[(c + 1) * MS_A_STRIDE], s1);
+                }
+                if (step == 0) tmp[(base + half + i) * MS_A_STRIDE + base + j] = s0 + s1;
+                else t[(base + half + i) * MS_A_STRIDE + base + j] = -(s0 + s1);
+            }
+            __syncthreads();
+        }
+    }
+}
+
+// One block per (head, chunk): U [MS_CHUNK, e] and W [MS_CHUNK, d] of the chunk (see the top), rows past its end zero, and the
+// decays to the chunk's end.
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 delta_solve_kernel(StateRows in, const int* __restrict__ chunk_start, const int* __restrict__ chunk_len, int n_heads, int d, int e,
-                   float* __restrict__ u_out, float* __restrict__ w_out) {
+                   float* __restrict__ u_out, float* __restrict__ w_out, float* __restrict__ decays) {
     extern __shared__ __align__(16) float smem[];
     __shared__ double sums[MS_CHUNK];
     __shared__ float beta[MS_CHUNK], beta_decay[MS_CHUNK];
     const int dp = ms_padded(d), stride = dp + 4;
     float* sk = smem;                           // [MS_CHUNK][stride]
-    float* sa = sk + MS_CHUNK * stride;         // [MS_CHUNK][MS_A_STRIDE]
+    float* sa = sk + MS_CHUNK * stride;         // [MS_CHUNK][MS_A_STRIDE]: A
+    float* st = sa + MS_CHUNK * MS_A_STRIDE;    // the same: its inverse
+    float* sv = st + MS_CHUNK * MS_A_STRIDE;    // the same: scratch, then 64 columns of values
     const int head = blockIdx.x, chunk = blockIdx.y, tid = threadIdx.x;
     const int first = chunk_start[chunk], count = chunk_len[chunk];
+    const size_t block = (size_t)chunk * n_heads + head;
     qil_wait_for_producer();
     qil_release_consumer();
     ms_load_rows(sk, stride, in.k + (size_t)first * in.qk_ld + (size_t)(head / in.group) * d, in.qk_ld, count, d, dp, true, tid, 256);
@@ -348,10 +401,12 @@ delta_solve_kernel(StateRows in, const int* __restrict__ chunk_start, const int*
         const float b = tid < count ? in.beta[(size_t)(first + tid) * n_heads + head] : 0.f;
         beta[tid] = b;
         beta_decay[tid] = b * expf((float)sums[tid]);
+    } else if (tid >= 224) {
+        chunk_tail_decays(sums, decays + block * MS_DECAY_STRIDE, tid & 31);
     }
     __syncthreads();
+    const int ty = tid >> 4, tx = tid & 15;
     {
-        const int ty = tid >> 4, tx = tid & 15;
         float acc[4][4];
         ms_lower_products(sk, sk, stride, dp, ty, tx, acc);
 #pragma unroll
@@ -363,191 +418,310 @@ delta_solve_kernel(StateRows in, const int* __restrict__ chunk_start, const int*
             }
     }
     __syncthreads();
+    invert_unit_lower(sa, st, sv, tid);
+    for (int i = tid; i < MS_CHUNK * dp; i += 256) sk[i / dp * stride + i % dp] *= beta_decay[i / dp];      // the keys' right side
     const T* v = reinterpret_cast<const T*>(in.v);
-    const size_t block = (size_t)chunk * n_heads + head;
-    for (int column = tid; column < e + d; column += 256) {
-        const bool is_value = column < e;
-        const int c = is_value ? column : column - e;
-        float x[MS_CHUNK];
-        const T* from = v + (size_t)first * in.v_ld + (size_t)head * e + c;
-#pragma unroll
-        for (int i = 0; i < MS_CHUNK; ++i) {      // the right side first: its loads are all under way before the chain begins
-            if (is_value) x[i] = i < count ? beta[i] * to_f32<T>(*from) : 0.f;
-            else x[i] = beta_decay[i] * sk[i * stride + c];
-            from += in.v_ld;
-        }
-        float* dst = is_value ? u_out + block * MS_CHUNK * e + c : w_out + block * MS_CHUNK * d + c;
-        const int pitch = is_value ? e : d;
-#pragma unroll
-        for (int i = 0; i < MS_CHUNK; ++i) {
-            float s0 = x[i], s1 = 0.f, s2 = 0.f, s3 = 0.f;
-#pragma unroll
-            for (int j = 0; j < i; j += 4) {       // entries at and past the diagonal are zero
-                const float4 a = *reinterpret_cast<const float4*>(sa + i * MS_A_STRIDE + j);
-                s0 = fmaf(-a.x, x[j], s0);
-                if (j + 1 < i) s1 = fmaf(-a.y, x[j + 1], s1);
-                if (j + 2 < i) s2 = fmaf(-a.z, x[j + 2], s2);
-                if (j + 3 < i) s3 = fmaf(-a.w, x[j + 3], s3);
+    for (int tile = 0; tile < (e + 63) / 64 + (d + 63) / 64; ++tile) {
+        const bool is_value = tile < (e + 63) / 64;
+        const int col0 = (is_value ? tile : tile - (e + 63) / 64) * 64, width = is_value ? e : d;
+        if (is_value) {
+            __syncthreads();            // the tile before has been read
+            for (int i = tid; i < MS_CHUNK * 64; i += 256) {
+                const int r = i / 64, c = col0 + i % 64;
+                sv[r * MS_A_STRIDE + i % 64] = (r < count && c < e)
+                    ? beta[r] * to_f32<T>(v[(size_t)(first + r) * in.v_ld + (size_t)head * e + c]) : 0.f;
             }
-            x[i] = (s0 + s1) + (s2 + s3);
-            *dst = x[i];
-            dst += pitch;
+        }
+        __syncthreads();
+        const float* right = is_value ? sv + 4 * tx : sk + col0 + 4 * tx;
+        const int right_stride = is_value ? MS_A_STRIDE : stride;
+        const bool real = is_value || col0 + 4 * tx < dp;
+        float acc[4][4];
+#pragma unroll
+        for (int a = 0; a < 4; ++a)
+#pragma unroll
+            for (int b = 0; b < 4; ++b) acc[a][b] = 0.f;
+#pragma unroll
+        for (int jb = 0; jb < 4; ++jb)         // rows of block a read columns of blocks up to a
+#pragma unroll 2
+            for (int c = 16 * jb; c < 16 * jb + 16 && real; c += 4) {
+                float4 xv[4];
+#pragma unroll
+                for (int a = jb; a < 4; ++a) xv[a] = *reinterpret_cast<const float4*>(st + (ty + 16 * a) * MS_A_STRIDE + c);
+#pragma unroll
+                for (int r = 0; r < 4; ++r) {
+                    const float4 b = *reinterpret_cast<const float4*>(right + (c + r) * right_stride);
+#pragma unroll
+                    for (int a = jb; a < 4; ++a) {
+                        const float x = r == 0 ? xv[a].x : r == 1 ? xv[a].y : r == 2 ? xv[a].z : xv[a].w;
+                        acc[a][0] = fmaf(x, b.x, acc[a][0]); acc[a][1] = fmaf(x, b.y, acc[a][1]);
+                        acc[a][2] = fmaf(x, b.z, acc[a][2]); acc[a][3] = fmaf(x, b.w, acc[a][3]);
+                    }
+                }
+            }
+        float* dst = (is_value ? u_out : w_out) + block * MS_CHUNK * width + col0 + 4 * tx;
+#pragma unroll
+        for (int a = 0; a < 4; ++a) {
+            float* at = dst + (size_t)(ty + 16 * a) * width;
+            if (width % 4 == 0 && col0 + 4 * tx + 3 < width) {
+                *reinterpret_cast<float4*>(at) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+            } else {
+#pragma unroll
+                for (int b = 0; b < 4; ++b) if (col0 + 4 * tx + b < width) at[b] = acc[a][b];
+            }
         }
     }
 }
 
 // ------------------------------------------------------------------ the chunks of a portion in order
-// One block per (head, MS_COLS value columns, long portion).  carry: int32 [portions, 3] = (state slot, first chunk, chunks).
+// Sums of 16 values over LANES neighbouring lanes; lane l of them keeps values l * 16 / LANES and following, at the front.
+template <int LANES>
+__device__ __forceinline__ void scatter_sums(float (&v)[16], int lane) {
+    int n = 16;
+#pragma unroll
+    for (int step = LANES / 2; step > 0; step >>= 1) {
+        n >>= 1;
+        const bool upper = (lane & step) != 0;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            if (i >= n) break;
+            const float other = __shfl_xor_sync(0xffffffffu, upper ? v[i] : v[i + n], step);
+            v[i] = (upper ? v[i + n] : v[i]) + other;
+        }
+    }
+}
+
+// One block per (head, COLS value columns, long portion).  carry: int32 [portions, 3] = (state slot, first chunk, chunks).
 // chunk_state [chunks, heads, d, e] receives the state that comes into every chunk, y [chunks, heads, MS_CHUNK, e] the
-// corrected values (DELTA: in place of u); the state after the last chunk goes to the request's slot.
-#define MS_COLS 16
-template <typename T, bool DELTA>
+// corrected values in place of u; the state after the last chunk goes to the request's slot.  The state's columns live in
+// registers, with a copy in shared memory for the first product.  ITEMS: of 128 key channels that a thread serves.
+template <int COLS, int ITEMS>
 __global__ void __launch_bounds__(256, 1)
-state_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* __restrict__ chunk_len, const int* __restrict__ carry,
-                  int n_heads, int d, int e, float* __restrict__ y, const float* __restrict__ w_in, float* __restrict__ chunk_state,
-                  float* __restrict__ slots, int stages) {
+delta_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* __restrict__ chunk_len, const int* __restrict__ carry,
+                  int n_heads, int d, int e, float* __restrict__ y, const float* __restrict__ w_in, const float* __restrict__ decays,
+                  float* __restrict__ chunk_state, float* __restrict__ slots, int stages) {
+    constexpr int CG = COLS / 4;           // groups of four columns
+    constexpr int KS = 16 / CG;            // lanes that share 4 x 4 elements of the first product, each over a part of the channels
+    constexpr int TS = 8 / CG;             // the same for the second product, over the tokens
+    constexpr int KEEP = 16 / KS, HOLD = 16 / TS;
     extern __shared__ __align__(16) float smem[];
-    __shared__ double sums[MS_CHUNK];
-    __shared__ float tail_decay[MS_CHUNK];
-    __shared__ __align__(16) float sy[MS_CHUNK * MS_COLS];       // y times its decay to the chunk's end
-    const int dp = ms_padded(d), stride = ms_walk_stride(dp), tile = MS_CHUNK * stride;
+    const int dp = (d + 31) / 32 * 32, stride = dp + 16, state_stride = dp + 4, tile = MS_CHUNK * stride;
     float* sk = smem;                                  // [stages][MS_CHUNK][stride]
-    float* sw = sk + stages * tile;                    // the same, with the correction
-    float* ss = sw + (DELTA ? stages * tile : 0);      // [MS_COLS][stride]: the state's columns
-    const int tiles = (e + MS_COLS - 1) / MS_COLS;
-    const int head = blockIdx.x / tiles, col0 = (blockIdx.x % tiles) * MS_COLS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    float* sw = sk + stages * tile;                    // the same
+    float* ss = sw + stages * tile;                    // [COLS][state_stride]
+    float* sy = ss + COLS * state_stride;              // [MS_CHUNK][COLS]: y times its decay to the chunk's end
+    float* sd = sy + MS_CHUNK * COLS;                  // [stages][MS_DECAY_STRIDE]
+    const int tiles = (e + COLS - 1) / COLS;
+    const int head = blockIdx.x / tiles, col0 = (blockIdx.x % tiles) * COLS, tid = threadIdx.x;
     const int row = carry[3 * blockIdx.y], chunk0 = carry[3 * blockIdx.y + 1], chunks = carry[3 * blockIdx.y + 2];
     const size_t qk_at = (size_t)(head / in.group) * d;
-    const T* v = reinterpret_cast<const T*>(in.v);
-    for (int i = tid; i < stages * tile * (DELTA ? 2 : 1) + MS_COLS * stride; i += 256) smem[i] = 0.f;      // the padding stays zero
+    const int total = stages * (2 * tile + MS_DECAY_STRIDE) + COLS * (state_stride + MS_CHUNK);
+    for (int i = tid; i < total; i += 256) smem[i] = 0.f;      // the padding stays zero
+    const int part = tid % KS, cg = tid / KS % CG, rg = tid / KS / CG;                  // first product: rows rg + 16 a
+    const int my_row = rg + 16 * (part * KEEP / 4), my_col = 4 * cg + part * KEEP % 4;  // of the sums this thread keeps
+    const int ts = tid % TS, gc = tid / TS % CG, d_first = tid / TS / CG * 4;           // second product: channels d_first + 128 it
+    const int hold_d = ts * HOLD / 4;                                                   // of the sums this thread keeps: HOLD / 4 channels
+    const bool aligned = e % 4 == 0 && col0 + COLS <= e;
     qil_wait_for_producer();
     qil_release_consumer();
     __syncthreads();
-    float* slot = slots + ((size_t)row * n_heads + head) * d * e;
-    for (int i = tid; i < d * MS_COLS; i += 256) {
-        const int dd = i / MS_COLS, c = i % MS_COLS;
-        if (col0 + c < e) ss[c * stride + dd] = slot[(size_t)dd * e + col0 + c];
-    }
+    float S[ITEMS][HOLD];
+    float* slot = slots + ((size_t)row * n_heads + head) * d * e + col0 + 4 * gc;
+#pragma unroll
+    for (int it = 0; it < ITEMS; ++it)
+#pragma unroll
+        for (int i = 0; i < HOLD; ++i) {
+            const int dd = d_first + 128 * it + hold_d + i / 4;
+            S[it][i] = (dd < d && col0 + 4 * gc + i % 4 < e) ? slot[(size_t)dd * e + i % 4] : 0.f;
+            if (dd < dp) ss[(4 * gc + i % 4) * state_stride + dd] = S[it][i];
+        }
     auto fetch = [&](int chunk, int stage) {
         const int first = chunk_start[chunk], count = chunk_len[chunk];
+        const size_t block = (size_t)chunk * n_heads + head;
         ms_load_rows(sk + stage * tile, stride, in.k + (size_t)first * in.qk_ld + qk_at, in.qk_ld, count, d, dp, false, tid, 256);
-        if (DELTA) ms_load_rows(sw + stage * tile, stride, w_in + ((size_t)chunk * n_heads + head) * MS_CHUNK * d, d, MS_CHUNK, d, dp,
-                                false, tid, 256);
+        ms_load_rows(sw + stage * tile, stride, w_in + block * MS_CHUNK * d, d, MS_CHUNK, d, dp, false, tid, 256);
+        if (tid < MS_DECAY_STRIDE / 4) ms_copy16(sd + stage * MS_DECAY_STRIDE + 4 * tid, decays + block * MS_DECAY_STRIDE + 4 * tid, true);
+        ms_commit();
     };
-    // The first product: 64 rows x 16 columns, contracted over the channels.  Four neighbouring lanes share 4 x 4 elements
-    // (rows rg + 16 a, columns cg + 4 b), each over a quarter of the channels, and keep column cg + 4 part of the sum.
-    const int part = lane & 3, cg = (lane >> 2) & 3, rg = warp * 2 + (lane >> 4);
-    const int my_col = col0 + cg + 4 * part;
-    auto values_of = [&](int chunk, float (&u)[4]) {
-        const int first = chunk_start[chunk], count = chunk_len[chunk];
+    auto at_y = [&](int chunk) { return y + (((size_t)chunk * n_heads + head) * MS_CHUNK + my_row) * e + col0 + my_col; };
+    auto read_u = [&](int chunk, float (&u)[KEEP]) {
+        const float* p = at_y(chunk);
+        if (aligned && KEEP == 4) {
+            const float4 q = *reinterpret_cast<const float4*>(p);
+            u[0] = q.x; u[1 % KEEP] = q.y; u[2 % KEEP] = q.z; u[3 % KEEP] = q.w;
+        } else if (aligned && KEEP == 2) {
+            const float2 q = *reinterpret_cast<const float2*>(p);
+            u[0] = q.x; u[1 % KEEP] = q.y;
+        } else {
 #pragma unroll
-        for (int a = 0; a < 4; ++a) {
-            const int i = rg + 16 * a;
-            u[a] = 0.f;
-            if (my_col < e && i < count)
-                u[a] = DELTA ? y[(((size_t)chunk * n_heads + head) * MS_CHUNK + i) * e + my_col]
-                             : to_f32<T>(v[(size_t)(first + i) * in.v_ld + (size_t)head * e + my_col]);
+            for (int i = 0; i < KEEP; ++i) u[i] = col0 + my_col + i < e ? p[i] : 0.f;
         }
     };
-    float u[4];
-    values_of(chunk0, u);
-    if (stages == 2) { fetch(chunk0, 0); ms_commit(); }
+    float u[KEEP];
+    read_u(chunk0, u);
+    if (stages == 2) fetch(chunk0, 0);
     for (int n = 0; n < chunks; ++n) {
         const int chunk = chunk0 + n, stage = stages == 2 ? (n & 1) : 0;
-        if (stages == 2) {
-            if (n + 1 < chunks) fetch(chunk + 1, stage ^ 1);
-            ms_commit();
-        } else {
-            fetch(chunk, 0);
-            ms_commit();
-        }
-        if (warp == 0) {
-            chunk_log_sums(in, sums, chunk_start[chunk], chunk_len[chunk], head, n_heads, lane);
-            __syncwarp();
-            const double last = sums[MS_CHUNK - 1];
-            for (int i = lane; i < MS_CHUNK; i += 32) tail_decay[i] = expf((float)(last - sums[i]));
-        }
-        if (stages == 2) ms_wait<1>(); else ms_wait<0>();
-        __syncthreads();
+        if (stages == 1) fetch(chunk, 0);
+        ms_wait<0>();
+        __syncthreads();                   // this chunk's tiles are here, everyone has left the chunk before
+        if (stages == 2 && n + 1 < chunks) fetch(chunk + 1, stage ^ 1);
         const float* tk = sk + stage * tile;
-        const size_t block = (size_t)chunk * n_heads + head;
-        for (int i = tid; i < d * MS_COLS; i += 256) {
-            const int dd = i / MS_COLS, c = i % MS_COLS;
-            if (col0 + c < e) chunk_state[(block * d + dd) * e + col0 + c] = ss[c * stride + dd];
-        }
-        if (DELTA) {
-            const float* tw = sw + stage * tile;
-            float acc[4][4];
+        const float* tw = sw + stage * tile;
+        const float* tail = sd + stage * MS_DECAY_STRIDE;
+        float* into = chunk_state + ((size_t)chunk * n_heads + head) * d * e + col0 + 4 * gc;
 #pragma unroll
-            for (int a = 0; a < 4; ++a)
+        for (int it = 0; it < ITEMS; ++it)
 #pragma unroll
-                for (int b = 0; b < 4; ++b) acc[a][b] = 0.f;
-            for (int c = part * 4; c < dp; c += 16) {
+            for (int i = 0; i < HOLD; i += 4) {
+                const int dd = d_first + 128 * it + hold_d + i / 4;
+                if (dd >= d) continue;
+                if (aligned) {
+                    *reinterpret_cast<float4*>(into + (size_t)dd * e) = make_float4(S[it][i], S[it][i + 1], S[it][i + 2], S[it][i + 3]);
+                } else {
+#pragma unroll
+                    for (int b = 0; b < 4; ++b) if (col0 + 4 * gc + b < e) into[(size_t)dd * e + b] = S[it][i + b];
+                }
+            }
+        {
+            float acc[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i) acc[i] = 0.f;
+#pragma unroll 2
+            for (int c = part * 4; c < dp; c += 4 * KS) {
                 float4 wv[4], sv[4];
 #pragma unroll
                 for (int a = 0; a < 4; ++a) {
                     wv[a] = *reinterpret_cast<const float4*>(tw + (rg + 16 * a) * stride + c);
-                    sv[a] = *reinterpret_cast<const float4*>(ss + (cg + 4 * a) * stride + c);
+                    sv[a] = *reinterpret_cast<const float4*>(ss + (4 * cg + a) * state_stride + c);
                 }
 #pragma unroll
                 for (int a = 0; a < 4; ++a)
 #pragma unroll
                     for (int b = 0; b < 4; ++b) {
-                        acc[a][b] = fmaf(wv[a].x, sv[b].x, acc[a][b]); acc[a][b] = fmaf(wv[a].y, sv[b].y, acc[a][b]);
-                        acc[a][b] = fmaf(wv[a].z, sv[b].z, acc[a][b]); acc[a][b] = fmaf(wv[a].w, sv[b].w, acc[a][b]);
+                        acc[4 * a + b] = fmaf(wv[a].x, sv[b].x, acc[4 * a + b]); acc[4 * a + b] = fmaf(wv[a].y, sv[b].y, acc[4 * a + b]);
+                        acc[4 * a + b] = fmaf(wv[a].z, sv[b].z, acc[4 * a + b]); acc[4 * a + b] = fmaf(wv[a].w, sv[b].w, acc[4 * a + b]);
                     }
             }
+            scatter_sums<KS>(acc, part);
+            const float decay = tail[my_row];
+            float* p = at_y(chunk);
 #pragma unroll
-            for (int a = 0; a < 4; ++a) {
-                // lanes 0, 1 of the four keep columns b = 0, 1, lanes 2, 3 columns 2, 3; then one column each
-                const bool upper = part & 2, odd = part & 1;
-                const float x0 = __shfl_xor_sync(0xffffffffu, upper ? acc[a][0] : acc[a][2], 2);
-                const float x1 = __shfl_xor_sync(0xffffffffu, upper ? acc[a][1] : acc[a][3], 2);
-                const float k0 = (upper ? acc[a][2] : acc[a][0]) + x0, k1 = (upper ? acc[a][3] : acc[a][1]) + x1;
-                const float z = __shfl_xor_sync(0xffffffffu, odd ? k0 : k1, 1);
-                u[a] -= (odd ? k1 : k0) + z;
-                const int i = rg + 16 * a;
-                if (my_col < e) y[(block * MS_CHUNK + i) * e + my_col] = u[a];
+            for (int i = 0; i < KEEP; ++i) {
+                u[i] -= acc[i];
+                sy[my_row * COLS + my_col + i] = u[i] * decay;
             }
+            if (aligned && KEEP == 4) {
+                *reinterpret_cast<float4*>(p) = make_float4(u[0], u[1 % KEEP], u[2 % KEEP], u[3 % KEEP]);
+            } else if (aligned && KEEP == 2) {
+                *reinterpret_cast<float2*>(p) = make_float2(u[0], u[1 % KEEP]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < KEEP; ++i) if (col0 + my_col + i < e) p[i] = u[i];
+            }
+            if (n + 1 < chunks) read_u(chunk + 1, u);
         }
+        const float whole = tail[MS_CHUNK];
+        __syncthreads();                   // y is here, everyone has read the state's columns
 #pragma unroll
-        for (int a = 0; a < 4; ++a) sy[(rg + 16 * a) * MS_COLS + cg + 4 * part] = u[a] * tail_decay[rg + 16 * a];
-        if (n + 1 < chunks) values_of(chunk + 1, u);
-        const float whole = expf((float)sums[MS_CHUNK - 1]);
-        __syncthreads();
-        // The second product: d channels x 16 columns, contracted over the tokens: two neighbouring lanes share 4 x 4 elements,
-        // one over the even tokens, one over the odd ones, and keep two columns each.
-        const int half = tid & 1, gc = (tid >> 1) & 3;
-        for (int d4 = (tid >> 3) * 4; d4 < dp; d4 += 128) {      // dp is a multiple of 16: whole warps leave together
-            float acc[4][4];
+        for (int it = 0; it < ITEMS; ++it) {
+            const int d4 = d_first + 128 * it;
+            if (d4 >= dp) break;           // dp is a multiple of 32: whole warps leave together
+            float acc[16];
 #pragma unroll
-            for (int a = 0; a < 4; ++a)
-#pragma unroll
-                for (int b = 0; b < 4; ++b) acc[a][b] = 0.f;
+            for (int i = 0; i < 16; ++i) acc[i] = 0.f;
 #pragma unroll 4
-            for (int t = half; t < MS_CHUNK; t += 2) {
+            for (int t = ts; t < MS_CHUNK; t += TS) {
                 const float4 kv = *reinterpret_cast<const float4*>(tk + t * stride + d4);
-                const float4 yv = *reinterpret_cast<const float4*>(sy + t * MS_COLS + 4 * gc);
+                const float4 yv = *reinterpret_cast<const float4*>(sy + t * COLS + 4 * gc);
                 const float ka[4] = {kv.x, kv.y, kv.z, kv.w}, ya[4] = {yv.x, yv.y, yv.z, yv.w};
 #pragma unroll
                 for (int a = 0; a < 4; ++a)
 #pragma unroll
-                    for (int b = 0; b < 4; ++b) acc[a][b] = fmaf(ka[a], ya[b], acc[a][b]);
+                    for (int b = 0; b < 4; ++b) acc[4 * a + b] = fmaf(ka[a], ya[b], acc[4 * a + b]);
             }
+            scatter_sums<TS>(acc, ts);
 #pragma unroll
-            for (int a = 0; a < 4; ++a) {
-                const float x0 = __shfl_xor_sync(0xffffffffu, half ? acc[a][0] : acc[a][2], 1);
-                const float x1 = __shfl_xor_sync(0xffffffffu, half ? acc[a][1] : acc[a][3], 1);
-                float* s0 = ss + (4 * gc + 2 * half) * stride + d4 + a;
-                s0[0] = fmaf(whole, s0[0], (half ? acc[a][2] : acc[a][0]) + x0);
-                s0[stride] = fmaf(whole, s0[stride], (half ? acc[a][3] : acc[a][1]) + x1);
+            for (int i = 0; i < HOLD; ++i) {
+                S[it][i] = fmaf(whole, S[it][i], acc[i]);
+                ss[(4 * gc + i % 4) * state_stride + d4 + hold_d + i / 4] = S[it][i];
             }
         }
-        __syncthreads();
+        if (stages == 1) __syncthreads();  // the tiles are overwritten next
     }
-    for (int i = tid; i < d * MS_COLS; i += 256) {
-        const int dd = i / MS_COLS, c = i % MS_COLS;
-        if (col0 + c < e) slot[(size_t)dd * e + col0 + c] = ss[c * stride + dd];
+#pragma unroll
+    for (int it = 0; it < ITEMS; ++it)
+#pragma unroll
+        for (int i = 0; i < HOLD; ++i) {
+            const int dd = d_first + 128 * it + hold_d + i / 4;
+            if (dd < d && col0 + 4 * gc + i % 4 < e) slot[(size_t)dd * e + i % 4] = S[it][i];
+        }
+}
+
+// Without the correction a chunk's own state needs no state: sum_j e^(L_C - L_j) k_j v_j^T for all chunks at once (chunk_state
+// [chunks, heads, d, e]) and the chunk's decay for every channel (decay_product [chunks, heads, d]); gla_carry walks them.
+// One block per (head, chunk, 64 value columns).
+template <typename T>
+__global__ void __launch_bounds__(256)
+state_own_kernel(StateRows in, const int* __restrict__ chunk_start, const int* __restrict__ chunk_len, int n_heads, int d, int e,
+                 float* __restrict__ chunk_state, float* __restrict__ decay_product) {
+    extern __shared__ __align__(16) float smem[];
+    __shared__ double sums[MS_CHUNK];
+    __shared__ float tail[MS_DECAY_STRIDE];
+    const int dp = ms_padded(d), stride = dp + 4;
+    float* sk = smem;                           // [MS_CHUNK][stride]
+    float* sv = sk + MS_CHUNK * stride;         // [MS_CHUNK][MS_A_STRIDE]
+    const int head = blockIdx.x, chunk = blockIdx.y, col0 = blockIdx.z * 64, tid = threadIdx.x;
+    const int first = chunk_start[chunk], count = chunk_len[chunk];
+    const size_t block = (size_t)chunk * n_heads + head;
+    const T* v = reinterpret_cast<const T*>(in.v);
+    qil_wait_for_producer();
+    qil_release_consumer();
+    ms_load_rows(sk, stride, in.k + (size_t)first * in.qk_ld + (size_t)(head / in.group) * d, in.qk_ld, count, d, dp, true, tid, 256);
+    ms_commit();
+    if (tid < 32) {
+        chunk_log_sums(in, sums, first, count, head, n_heads, tid);
+        __syncwarp();
+        chunk_tail_decays(sums, tail, tid);
+    }
+    __syncthreads();
+    for (int i = tid; i < MS_CHUNK * 64; i += 256) {
+        const int r = i / 64, c = col0 + i % 64;
+        sv[r * MS_A_STRIDE + i % 64] = (r < count && c < e) ? tail[r] * to_f32<T>(v[(size_t)(first + r) * in.v_ld + (size_t)head * e + c]) : 0.f;
+    }
+    if (blockIdx.z == 0)
+        for (int i = tid; i < d; i += 256) decay_product[block * d + i] = tail[MS_CHUNK];
+    ms_wait<0>();
+    __syncthreads();
+    const int ty = tid >> 4, tx = tid & 15;
+    for (int d4 = 4 * ty; d4 < dp; d4 += 64) {
+        float acc[4][4];
+#pragma unroll
+        for (int a = 0; a < 4; ++a)
+#pragma unroll
+            for (int b = 0; b < 4; ++b) acc[a][b] = 0.f;
+#pragma unroll 8
+        for (int t = 0; t < MS_CHUNK; ++t) {
+            const float4 kv = *reinterpret_cast<const float4*>(sk + t * stride + d4);
+            const float4 yv = *reinterpret_cast<const float4*>(sv + t * MS_A_STRIDE + 4 * tx);
+            const float ka[4] = {kv.x, kv.y, kv.z, kv.w}, ya[4] = {yv.x, yv.y, yv.z, yv.w};
+#pragma unroll
+            for (int a = 0; a < 4; ++a)
+#pragma unroll
+                for (int b = 0; b < 4; ++b) acc[a][b] = fmaf(ka[a], ya[b], acc[a][b]);
+        }
+        const int c = col0 + 4 * tx;
+#pragma unroll
+        for (int a = 0; a < 4; ++a) {
+            if (d4 + a >= d) break;
+            float* dst = chunk_state + (block * d + d4 + a) * e + c;
+            if (e % 4 == 0 && c + 3 < e) {
+                *reinterpret_cast<float4*>(dst) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+            } else {
+#pragma unroll
+                for (int b = 0; b < 4; ++b) if (c + b < e) dst[b] = acc[a][b];
+            }
+        }
     }
 }
 
@@ -636,6 +810,7 @@ state_outputs_kernel(StateRows in, const int* __restrict__ chunk_start, const in
 #pragma unroll
             for (int b = 0; b < 4; ++b) acc[a][b] = 0.f;
         auto gather = [&](const float* left, int left_stride, const float* right, int depth) {
+#pragma unroll 2
             for (int c = 0; c < depth; c += 4) {
                 float4 xv[4];
 #pragma unroll
@@ -679,48 +854,83 @@ static cudaError_t ms_reserve(Kernel kernel, size_t smem) {
     return smem > 40 * 1024 ? cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : cudaSuccess;
 }
 
-// The chunked form over a step's long portions.  y float32 [chunks, heads, MS_CHUNK, e] and w [chunks, heads, MS_CHUNK, d]
-// (both for the correction only), chunk_state float32 [chunks, heads, d, e]: scratch.  o_raw float32 [tokens, heads * e]: the
-// outputs of the chunks' tokens, as they are.
+extern "C" int qil_gla_carry(float* chunk_state, const float* decay_product, float* slots, const int* carry, int n_carries,
+                             int n_heads, int d, int e, cudaStream_t stream);
+
+static size_t delta_walk_smem(int d, int cols, int stages) {
+    const int dp = (d + 31) / 32 * 32;
+    return (size_t)(stages * (2 * MS_CHUNK * (dp + 16) + MS_DECAY_STRIDE) + cols * (dp + 4 + MS_CHUNK)) * sizeof(float);
+}
+
+// Floats of scratch per (chunk, head) that qil_state_chunks wants beside the chunks' states: with the correction U, W and the
+// decays, without it a decay per channel.
+extern "C" int qil_state_chunk_scratch(int d, int e, int delta) {
+    return delta ? MS_CHUNK * (d + e) + MS_DECAY_STRIDE : d;
+}
+
+// The chunked form over a step's long portions.  scratch: float32 [chunks * heads * qil_state_chunk_scratch]; chunk_state float32
+// [chunks, heads, d, e]: scratch too.  o_raw float32 [tokens, heads * e]: the outputs of the chunks' tokens, as they are.
 extern "C" int qil_state_chunks(const float* q, const float* k, long long qk_ld, int group, const void* v, long long v_ld,
                                 const float* log_decay, const float* head_decay, const float* beta, const int* chunk_start,
                                 const int* chunk_len, int n_chunks, const int* carry, int n_carries, int n_heads, int d, int e,
-                                float* y, float* w, float* chunk_state, float* slots, float* o_raw, int act_dtype,
-                                cudaStream_t stream) {
+                                float* scratch, float* chunk_state, float* slots, float* o_raw, int act_dtype, cudaStream_t stream) {
     if (n_chunks <= 0) return 0;
     const StateRows in = {q, k, qk_ld, group, v, v_ld, log_decay, head_decay, beta};
     const bool delta = beta != nullptr;
     if (state_rows_check("state_chunks", in, n_heads, d, e, delta)) return -1;
     if (d > MS_MOST_D) QIL_REFUSE("state_chunks: %d key channels per head are more than %d", d, MS_MOST_D);
     if (n_chunks > 65535 || n_carries <= 0 || n_carries > 65535) QIL_REFUSE("state_chunks: %d chunks of %d portions", n_chunks, n_carries);
-    if (delta && (y == nullptr || w == nullptr)) QIL_REFUSE("state_chunks: the correction needs its scratch buffers");
-    const int dp = ms_padded(d), tiles = (e + MS_COLS - 1) / MS_COLS;
+    if (scratch == nullptr || ((uintptr_t)scratch & 15) != 0 || ((uintptr_t)chunk_state & 15) != 0)
+        QIL_REFUSE("state_chunks: scratch on 16-byte boundaries");
+    const int dp = ms_padded(d);
     const size_t row_tile = (size_t)MS_CHUNK * (dp + 4) * sizeof(float), a_tile = (size_t)MS_CHUNK * MS_A_STRIDE * sizeof(float);
-    const size_t walk_tile = (size_t)MS_CHUNK * ms_walk_stride(dp) * sizeof(float);
-    const size_t walk_state = (size_t)MS_COLS * ms_walk_stride(dp) * sizeof(float);
-    const int stages = 2 * walk_tile * (delta ? 2 : 1) + walk_state <= 200 * 1024 ? 2 : 1;
-    const size_t walk_smem = stages * walk_tile * (delta ? 2 : 1) + walk_state;
     const size_t after_keys = (size_t)(dp + MS_CHUNK) * MS_OUT_COLS * sizeof(float);
     const size_t out_smem = row_tile + a_tile + (row_tile > after_keys ? row_tile : after_keys);
+    const size_t pairs = (size_t)n_chunks * n_heads;
+    // the decays first: their stride is a multiple of four, so that all three parts can start on 16-byte boundaries
+    float* decays = scratch;
+    float* y = decays + (delta ? pairs * MS_DECAY_STRIDE : 0);
+    float* w = y + (delta ? pairs * MS_CHUNK * e : 0);
+    // few columns a block where that still leaves every block a multiprocessor of its own
+    const int cols = (long long)n_heads * ((e + 7) / 8) * n_carries <= 148 ? 8 : 16;
+    const int tiles = (e + cols - 1) / cols;
+    const int stages = delta_walk_smem(d, cols, 2) <= 200 * 1024 ? 2 : 1;
+    const size_t walk_smem = delta_walk_smem(d, cols, stages);
     cudaError_t err = cudaSuccess;
 #define QIL_MS(...) do { if (err == cudaSuccess) err = (__VA_ARGS__); } while (0)
-#define QIL_MS_WALK(DELTA)                                                                                              \
-    QIL_MS(ms_reserve(state_walk_kernel<T, DELTA>, walk_smem));                                                         \
-    QIL_MS(qil_launch_chained(state_walk_kernel<T, DELTA>, dim3(n_heads * tiles, n_carries), dim3(256), walk_smem, stream, in, \
-                              chunk_start, chunk_len, carry, n_heads, d, e, y, (const float*)w, chunk_state, slots, stages));  \
-    QIL_MS(ms_reserve(state_outputs_kernel<T, DELTA>, out_smem));                                                       \
-    QIL_MS(qil_launch_chained(state_outputs_kernel<T, DELTA>, dim3(n_heads, n_chunks), dim3(256), out_smem, stream, in, \
-                              chunk_start, chunk_len, n_heads, d, e, (const float*)y, (const float*)chunk_state, o_raw))
+#define QIL_MS_WALK(COLS, ITEMS)                                                                                        \
+    do {                                                                                                                \
+        QIL_MS(ms_reserve(delta_walk_kernel<COLS, ITEMS>, walk_smem));                                                  \
+        QIL_MS(qil_launch_chained(delta_walk_kernel<COLS, ITEMS>, dim3(n_heads * tiles, n_carries), dim3(256), walk_smem, stream, \
+                                  in, chunk_start, chunk_len, carry, n_heads, d, e, y, (const float*)w, (const float*)decays,     \
+                                  chunk_state, slots, stages));                                                         \
+    } while (0)
+#define QIL_MS_OUTPUTS(DELTA)                                                                                           \
+    do {                                                                                                                \
+        QIL_MS(ms_reserve(state_outputs_kernel<T, DELTA>, out_smem));                                                   \
+        QIL_MS(qil_launch_chained(state_outputs_kernel<T, DELTA>, dim3(n_heads, n_chunks), dim3(256), out_smem, stream, in, \
+                                  chunk_start, chunk_len, n_heads, d, e, (const float*)y, (const float*)chunk_state, o_raw)); \
+    } while (0)
     QIL_DISPATCH_1(act_dtype, {
         if (delta) {
-            QIL_MS(ms_reserve(delta_solve_kernel<T>, row_tile + a_tile));
-            QIL_MS(qil_launch_chained(delta_solve_kernel<T>, dim3(n_heads, n_chunks), dim3(256), row_tile + a_tile, stream, in,
-                                      chunk_start, chunk_len, n_heads, d, e, y, w));
-            QIL_MS_WALK(true);
+            QIL_MS(ms_reserve(delta_solve_kernel<T>, row_tile + 3 * a_tile));
+            QIL_MS(qil_launch_chained(delta_solve_kernel<T>, dim3(n_heads, n_chunks), dim3(256), row_tile + 3 * a_tile, stream, in,
+                                      chunk_start, chunk_len, n_heads, d, e, y, w, decays));
+            if (d <= 128) { if (cols == 8) QIL_MS_WALK(8, 1); else QIL_MS_WALK(16, 1); }
+            else { if (cols == 8) QIL_MS_WALK(8, 2); else QIL_MS_WALK(16, 2); }
+            QIL_MS_OUTPUTS(true);
         } else {
-            QIL_MS_WALK(false);
+            QIL_MS(ms_reserve(state_own_kernel<T>, row_tile + a_tile));
+            QIL_MS(qil_launch_chained(state_own_kernel<T>, dim3(n_heads, n_chunks, (e + 63) / 64), dim3(256), row_tile + a_tile, stream,
+                                      in, chunk_start, chunk_len, n_heads, d, e, chunk_state, decays));
+            if (err == cudaSuccess) {
+                const int code = qil_gla_carry(chunk_state, decays, slots, carry, n_carries, n_heads, d, e, stream);
+                if (code != 0) return code;
+            }
+            QIL_MS_OUTPUTS(false);
         }
     });
+#undef QIL_MS_OUTPUTS
 #undef QIL_MS_WALK
 #undef QIL_MS
     if (err != cudaSuccess) { snprintf(qil_error_text, sizeof(qil_error_text), "%s", cudaGetErrorString(err)); return (int)err; }
@@ -762,25 +972,49 @@ __device__ __forceinline__ void ms_write(bf16* p, const MsVec<4>& v) {
     *reinterpret_cast<uint2*>(p) = raw;
 }
 
+struct DeltaInputs {
+    long long ld;
+    int b_col, a_col;
+    const float* taps_w;
+    int taps;
+    float* state;
+    const float* a_log;
+    const float* dt_bias;
+    float q_scale;
+    const int* positions;
+    const int* token_row;
+    int n_tokens, heads, kv_heads, d, e;
+    float* qk;
+    float* beta;
+    float* log_decay;
+};
+
+template <typename T>
+__device__ __forceinline__ void delta_gates(const DeltaInputs& in, const T* row, int token, int lane) {
+    for (int h = lane; h < in.heads; h += 32) {
+        const float b = to_f32<T>(row[in.b_col + h]), a = to_f32<T>(row[in.a_col + h]) + in.dt_bias[h];
+        in.beta[(size_t)token * in.heads + h] = 1.f / (1.f + expf(-b));
+        const float softplus = fmaxf(a, 0.f) + log1pf(expf(-fabsf(a)));
+        in.log_decay[(size_t)token * in.heads + h] = -expf(in.a_log[h]) * softplus;
+    }
+}
+
+__device__ __forceinline__ float ms_silu(float y) { return y / (1.f + expf(-y)); }
+
+// One token, its items (q and k heads, runs of value channels, the gates) over the warps of `splits` blocks.
 template <typename T, int V>
-__global__ void __launch_bounds__(256)
-delta_prepare_kernel(const T* __restrict__ proj, long long ld, int b_col, int a_col, const float* __restrict__ taps_w, int taps,
-                     float* __restrict__ state, const float* __restrict__ a_log, const float* __restrict__ dt_bias, float q_scale,
-                     const int* __restrict__ positions, const int* __restrict__ token_row, int n_tokens, int heads, int kv_heads,
-                     int d, int e, float* __restrict__ qk, T* __restrict__ v_out, float* __restrict__ beta,
-                     float* __restrict__ log_decay) {
-    const int token = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int pos = positions[token], row = token_row[token];
+__device__ __forceinline__ void delta_prepare_token(const DeltaInputs& in, const T* __restrict__ proj, T* __restrict__ v_out, int token,
+                                                    int item0, int step, int lane) {
+    const int d = in.d, taps = in.taps, heads = in.heads, kv_heads = in.kv_heads, e = in.e;
+    const int pos = in.positions[token], row = in.token_row[token];
     const int qk_width = kv_heads * d, channels = 2 * qk_width + heads * e;
     int history = 0;                 // how many earlier positions this step itself brought (at most taps - 1 matter)
-    while (history < taps - 1 && token - history - 1 >= 0 && token_row[token - history - 1] == row
-           && positions[token - history - 1] == pos - history - 1)
+    while (history < taps - 1 && token - history - 1 >= 0 && in.token_row[token - history - 1] == row
+           && in.positions[token - history - 1] == pos - history - 1)
         ++history;
-    const bool alone = history == 0 && (token + 1 >= n_tokens || token_row[token + 1] != row);
-    float* slot = state + (size_t)row * (taps - 1) * channels;
-    qil_wait_for_producer();
-    qil_release_consumer();
-    const T* mine = proj + (size_t)token * ld;
+    const bool alone = history == 0 && (token + 1 >= in.n_tokens || in.token_row[token + 1] != row);
+    float* slot = in.state + (size_t)row * (taps - 1) * channels;
+    const T* mine = proj + (size_t)token * in.ld;
     auto convolved = [&](int c) {
         MsVec<V> y;
 #pragma unroll
@@ -790,24 +1024,24 @@ delta_prepare_kernel(const T* __restrict__ proj, long long ld, int b_col, int a_
             MsVec<V> u;
 #pragma unroll
             for (int i = 0; i < V; ++i) u.x[i] = 0.f;
-            if (back <= history) u = ms_read<T, V>(mine - (long long)back * ld + c);
+            if (back <= history) u = ms_read<T, V>(mine - (long long)back * in.ld + c);
             else if (pos - back >= 0) u = ms_read<float, V>(slot + (size_t)(taps - 1 - (back - history)) * channels + c);
             // row j of the slot is read before row j - 1 is overwritten by it, and by this thread alone
             if (alone && j > 0) ms_write(slot + (size_t)(j - 1) * channels + c, u);
-            const MsVec<V> w = ms_read<float, V>(taps_w + (size_t)j * channels + c);
+            const MsVec<V> w = ms_read<float, V>(in.taps_w + (size_t)j * channels + c);
 #pragma unroll
             for (int i = 0; i < V; ++i) y.x[i] = fmaf(w.x[i], u.x[i], y.x[i]);
         }
 #pragma unroll
-        for (int i = 0; i < V; ++i) y.x[i] = y.x[i] / (1.f + expf(-y.x[i]));
+        for (int i = 0; i < V; ++i) y.x[i] = ms_silu(y.x[i]);
         return y;
     };
     const int v_items = (heads * e + 32 * V - 1) / (32 * V);
-    float* qk_row = qk + (size_t)token * 2 * qk_width;
-    for (int item = warp; item < 2 * kv_heads + v_items + 1; item += 8) {
+    float* qk_row = in.qk + (size_t)token * 2 * qk_width;
+    for (int item = item0; item < 2 * kv_heads + v_items + 1; item += step) {
         if (item < 2 * kv_heads) {                      // a q or a k head
             const int c0 = item * d;
-            const float scale = item < kv_heads ? q_scale : 1.f;
+            const float scale = item < kv_heads ? in.q_scale : 1.f;
             MsVec<V> kept[MS_PREPARE_KEPT / V];
             float ss = 0.f;
             for (int n = 0, c = lane * V; c < d; ++n, c += 32 * V) {
@@ -833,12 +1067,77 @@ delta_prepare_kernel(const T* __restrict__ proj, long long ld, int b_col, int a_
             const int c = (item - 2 * kv_heads) * 32 * V + lane * V;
             if (c < heads * e) ms_write(v_out + (size_t)token * heads * e + c, convolved(2 * qk_width + c));
         } else {
-            for (int h = lane; h < heads; h += 32) {
-                const float b = to_f32<T>(mine[b_col + h]), a = to_f32<T>(mine[a_col + h]) + dt_bias[h];
-                beta[(size_t)token * heads + h] = 1.f / (1.f + expf(-b));
-                const float softplus = fmaxf(a, 0.f) + log1pf(expf(-fabsf(a)));
-                log_decay[(size_t)token * heads + h] = -expf(a_log[h]) * softplus;
+            delta_gates<T>(in, mine, token, lane);
+        }
+    }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+delta_prepare_kernel(const T* __restrict__ proj, DeltaInputs in, T* __restrict__ v_out) {
+    qil_wait_for_producer();
+    qil_release_consumer();
+    delta_prepare_token<T, V>(in, proj, v_out, blockIdx.x, blockIdx.y * 8 + (threadIdx.x >> 5), 8 * gridDim.y, threadIdx.x & 31);
+}
+
+// Prompts: MS_RUN tokens a block.  Where they and the TAPS - 1 rows before them are one request's, a lane reads every row of its
+// four channels once for all of them (heads of at most 128 channels); else token by token.  The same sums in the same order.
+#define MS_RUN 4
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256)
+delta_prepare_run_kernel(const T* __restrict__ proj, DeltaInputs in, T* __restrict__ v_out) {
+    const int token0 = blockIdx.x * MS_RUN, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int before = token0 - (TAPS - 1), last = token0 + MS_RUN - 1;
+    const bool whole = before >= 0 && last < in.n_tokens && in.token_row[before] == in.token_row[last]
+                       && in.positions[last] - in.positions[before] == MS_RUN + TAPS - 2;
+    qil_wait_for_producer();
+    qil_release_consumer();
+    if (!whole) {
+        for (int token = token0; token <= min(last, in.n_tokens - 1); ++token)
+            delta_prepare_token<T, 4>(in, proj, v_out, token, warp, 8, lane);
+        return;
+    }
+    const int d = in.d, heads = in.heads, kv_heads = in.kv_heads, e = in.e;
+    const int qk_width = kv_heads * d, channels = 2 * qk_width + heads * e, v_items = (heads * e + 127) / 128;
+    const T* first_row = proj + (size_t)before * in.ld;
+    for (int item = warp; item < 2 * kv_heads + v_items + MS_RUN; item += 8) {
+        if (item >= 2 * kv_heads + v_items) {
+            const int token = token0 + item - (2 * kv_heads + v_items);
+            delta_gates<T>(in, proj + (size_t)token * in.ld, token, lane);
+            continue;
+        }
+        const bool is_head = item < 2 * kv_heads;
+        const int c = is_head ? item * d + lane * 4 : 2 * qk_width + (item - 2 * kv_heads) * 128 + lane * 4;
+        const bool mine = is_head ? lane * 4 < d : c < channels;
+        MsVec<4> u[MS_RUN + TAPS - 1], w[TAPS], y[MS_RUN];
+#pragma unroll
+        for (int i = 0; i < MS_RUN + TAPS - 1; ++i) u[i] = mine ? ms_read<T, 4>(first_row + (size_t)i * in.ld + c) : MsVec<4>{{0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = mine ? ms_read<float, 4>(in.taps_w + (size_t)j * channels + c) : MsVec<4>{{0.f, 0.f, 0.f, 0.f}};
+        float ss[MS_RUN];
+#pragma unroll
+        for (int t = 0; t < MS_RUN; ++t) {
+            ss[t] = 0.f;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                float sum = 0.f;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) sum = fmaf(w[j].x[i], u[t + j].x[i], sum);
+                y[t].x[i] = ms_silu(sum);
+                ss[t] = fmaf(y[t].x[i], y[t].x[i], ss[t]);
             }
+        }
+        if (is_head) {
+#pragma unroll
+            for (int t = 0; t < MS_RUN; ++t) {
+                const float inv = (item < kv_heads ? in.q_scale : 1.f) / sqrtf(warp_sum(ss[t]) + 1e-6f);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) y[t].x[i] *= inv;
+                if (mine) ms_write(in.qk + (size_t)(token0 + t) * 2 * qk_width + c, y[t]);
+            }
+        } else if (mine) {
+#pragma unroll
+            for (int t = 0; t < MS_RUN; ++t) ms_write(v_out + (size_t)(token0 + t) * heads * e + c - 2 * qk_width, y[t]);
         }
     }
 }
@@ -853,11 +1152,23 @@ extern "C" int qil_delta_prepare(const void* proj, long long ld, int b_col, int 
     if (taps > 1 && state == nullptr) QIL_REFUSE("delta_prepare: a convolution over time needs its state");
     const bool wide = d % 4 == 0 && (heads * e) % 4 == 0 && ld % 4 == 0 &&
                       (((uintptr_t)proj | (uintptr_t)taps_w | (uintptr_t)state | (uintptr_t)qk | (uintptr_t)v_out) & 15) == 0;
+    const DeltaInputs in = {ld, b_col, a_col, taps_w, taps, state, a_log, dt_bias, q_scale, positions, token_row, n_tokens, heads,
+                            kv_heads, d, e, qk, beta, log_decay};
+    const int lanes = wide ? 4 : 1, items = 2 * kv_heads + (heads * e + 32 * lanes - 1) / (32 * lanes) + 1;
+    int splits = 1;                 // few tokens (a decode step): a token's items over several blocks
+    while (splits < 16 && (long long)n_tokens * splits < 148 && splits * 8 < items) splits <<= 1;
+    const bool runs = wide && d <= 128 && taps >= 2 && taps <= 4 && n_tokens >= 16 * MS_RUN;
+#define QIL_PREPARE_RUN(TAPS)                                                                                              \
+    qil_launch_chained(delta_prepare_run_kernel<T, TAPS>, dim3((n_tokens + MS_RUN - 1) / MS_RUN), dim3(256), 0, stream,    \
+                       (const T*)proj, in, (T*)v_out)
 #define QIL_PREPARE_GO(V)                                                                                                  \
-    qil_launch_chained(delta_prepare_kernel<T, V>, dim3(n_tokens), dim3(256), 0, stream, (const T*)proj, ld, b_col, a_col, \
-                       taps_w, taps, state, a_log, dt_bias, q_scale, positions, token_row, n_tokens, heads, kv_heads, d, e, \
-                       qk, (T*)v_out, beta, log_decay)
-    QIL_DISPATCH_1(act_dtype, { if (wide) QIL_PREPARE_GO(4); else QIL_PREPARE_GO(1); });
+    qil_launch_chained(delta_prepare_kernel<T, V>, dim3(n_tokens, splits), dim3(256), 0, stream, (const T*)proj, in, (T*)v_out)
+    QIL_DISPATCH_1(act_dtype, {
+        if (runs) { if (taps == 2) QIL_PREPARE_RUN(2); else if (taps == 3) QIL_PREPARE_RUN(3); else QIL_PREPARE_RUN(4); }
+        else if (wide) QIL_PREPARE_GO(4);
+        else QIL_PREPARE_GO(1);
+    });
+#undef QIL_PREPARE_RUN
 #undef QIL_PREPARE_GO
     QIL_CHECK_LAUNCH();
 }

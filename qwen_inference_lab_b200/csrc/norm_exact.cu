@@ -430,9 +430,9 @@ __device__ __forceinline__ void join_store4(bf16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = raw;
 }
 
-// Rows of up to 1024 * V4 values, a multiple of four, held in registers: 16 bytes a load.
-template <typename TX, typename W, typename TO, int V4, bool NORMED>
-__global__ void __launch_bounds__(256)
+// Rows of up to 4 * NT * V4 values, a multiple of four, held in registers: 16 bytes a load.
+template <typename TX, typename W, typename TO, int NT, int V4, bool NORMED>
+__global__ void __launch_bounds__(NT)
 branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext next, TO* __restrict__ rows) {
     __shared__ float scratch[32];
     qil_wait_for_producer();
@@ -444,7 +444,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext
     float ss[JOIN_MOST_NORMED] = {0.f, 0.f};
 #pragma unroll
     for (int c = 0; c < V4; ++c) {
-        const int col = (threadIdx.x + c * 256) * 4;
+        const int col = (threadIdx.x + c * NT) * 4;
         v[c] = stream[c] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (NORMED) {
 #pragma unroll
@@ -491,7 +491,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext
                     const float r = 1.0f / sqrtf(block_sum(ss[m], scratch) / (float)width + in.eps);
 #pragma unroll
                     for (int c = 0; c < V4; ++c) {
-                        const int col = (threadIdx.x + c * 256) * 4;
+                        const int col = (threadIdx.x + c * NT) * 4;
                         if (col >= width) continue;
                         const float4 w = join_load4<float>(in.w[k] + col);
                         v[c].x = fmaf(in.scale[k], held[m][c].x * r * w.x, v[c].x); v[c].y = fmaf(in.scale[k], held[m][c].y * r * w.y, v[c].y);
@@ -504,7 +504,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext
     float sum = 0.f;
 #pragma unroll
     for (int c = 0; c < V4; ++c) {
-        const int col = (threadIdx.x + c * 256) * 4;
+        const int col = (threadIdx.x + c * NT) * 4;
         if (col >= width) continue;
         float4 now = make_float4(stream[c].x + v[c].x, stream[c].y + v[c].y, stream[c].z + v[c].z, stream[c].w + v[c].w);
         now.x = round_to<TX>(now.x); now.y = round_to<TX>(now.y); now.z = round_to<TX>(now.z); now.w = round_to<TX>(now.w);
@@ -518,7 +518,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext
     if (next_w == nullptr) {
 #pragma unroll
         for (int c = 0; c < V4; ++c) {
-            const int col = (threadIdx.x + c * 256) * 4;
+            const int col = (threadIdx.x + c * NT) * 4;
             if (col < width) join_store4(out + col, v[c]);
         }
         return;
@@ -527,7 +527,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext
         const W* next_b = reinterpret_cast<const W*>(next.b);
 #pragma unroll
         for (int c = 0; c < V4; ++c) {
-            const int col = (threadIdx.x + c * 256) * 4;
+            const int col = (threadIdx.x + c * NT) * 4;
             if (col >= width) continue;
             const float4 w = join_load4<W>(next_w + col), b = join_load4<W>(next_b + col);
             join_store4(out + col, make_float4(fmaf(tanhf(next.alpha * v[c].x), w.x, b.x), fmaf(tanhf(next.alpha * v[c].y), w.y, b.y),
@@ -540,7 +540,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext
     float sq = 0.f;
 #pragma unroll
     for (int c = 0; c < V4; ++c) {
-        if ((threadIdx.x + c * 256) * 4 >= width) continue;
+        if ((threadIdx.x + c * NT) * 4 >= width) continue;
         v[c].x -= mean; v[c].y -= mean; v[c].z -= mean; v[c].w -= mean;
         sq = fmaf(v[c].x, v[c].x, sq); sq = fmaf(v[c].y, v[c].y, sq);
         sq = fmaf(v[c].z, v[c].z, sq); sq = fmaf(v[c].w, v[c].w, sq);
@@ -549,7 +549,7 @@ branch_join_regs_kernel(TX* __restrict__ x, JoinBranches in, int width, JoinNext
     const float scale = 1.0f / sqrtf(sq / (float)width + next.eps);
 #pragma unroll
     for (int c = 0; c < V4; ++c) {
-        const int col = (threadIdx.x + c * 256) * 4;
+        const int col = (threadIdx.x + c * NT) * 4;
         if (col >= width) continue;
         const float4 w = join_load4<W>(next_w + col);
         join_store4(out + col, make_float4(v[c].x * scale * w.x, v[c].y * scale * w.y, v[c].z * scale * w.z, v[c].w * scale * w.w));
@@ -637,16 +637,16 @@ extern "C" int qil_branch_join(void* x, int x_dtype, const float* const* branche
     in.n = n_branches; in.eps = branch_eps; in.y = y; in.top = top;
     const JoinNext next = {next_w, next_b, next_eps, next_alpha, next_kind};
     const bool wide = width % 4 == 0 && (bits & 15) == 0 && normed <= JOIN_MOST_NORMED;
-#define QIL_JOIN_ARGS(TX, TO) dim3(n_rows), dim3(256), 0, stream, (TX*)x, in, width, next, (TO*)rows
+#define QIL_JOIN_ARGS(TX, TO, NT) dim3(n_rows), dim3(NT), 0, stream, (TX*)x, in, width, next, (TO*)rows
 #define QIL_JOIN_SIZE(TX, WT, TO, N)                                                                                           \
     do {                                                                                                                       \
-        if (width <= 1024) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 1, N>, QIL_JOIN_ARGS(TX, TO));               \
-        else if (width <= 2048) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 2, N>, QIL_JOIN_ARGS(TX, TO));          \
-        else qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 4, N>, QIL_JOIN_ARGS(TX, TO));                             \
+        if (width <= 1024) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 256, 1, N>, QIL_JOIN_ARGS(TX, TO, 256));     \
+        else if (width <= 2048) qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 256, 2, N>, QIL_JOIN_ARGS(TX, TO, 256)); \
+        else qil_launch_chained(branch_join_regs_kernel<TX, WT, TO, 512, 2, N>, QIL_JOIN_ARGS(TX, TO, 512));                   \
     } while (0)
 #define QIL_JOIN_GO(TX, WT, TO)                                                                                                \
     do {                                                                                                                       \
-        if (!wide || width > 4096) qil_launch_chained(branch_join_kernel<TX, WT, TO>, QIL_JOIN_ARGS(TX, TO));                  \
+        if (!wide || width > 4096) qil_launch_chained(branch_join_kernel<TX, WT, TO>, QIL_JOIN_ARGS(TX, TO, 256));                  \
         else if (normed) QIL_JOIN_SIZE(TX, WT, TO, true);                                                                      \
         else QIL_JOIN_SIZE(TX, WT, TO, false);                                                                                 \
     } while (0)

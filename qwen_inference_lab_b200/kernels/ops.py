@@ -1201,14 +1201,12 @@ def state_chunks(inputs, slots, chunk_start, chunk_len, n_chunks, carry, n_carri
     if tuple(slots.shape[1:]) != (heads, d, e) or raw.shape != (inputs.n, heads * e):
         raise KernelError("state_chunks: shapes do not fit together")
     lib = core()
-    chunk = lib.qil_state_chunk()
     empty = lambda *shape: torch.empty(shape, dtype=torch.float32, device=slots.device)
-    y, w = (empty(n_chunks, heads, chunk, e), empty(n_chunks, heads, chunk, d)) if inputs.delta else (None, None)
+    scratch = empty(n_chunks * heads * lib.qil_state_chunk_scratch(c_int(d), c_int(e), c_int(1 if inputs.delta else 0)))
     states = empty(n_chunks, heads, d, e)
     _check(lib, lib.qil_state_chunks(*inputs.arguments, _p(chunk_start), _p(chunk_len), c_int(n_chunks), _p(carry),
-                                     c_int(n_carries), c_int(heads), c_int(d), c_int(e), _p(y), _p(w), _p(states), _p(slots),
-                                     _p(raw), c_int(dtype_code(inputs.dtype)), _stream()), "state_chunks",
-           kernels=3 if inputs.delta else 2)
+                                     c_int(n_carries), c_int(heads), c_int(d), c_int(e), _p(scratch), _p(states), _p(slots),
+                                     _p(raw), c_int(dtype_code(inputs.dtype)), _stream()), "state_chunks", kernels=3)
 
 
 def delta_prepare(proj, columns, taps_weight, state, a_log, dt_bias, q_scale, positions, token_row, heads, kv_heads, d, e):
