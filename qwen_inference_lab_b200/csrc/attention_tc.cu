@@ -1,13 +1,15 @@
 // Causal grouped-query attention of whole 128-token query tiles over the paged cache on the
 // fifth-generation tensor cores (tcgen05.mma, accumulators in tensor memory, operands brought by
-// TMA), for head size 128 and bfloat16.  Same arithmetic as attention_mma.cu (scores = q k^T *
+// TMA), for bfloat16 and one pair of sizes: -DQIL_HEAD_DIM=<of queries and keys> -DQIL_V_DIM=<of values>, each a multiple
+// of 16 up to 128 (the default of both).  Same arithmetic as attention_mma.cu (scores = q k^T *
 // head_dim^-1/2 over keys j <= the token's absolute position, float32 softmax, times v;
 // qil/model.py:59-68); this kernel takes the bulk of long prompt portions, the mma.sync kernel what
 // is left over.
 //
 // One block per (tile of 128 query tokens, query head), 224 threads:
 //   warp 0, 6   issue TMA loads: warp 0 the query tile once and then per 64 keys the pages of K, warp 6 the
-//               pages of V (one box per page and 64-wide half of the head, 128-byte swizzle);
+//               pages of V (one box per page and 64-wide slab of the head, 128-byte swizzle; what a box reaches past
+//               the head's columns is filled with zeros);
 //   warp 1      one thread issues tcgen05.mma: S = Q K^T (128 x 128 x 128) into one of two score
 //               buffers in tensor memory, and O += P V once the softmax warps have published P;
 //               it runs one score tile ahead of the softmax;
@@ -18,7 +20,7 @@
 //               2^8 (until then P is computed against the older maximum, which is exact algebra and
 //               safe in float32); finally O / l -> global memory.
 // K tiles are K-major operands and V tiles MN-major operands of the same shared-memory image
-// ([key][64 elements = 128 bytes] x two halves of the head).
+// ([key][64 elements = 128 bytes] x the slabs of the head).
 //
 // Every mbarrier wait is bounded (about a second), records its place in the error word when it runs
 // out and makes its role stop; the block then frees its tensor memory and returns.
@@ -27,15 +29,27 @@
 
 QIL_ERROR_STORAGE
 
-#define AT_D 128
+#ifndef QIL_HEAD_DIM
+#define QIL_HEAD_DIM 128
+#endif
+#ifndef QIL_V_DIM
+#define QIL_V_DIM QIL_HEAD_DIM
+#endif
+#define AT_D QIL_HEAD_DIM        // of a query and a key
+#define AT_E QIL_V_DIM           // of a value and an output
+static_assert(AT_D % 16 == 0 && AT_D >= 16 && AT_D <= 128 && AT_E % 16 == 0 && AT_E >= 16 && AT_E <= 128,
+              "the tensor-memory attention takes head and value sizes 16, 32, ..., 128");
+#define AT_DS ((AT_D + 63) / 64) // slabs of 64 columns of a query or key row
+#define AT_ES ((AT_E + 63) / 64) // and of a value row
 #define AT_M 128                 // query tokens per block
 #ifndef AT_N
 #define AT_N 64                  // keys per tile (64: two blocks fit an SM and overlap each other's softmax and MMAs)
 #endif
 #define AT_QSLAB (AT_M * 128)    // bytes of a [128 query rows][64 elements] slab (also of a P slab: 64 keys)
-#define AT_QTILE (2 * AT_QSLAB)  // the query tile: two halves of the head
+#define AT_QTILE (AT_DS * AT_QSLAB)   // the query tile
 #define AT_SLAB (AT_N * 128)     // bytes of a [keys][64 elements] slab of K or V
-#define AT_TILE (2 * AT_SLAB)    // a K or V tile: two halves of the head
+#define AT_KTILE (AT_DS * AT_SLAB)    // a K tile
+#define AT_VTILE (AT_ES * AT_SLAB)    // a V tile
 #define AT_TMEM_COLS (AT_N == 64 ? 256 : 512)
 #define AT_STAGES 2
 #define AT_WAIT_CYCLES 2000000000ll
@@ -65,10 +79,6 @@ __device__ __forceinline__ bool at_wait(unsigned long long* bar, unsigned parity
         if (clock64() - start > AT_WAIT_CYCLES) return false;
     }
     return true;
-}
-__device__ __forceinline__ void at_tma_2d(void* smem, const CUtensorMap* map, unsigned long long* bar, int x, int y) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];\n"
-                 ::"r"(at_smem(smem)), "l"((unsigned long long)map), "r"(at_smem(bar)), "r"(x), "r"(y) : "memory");
 }
 __device__ __forceinline__ void at_tma_3d(void* smem, const CUtensorMap* map, unsigned long long* bar, int x, int y, int z) {
     asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];\n"
@@ -164,7 +174,7 @@ struct AtShared {
 };
 
 struct AtParams {
-    bf16* out;                  // [N, Hq, 128]
+    bf16* out;                  // [N, Hq, AT_E]
     const int* block_table;
     int table_stride;
     int n_q_heads, n_kv_heads, page_size;
@@ -190,8 +200,8 @@ struct AtParams {
 #define AT_VALUE_WARP 6                  // warps: 0 keys, 1 MMA issue, 2-5 softmax, 6 values
 #define AT_THREADS 224
 __global__ void __launch_bounds__(AT_THREADS, (AT_N == 64) ? 2 : 1)
-attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
-               AtParams p, const int4* __restrict__ tile_info) {
+attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+               const __grid_constant__ CUtensorMap map_v, AtParams p, const int4* __restrict__ tile_info) {
     // swizzled operand tiles need 1024-byte alignment; the declaration asks for it and a misaligned
     // window is refused below rather than padded, so that two blocks fit the SM's shared memory
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -200,10 +210,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         if (threadIdx.x == 0) atomicExch(p.error_word, 31);
         return;
     }
-    unsigned char* sQ = base;                               // [2 slabs]
-    unsigned char* sK = sQ + AT_QTILE;                      // [stages][2 slabs]
-    unsigned char* sV = sK + AT_STAGES * AT_TILE;           // [stages][2 slabs]
-    AtShared* sh = reinterpret_cast<AtShared*>(sV + AT_STAGES * AT_TILE);
+    unsigned char* sQ = base;                               // [slabs]
+    unsigned char* sK = sQ + AT_QTILE;                      // [stages][slabs]
+    unsigned char* sV = sK + AT_STAGES * AT_KTILE;          // [stages][slabs]
+    AtShared* sh = reinterpret_cast<AtShared*>(sV + AT_STAGES * AT_VTILE);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     // heads vary fastest, so all heads of the longest tile start first (tiles come sorted, longest first)
     const int head = blockIdx.x;
@@ -250,26 +260,27 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         // free as soon as the scores of two tiles ago are computed, a stage of values only when that tile's
         // output is, and the next scores must not wait behind a copy of values.  The whole warp walks the
         // tiles: every lane fetches one block-table entry of a batch of 32 in one coalesced read, lane 0
-        // waits and arms the barrier, and the copies go out one per lane (lane = half of the head, page of
+        // waits and arms the barrier, and the copies go out one per lane (lane = slab of the head, page of
         // the tile) with page ids handed over by shuffles; issuing a tile's copies from one thread one after
         // the other would cost that thread more than the tile's MMAs take.
         const int kv = warp == 0 ? 0 : 1;
+        const CUtensorMap* const map = kv == 0 ? &map_k : &map_v;
         if (lane == 0) {
-            asm volatile("prefetch.tensormap [%0];\n" ::"l"((unsigned long long)&map_kv) : "memory");
+            asm volatile("prefetch.tensormap [%0];\n" ::"l"((unsigned long long)map) : "memory");
             if (kv == 0) {
                 asm volatile("prefetch.tensormap [%0];\n" ::"l"((unsigned long long)&map_q) : "memory");
-                // queries: box (64 elements, 1 head, 128 tokens) per half of the head
+                // queries: box (64 elements, 1 head, 128 tokens) per slab of the head
                 at_expect_tx(&sh->q_full, AT_QTILE);
-                at_tma_3d(sQ, &map_q, &sh->q_full, 0, head, n0);
-                at_tma_3d(sQ + AT_QSLAB, &map_q, &sh->q_full, 64, head, n0);
+                for (int slab = 0; slab < AT_DS; ++slab) at_tma_3d(sQ + slab * AT_QSLAB, &map_q, &sh->q_full, slab * 64, head, n0);
             }
         }
         unsigned long long* const full = kv == 0 ? sh->k_full : sh->v_full;
         unsigned long long* const empty = kv == 0 ? sh->k_empty : sh->v_empty;
         unsigned char* const tiles = kv == 0 ? sK : sV;
+        const int slabs = kv == 0 ? AT_DS : AT_ES, tile_bytes = kv == 0 ? AT_KTILE : AT_VTILE;
         const int pages_per_tile = AT_N / p.page_size;
         const int tiles_per_batch = 32 / pages_per_tile;       // pages_per_tile is 1, 2, 4 or 8
-        const int page_bytes = p.page_size * 128;               // one page of one half: page_size rows of 128 bytes
+        const int page_bytes = p.page_size * 128;               // one page of one slab: page_size rows of 128 bytes
         const int last_page = hi / p.page_size;
         int ok = 1;
         int my_page = -1;
@@ -283,23 +294,21 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             const int first_key = (tile0 + j) * AT_N;
             int pages = pages_per_tile;
             if (first_key + AT_N - 1 > hi) pages = (hi - first_key) / p.page_size + 1;
-            const int pg = lane % pages_per_tile, half = (lane / pages_per_tile) & 1;
+            const int pg = lane % pages_per_tile, slab = (lane / pages_per_tile) & 1;
             const int page = __shfl_sync(0xffffffffu, my_page, (j % tiles_per_batch) * pages_per_tile + pg);
             if (lane == 0) {
                 if (!at_wait(&empty[stage], parity)) {
                     atomicExch(p.error_word, 11);
                     ok = 0;
                 } else {
-                    at_expect_tx(&full[stage], (unsigned)(pages * 2 * page_bytes));
+                    at_expect_tx(&full[stage], (unsigned)(pages * slabs * page_bytes));
                 }
             }
             ok = __shfl_sync(0xffffffffu, ok, 0);
             if (!ok) break;
-            if (lane < 2 * pages_per_tile && pg < pages) {
-                // cache rows of one layer: ((page * 2 + kv) * kv_heads + kv_head) * page_size + slot
-                const int row = ((page * 2 + kv) * p.n_kv_heads + kv_head) * p.page_size;
-                at_tma_2d(tiles + stage * AT_TILE + half * AT_SLAB + pg * page_bytes, &map_kv, &full[stage], half * 64, row);
-            }
+            if (lane < slabs * pages_per_tile && pg < pages)      // a page's rows of this kv head begin at kv_head * page_size
+                at_tma_3d(tiles + stage * tile_bytes + slab * AT_SLAB + pg * page_bytes, map, &full[stage], slab * 64,
+                          kv_head * p.page_size, page);
             if (lane == 0) AT_STAMP(0, 2 * j + kv);
         }
         // leave only after the copies have been consumed or have had a second to land
@@ -313,9 +322,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            // bfloat16 -> float32, M = 128; scores: N = keys; output: N = head size, B (V) read MN-major
+            // bfloat16 -> float32, M = 128; scores: N = keys; output: N = the value slabs' columns, B (V) read MN-major
             const unsigned idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((unsigned)(AT_N >> 3) << 17) | ((unsigned)(AT_M >> 4) << 24);
-            const unsigned idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((unsigned)(AT_D >> 3) << 17) | ((unsigned)(AT_M >> 4) << 24);
+            const unsigned idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((unsigned)(AT_ES * 64 >> 3) << 17) | ((unsigned)(AT_M >> 4) << 24);
             bool ok = at_wait(&sh->q_full, 0);
             if (!ok) atomicExch(p.error_word, 13);
             auto issue_scores = [&](int j) -> bool {
@@ -324,10 +333,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 // The score buffer of tile j held P of tile j - 2: the MMA that read it was issued before this one
                 // and MMAs run in the order of their issue, so the buffer needs no barrier of its own.
                 at_fence_after();
-                const unsigned q_addr = at_smem(sQ), k_addr = at_smem(sK + stage * AT_TILE);
+                const unsigned q_addr = at_smem(sQ), k_addr = at_smem(sK + stage * AT_KTILE);
 #pragma unroll
                 for (int kk = 0; kk < AT_D / 16; ++kk) {
-                    // half of the head, then 16 elements = 32 bytes inside the 128-byte row
+                    // slab of the head, then 16 elements = 32 bytes inside the 128-byte row
                     at_mma(tmem_s(buf), at_desc_kmajor(q_addr + (kk >> 2) * AT_QSLAB + (kk & 3) * 32),
                            at_desc_kmajor(k_addr + (kk >> 2) * AT_SLAB + (kk & 3) * 32), idesc_s, kk ? 1u : 0u);
                 }
@@ -348,7 +357,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 if (!at_wait(&sh->p_full[j & 1], (j >> 1) & 1)) { atomicExch(p.error_word, 17); ok = false; break; }
                 AT_STAMP(1, 4 * j + 2);
                 at_fence_after();
-                const unsigned v_addr = at_smem(sV + stage * AT_TILE);
+                const unsigned v_addr = at_smem(sV + stage * AT_VTILE);
 #pragma unroll
                 for (int kk = 0; kk < AT_N / 16; ++kk) {
                     // P: 16 keys = 8 columns of tensor memory; V: 16 keys = 16 rows of 128 bytes
@@ -456,7 +465,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 if (!at_wait(&sh->pv_done, (j - 1) & 1)) { if (lane == 0) atomicExch(p.error_word, 22); ok = false; break; }
                 at_fence_after();
 #pragma unroll 1
-                for (int c = 0; c < AT_D / 32; ++c) {
+                for (int c = 0; c < (AT_E + 31) / 32; ++c) {
                     unsigned r[32];
                     at_tmem_ld32(tmem_o + lane_base + c * 32, r);
                     at_wait_ld();
@@ -472,12 +481,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             if (j == n_tiles - 1) {
                 if (!at_wait(&sh->v_full[stage], (j / AT_STAGES) & 1)) { if (lane == 0) atomicExch(p.error_word, 23); ok = false; break; }
                 if (row < AT_N && key0 + row > hi) {
-                    unsigned char* v_row = sV + stage * AT_TILE + row * 128;
+                    unsigned char* v_row = sV + stage * AT_VTILE + row * 128;
 #pragma unroll
-                    for (int c = 0; c < 8; ++c) {
-                        *reinterpret_cast<uint4*>(v_row + c * 16) = make_uint4(0u, 0u, 0u, 0u);
-                        *reinterpret_cast<uint4*>(v_row + AT_SLAB + c * 16) = make_uint4(0u, 0u, 0u, 0u);
-                    }
+                    for (int c = 0; c < 8 * AT_ES; ++c)
+                        *reinterpret_cast<uint4*>(v_row + c / 8 * AT_SLAB + c % 8 * 16) = make_uint4(0u, 0u, 0u, 0u);
                 }
             }
             // P over the scores it came from: this thread's row, two keys per 32-bit column
@@ -505,15 +512,16 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             at_fence_after();
             if (p.sink_log2 != nullptr) l += (m_used == -INFINITY) ? 1.f : exp2f(p.sink_log2[head] - m_used);
             const float inv = l > 0.f ? 1.f / l : 0.f;
-            bf16* dst = p.out + ((size_t)(n0 + row) * p.n_q_heads + head) * AT_D;
+            bf16* dst = p.out + ((size_t)(n0 + row) * p.n_q_heads + head) * AT_E;
 #pragma unroll 1
-            for (int c = 0; c < AT_D / 32; ++c) {
+            for (int c = 0; c < (AT_E + 31) / 32; ++c) {
                 unsigned r[32];
                 __syncwarp();
                 at_tmem_ld32(tmem_o + lane_base + c * 32, r);
                 at_wait_ld();
 #pragma unroll
                 for (int q = 0; q < 4; ++q) {
+                    if (AT_E % 32 != 0 && c * 32 + q * 8 >= AT_E) break;
                     uint4 packed;
                     bf16* o = reinterpret_cast<bf16*>(&packed);
 #pragma unroll
@@ -548,9 +556,11 @@ static AtEncodeFn at_encode() {
 }
 
 extern "C" int qil_attn_tc_head_dim() { return AT_D; }
+extern "C" int qil_attn_tc_v_dim() { return AT_E; }
 extern "C" int qil_attn_tc_keys_per_tile() { return AT_N; }
 
-// q [N, Hq, 128], kv one layer's pages [pages, 2, Hkv, page_size, 128], out [N, Hq, 128], all bfloat16.
+// q [N, Hq, AT_D], out [N, Hq, AT_E], kv one layer's pages: a page's key rows [Hkv, page_size, AT_D] and behind them its value
+// rows [Hkv, page_size, AT_E]; all bfloat16.
 // tile_info int32 [n_tiles, 4] = (first token, its absolute position, 128, block-table row): whole tiles only.
 // page_size must divide the keys per tile and be a multiple of 8.  error_word: a device int, zeroed by the
 // caller once.  trace: null, or 3 * 1024 int64 for the time stamps of block (0, 0) in a build with AT_TRACE.
@@ -588,7 +598,7 @@ extern "C" int qil_attn_tc_prefill_capped(const void* q, const void* kv, void* o
     if (error_word == nullptr) QIL_REFUSE("attn_tc: needs an error word");
     AtEncodeFn encode = at_encode();
     if (encode == nullptr) QIL_REFUSE("attn_tc: the driver does not offer cuTensorMapEncodeTiled");
-    CUtensorMap map_q, map_kv;
+    CUtensorMap map_q, map_k, map_v;
     {
         const cuuint64_t dims[3] = {AT_D, (cuuint64_t)n_q_heads, (cuuint64_t)n_tokens};
         const cuuint64_t strides[2] = {AT_D * 2, (cuuint64_t)n_q_heads * AT_D * 2};
@@ -599,13 +609,15 @@ extern "C" int qil_attn_tc_prefill_capped(const void* q, const void* kv, void* o
                                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
         if (r != CUDA_SUCCESS) QIL_REFUSE("attn_tc: cuTensorMapEncodeTiled failed for the queries (%d)", (int)r);
     }
-    {
-        const cuuint64_t rows = (cuuint64_t)num_pages * 2 * n_kv_heads * page_size;
-        const cuuint64_t dims[2] = {AT_D, rows};
-        const cuuint64_t strides[1] = {AT_D * 2};
-        const cuuint32_t box[2] = {64, (cuuint32_t)page_size};
-        const cuuint32_t elem[2] = {1, 1};
-        const CUresult r = encode(&map_kv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(kv), dims, strides, box, elem,
+    for (int values = 0; values < 2; ++values) {
+        // (column, row of the page, page); the values' rows lie behind the keys' in every page
+        const cuuint64_t rows = (cuuint64_t)n_kv_heads * page_size, width = values ? AT_E : AT_D;
+        const cuuint64_t dims[3] = {width, rows, (cuuint64_t)num_pages};
+        const cuuint64_t strides[2] = {width * 2, rows * (AT_D + AT_E) * 2};
+        const cuuint32_t box[3] = {64, (cuuint32_t)page_size, 1};
+        const cuuint32_t elem[3] = {1, 1, 1};
+        void* from = (char*)const_cast<void*>(kv) + (values ? rows * AT_D * 2 : 0);
+        const CUresult r = encode(values ? &map_v : &map_k, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, from, dims, strides, box, elem,
                                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
         if (r != CUDA_SUCCESS) QIL_REFUSE("attn_tc: cuTensorMapEncodeTiled failed for the cache (%d)", (int)r);
@@ -623,14 +635,14 @@ extern "C" int qil_attn_tc_prefill_capped(const void* q, const void* kv, void* o
     }
     p.error_word = error_word;
     p.trace = trace;
-    const int smem = AT_QTILE + 2 * AT_STAGES * AT_TILE + (int)sizeof(AtShared);
+    const int smem = AT_QTILE + AT_STAGES * (AT_KTILE + AT_VTILE) + (int)sizeof(AtShared);
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) QIL_REFUSE("attn_tc: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
         configured = true;
     }
-    attn_tc_kernel<<<dim3(n_q_heads, n_tiles), AT_THREADS, smem, stream>>>(map_q, map_kv, p, (const int4*)tile_info);
+    attn_tc_kernel<<<dim3(n_q_heads, n_tiles), AT_THREADS, smem, stream>>>(map_q, map_k, map_v, p, (const int4*)tile_info);
     QIL_CHECK_LAUNCH();
 }
 

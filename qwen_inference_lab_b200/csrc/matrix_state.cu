@@ -280,17 +280,13 @@ template <int N> __device__ __forceinline__ void ms_wait() { asm volatile("cp.as
 // to dp become zero.  Rows and row stride on 16-byte boundaries take 16 bytes a copy.
 __device__ __forceinline__ void ms_load_rows(float* dst, int stride, const float* src, long long ld, int count, int d, int dp,
                                              bool pad, int tid, int threads) {
+    const int lane = tid & 31, warps = threads >> 5;
     if (d % 4 == 0 && ld % 4 == 0 && ((uintptr_t)src & 15) == 0) {
-        const int pieces = d / 4;
-        for (int i = tid; i < MS_CHUNK * pieces; i += threads) {
-            const int r = i / pieces, c = i % pieces * 4;
-            ms_copy16(dst + r * stride + c, src + (r < count ? r : 0) * ld + c, r < count);
-        }
+        for (int r = tid >> 5; r < MS_CHUNK; r += warps)         // a warp a row: no division by the row's length
+            for (int c = lane * 4; c < d; c += 128) ms_copy16(dst + r * stride + c, src + (r < count ? r : 0) * ld + c, r < count);
     } else {
-        for (int i = tid; i < MS_CHUNK * d; i += threads) {
-            const int r = i / d, c = i % d;
-            ms_copy4(dst + r * stride + c, src + (r < count ? r : 0) * ld + c, r < count);
-        }
+        for (int r = tid >> 5; r < MS_CHUNK; r += warps)
+            for (int c = lane; c < d; c += 32) ms_copy4(dst + r * stride + c, src + (r < count ? r : 0) * ld + c, r < count);
     }
     if (pad && dp > d)
         for (int i = tid; i < MS_CHUNK * (dp - d); i += threads) dst[i / (dp - d) * stride + d + i % (dp - d)] = 0.f;
@@ -419,13 +415,15 @@ delta_solve_kernel(StateRows in, const int* __restrict__ chunk_start, const int*
     }
     __syncthreads();
     invert_unit_lower(sa, st, sv, tid);
-    for (int i = tid; i < MS_CHUNK * dp; i += 256) sk[i / dp * stride + i % dp] *= beta_decay[i / dp];      // the keys' right side
+    for (int r = tid >> 5; r < MS_CHUNK; r += 8)                  // the keys' right side
+        for (int c = tid & 31; c < dp; c += 32) sk[r * stride + c] *= beta_decay[r];
     const T* v = reinterpret_cast<const T*>(in.v);
     for (int tile = 0; tile < (e + 63) / 64 + (d + 63) / 64; ++tile) {
         const bool is_value = tile < (e + 63) / 64;
         const int col0 = (is_value ? tile : tile - (e + 63) / 64) * 64, width = is_value ? e : d;
         if (is_value) {
             __syncthreads();            // the tile before has been read
+#pragma unroll 8
             for (int i = tid; i < MS_CHUNK * 64; i += 256) {
                 const int r = i / 64, c = col0 + i % 64;
                 sv[r * MS_A_STRIDE + i % 64] = (r < count && c < e)
@@ -685,6 +683,7 @@ state_own_kernel(StateRows in, const int* __restrict__ chunk_start, const int* _
         chunk_tail_decays(sums, tail, tid);
     }
     __syncthreads();
+#pragma unroll 8
     for (int i = tid; i < MS_CHUNK * 64; i += 256) {
         const int r = i / 64, c = col0 + i % 64;
         sv[r * MS_A_STRIDE + i % 64] = (r < count && c < e) ? tail[r] * to_f32<T>(v[(size_t)(first + r) * in.v_ld + (size_t)head * e + c]) : 0.f;
@@ -796,6 +795,7 @@ state_outputs_kernel(StateRows in, const int* __restrict__ chunk_start, const in
                 }
             }
         } else {
+#pragma unroll 8
             for (int i = tid; i < MS_CHUNK * MS_OUT_COLS; i += 256) {
                 const int t = i / MS_OUT_COLS, c = col0 + i % MS_OUT_COLS;
                 sy[i] = (t < count && c < e) ? to_f32<T>(v[(size_t)(first + t) * in.v_ld + (size_t)head * e + c]) : 0.f;

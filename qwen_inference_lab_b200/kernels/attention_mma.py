@@ -386,14 +386,14 @@ def attend(ctx, q, cache, out, n_q_heads, n_kv_heads, head_dim, window, scale, s
     n_tiles, n_big, n_rest, n_decode = (counts[name] // 4 for name in
                                         ("tile_info", "big_tile_info", "rest_tile_info", "decode_info"))
     if n_big and (not options or attention_tc.takes(options)) and not shared_rows \
-            and v_dim == head_dim and attention_tc.supports(head_dim, cache.page_size, window):
+            and attention_tc.supports(head_dim, cache.page_size, window, v_dim):
         # whole 128-token tiles on tcgen05 with the accumulators in tensor memory, the leftovers below
         if options:
             options.check(n_q_heads)
         attention_tc.prefill(q, cache.pages, out, arrays["big_tile_info"], n_big, cache.block_table,
                              n_q_heads, n_kv_heads, cache.page_size, scale, slopes_log2=slopes_log2,
                              chunk=options.chunk if options else 0, sink_log2=options._sink_log2 if options else None,
-                             softcap=options.softcap if options else 0.0, window=window)
+                             softcap=options.softcap if options else 0.0, window=window, head_dim=head_dim, v_dim=v_dim)
         if n_rest:
             prefill(q, cache.pages, out, arrays["rest_tile_info"], n_rest, cache.block_table, n_q_heads,
                     n_kv_heads, head_dim, cache.page_size, window, scale, slopes_log2, options, v_dim=v_dim)

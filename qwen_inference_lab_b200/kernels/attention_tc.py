@@ -1,4 +1,5 @@
-"""The tcgen05/TMA attention for whole 128-token query tiles (bfloat16, head size 128).
+"""The tcgen05/TMA attention for whole 128-token query tiles (bfloat16, head and value sizes up to 128), compiled per pair of
+sizes on first use.
 
 ``prefill`` takes tiles of exactly 128 tokens; :func:`attention_mma.prefill` takes what is left.
 The kernel's mbarrier waits are bounded and report through an error word that ``check()`` reads.
@@ -13,25 +14,37 @@ from . import build
 from . import ops
 from .ops import KernelError, _check, _need, _p, _stream
 
-HEAD_DIM = 128
+MOST_DIM = 128
 TILE = 128
-_lib = None
+_libs: dict = {}
 _fault = ops.ErrorWord(lambda code: f"attention_tc: a wait inside the kernel ran out (code {code}: 1x producer, "
                                     f"13-17 MMA issuer, 2x softmax warps)")
 
 
-def library():
-    global _lib
-    if _lib is None:
-        _lib = build.load("qil_attn_tc", ["attention_tc.cu"])
+def library_name(head_dim=MOST_DIM, v_dim=None):
+    """(name, defines) of the library for queries and keys of ``head_dim`` and values of ``v_dim`` (None: the same)."""
+    v_dim = head_dim if v_dim is None else v_dim
+    if head_dim == v_dim == MOST_DIM:
+        return "qil_attn_tc", {}
+    return f"qil_attn_tc_d{head_dim}_v{v_dim}", {"QIL_HEAD_DIM": head_dim, "QIL_V_DIM": v_dim}
+
+
+def library(head_dim=MOST_DIM, v_dim=None):
+    v_dim = head_dim if v_dim is None else v_dim
+    lib = _libs.get((head_dim, v_dim))
+    if lib is None:
+        name, defines = library_name(head_dim, v_dim)
+        lib = build.load(name, ["attention_tc.cu"], defines)
         ops.register_post_step_check(check)
-        if _lib.qil_attn_tc_head_dim() != HEAD_DIM:
-            raise KernelError("attention_tc was built for another head size")
-    return _lib
+        if lib.qil_attn_tc_head_dim() != head_dim or lib.qil_attn_tc_v_dim() != v_dim:
+            raise KernelError("attention_tc was built for other head sizes")
+        _libs[(head_dim, v_dim)] = lib
+    return lib
 
 
-def supports(head_dim, page_size, window) -> bool:
-    return head_dim == HEAD_DIM and window >= 0 and page_size in (8, 16, 32, 64)
+def supports(head_dim, page_size, window, v_dim=None) -> bool:
+    fits = lambda size: size % 16 == 0 and 16 <= size <= MOST_DIM
+    return fits(head_dim) and fits(head_dim if v_dim is None else v_dim) and window >= 0 and page_size in (8, 16, 32, 64)
 
 
 def takes(options) -> bool:
@@ -40,8 +53,9 @@ def takes(options) -> bool:
 
 
 def prefill(q, pages, out, tile_info, n_tiles, block_table, n_q_heads, n_kv_heads, page_size, scale, trace=None,
-            lib=None, slopes_log2=None, chunk=0, sink_log2=None, softcap=0.0, window=0):
-    """q, out bfloat16 [N, Hq*128]; pages [num_pages, 2, Hkv, page_size, 128];
+            lib=None, slopes_log2=None, chunk=0, sink_log2=None, softcap=0.0, window=0, head_dim=MOST_DIM, v_dim=None):
+    """q bfloat16 [N, Hq*head_dim], out [N, Hq*v_dim] (``v_dim`` None: head_dim); pages [num_pages, 2, Hkv, page_size, head_dim],
+    or with a value size of its own [num_pages, Hkv * page_size * (head_dim + v_dim)];
     tile_info int32 [n_tiles * 4] = (first token, its position, 128, block-table row).
     ``slopes_log2`` float32 [Hq] on the device: slope_h * log2(e) of a bias slope_h * (query position - key
     position) taken off the scaled score.  ``chunk`` > 0: a query sees the keys of its own chunk of that many
@@ -56,10 +70,12 @@ def prefill(q, pages, out, tile_info, n_tiles, block_table, n_q_heads, n_kv_head
         _need(slopes_log2, "slopes_log2", torch.float32, 1)
         if slopes_log2.shape[0] != n_q_heads:
             raise KernelError("attention_tc: one slope per query head")
-    _need(q, "q", torch.bfloat16, 2); _need(out, "out", torch.bfloat16, 2); _need(pages, "pages", torch.bfloat16, 5)
-    if tuple(pages.shape[1:]) != (2, n_kv_heads, page_size, HEAD_DIM) or q.shape[1] != n_q_heads * HEAD_DIM:
+    v_dim = head_dim if v_dim is None else v_dim
+    _need(q, "q", torch.bfloat16, 2); _need(out, "out", torch.bfloat16, 2)
+    ops.check_pages(pages, torch.bfloat16, n_kv_heads, page_size, head_dim, v_dim, "attention_tc")
+    if q.shape[1] != n_q_heads * head_dim or out.shape != (q.shape[0], n_q_heads * v_dim):
         raise KernelError("attention_tc: shapes do not match the head counts")
-    lib = lib or library()
+    lib = lib or library(head_dim, v_dim)
     word = _fault.tensor(q.device)
     _fault.mark()
     _check(lib, lib.qil_attn_tc_prefill_capped(

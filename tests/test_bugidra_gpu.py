@@ -341,13 +341,16 @@ def test_gated_attention_and_mixed_values(dtype, first, second):
                     close(got[rid][:, half], expected[rid][:, half], dtype)
 
 
-def test_whole_tiles_of_heads_of_128_take_the_tensor_memory_kernel(monkeypatch):
+@pytest.mark.parametrize("dim,vdim", [(128, 128), (128, 64), (64, 64), (48, 80), (32, 16), (16, 128), (112, 96)])
+def test_whole_tiles_take_the_tensor_memory_kernel(monkeypatch, dim, vdim):
+    """Whole 128-token tiles of a prompt go to the tcgen05 kernel whatever the sizes of keys and values: one slab of 64 columns
+    and two, whole and in part; leftovers and single tokens take the tiled kernels."""
     from qwen_inference_lab_b200.kernels import attention_tc
     calls = []
     original = attention_tc.prefill
     monkeypatch.setattr(attention_tc, "prefill", lambda *a, **k: (calls.append(k.get("softcap")), original(*a, **k))[1])
-    gated = dict(cases.left(4, 2, 128, 128, 0.2, cases.rot(10000.0, 128)), softcap=6.0)
-    unit = cases.left(4, 1, 128, 128, 0.2, cases.rot(10000.0, 64, (4.0, 128, 16.0, 1.0)))
+    gated = dict(cases.left(4, 2, dim, vdim, 2.2 * dim ** -0.5, cases.rot(10000.0, dim)), softcap=6.0)
+    unit = cases.left(4, 1, dim, vdim, 2.2 * dim ** -0.5, cases.rot(10000.0, dim // 2, (4.0, 128, 16.0, 1.0)))
     inputs = {"a": rows(460, 64, 32), "b": rows(140, 64, 33)}
     for m, part, mixer in ((gated, gated_part(64, gated), plain.gated_attention_mixer), (unit, left_part(64, unit), plain.unit_attention_mixer)):
         w = fill(part, 31, torch.bfloat16)
