@@ -472,6 +472,27 @@ delta_solve_kernel(StateRows in, const int* __restrict__ chunk_start, const int*
 }
 
 // ------------------------------------------------------------------ the chunks of a portion in order
+// MS_CHUNK rows of d floats, `ld` apart, into rows of DP + 16 floats by 256 threads; rows from `count` on become zero, columns from
+// d on stay as they are.
+template <int DP>
+__device__ __forceinline__ void ms_load_tile(float* dst, const float* src, long long ld, int count, int d, int tid) {
+    if (d % 4 != 0 || ld % 4 != 0 || ((uintptr_t)src & 15) != 0) {
+        ms_load_rows(dst, DP + 16, src, ld, count, d, DP, false, tid, 256);
+        return;
+    }
+    constexpr int PIECES = DP / 4, ROWS = 256 / PIECES;
+    const int r0 = tid / PIECES, c = tid % PIECES * 4;
+    if (c >= d) return;
+    const float* from = src + r0 * ld + c;
+    const long long step = ROWS * ld;
+#pragma unroll
+    for (int n = 0; n < MS_CHUNK / ROWS; ++n) {
+        const bool real = r0 + n * ROWS < count;
+        ms_copy16(dst + (r0 + n * ROWS) * (DP + 16) + c, real ? from : src, real);
+        from += step;
+    }
+}
+
 // Sums of 16 values over LANES neighbouring lanes; lane l of them keeps values l * 16 / LANES and following, at the front.
 template <int LANES>
 __device__ __forceinline__ void scatter_sums(float (&v)[16], int lane) {
@@ -492,8 +513,9 @@ __device__ __forceinline__ void scatter_sums(float (&v)[16], int lane) {
 // One block per (head, COLS value columns, long portion).  carry: int32 [portions, 3] = (state slot, first chunk, chunks).
 // chunk_state [chunks, heads, d, e] receives the state that comes into every chunk, y [chunks, heads, MS_CHUNK, e] the
 // corrected values in place of u; the state after the last chunk goes to the request's slot.  The state's columns live in
-// registers, with a copy in shared memory for the first product.  ITEMS: of 128 key channels that a thread serves.
-template <int COLS, int ITEMS>
+// registers, with a copy in shared memory for the first product.  DP: key channels that the tiles hold, at least d; the rest
+// stays zero.
+template <int COLS, int DP>
 __global__ void __launch_bounds__(256, 1)
 delta_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* __restrict__ chunk_len, const int* __restrict__ carry,
                   int n_heads, int d, int e, float* __restrict__ y, const float* __restrict__ w_in, const float* __restrict__ decays,
@@ -502,18 +524,19 @@ delta_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* 
     constexpr int KS = 16 / CG;            // lanes that share 4 x 4 elements of the first product, each over a part of the channels
     constexpr int TS = 8 / CG;             // the same for the second product, over the tokens
     constexpr int KEEP = 16 / KS, HOLD = 16 / TS;
+    constexpr int ITEMS = (DP + 127) / 128;                            // of 128 channels that a thread serves
+    constexpr int STRIDE = DP + 16, STATE_STRIDE = DP + 4, TILE = MS_CHUNK * STRIDE;      // 16 banks from row to row
     extern __shared__ __align__(16) float smem[];
-    const int dp = (d + 31) / 32 * 32, stride = dp + 16, state_stride = dp + 4, tile = MS_CHUNK * stride;
-    float* sk = smem;                                  // [stages][MS_CHUNK][stride]
-    float* sw = sk + stages * tile;                    // the same
-    float* ss = sw + stages * tile;                    // [COLS][state_stride]
-    float* sy = ss + COLS * state_stride;              // [MS_CHUNK][COLS]: y times its decay to the chunk's end
+    float* sk = smem;                                  // [stages][MS_CHUNK][STRIDE]
+    float* sw = sk + stages * TILE;                    // the same
+    float* ss = sw + stages * TILE;                    // [COLS][STATE_STRIDE]
+    float* sy = ss + COLS * STATE_STRIDE;              // [MS_CHUNK][COLS]: y times its decay to the chunk's end
     float* sd = sy + MS_CHUNK * COLS;                  // [stages][MS_DECAY_STRIDE]
     const int tiles = (e + COLS - 1) / COLS;
     const int head = blockIdx.x / tiles, col0 = (blockIdx.x % tiles) * COLS, tid = threadIdx.x;
     const int row = carry[3 * blockIdx.y], chunk0 = carry[3 * blockIdx.y + 1], chunks = carry[3 * blockIdx.y + 2];
     const size_t qk_at = (size_t)(head / in.group) * d;
-    const int total = stages * (2 * tile + MS_DECAY_STRIDE) + COLS * (state_stride + MS_CHUNK);
+    const int total = stages * (2 * TILE + MS_DECAY_STRIDE) + COLS * (STATE_STRIDE + MS_CHUNK);
     for (int i = tid; i < total; i += 256) smem[i] = 0.f;      // the padding stays zero
     const int part = tid % KS, cg = tid / KS % CG, rg = tid / KS / CG;                  // first product: rows rg + 16 a
     const int my_row = rg + 16 * (part * KEEP / 4), my_col = 4 * cg + part * KEEP % 4;  // of the sums this thread keeps
@@ -531,13 +554,13 @@ delta_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* 
         for (int i = 0; i < HOLD; ++i) {
             const int dd = d_first + 128 * it + hold_d + i / 4;
             S[it][i] = (dd < d && col0 + 4 * gc + i % 4 < e) ? slot[(size_t)dd * e + i % 4] : 0.f;
-            if (dd < dp) ss[(4 * gc + i % 4) * state_stride + dd] = S[it][i];
+            if (dd < DP) ss[(4 * gc + i % 4) * STATE_STRIDE + dd] = S[it][i];
         }
     auto fetch = [&](int chunk, int stage) {
         const int first = chunk_start[chunk], count = chunk_len[chunk];
         const size_t block = (size_t)chunk * n_heads + head;
-        ms_load_rows(sk + stage * tile, stride, in.k + (size_t)first * in.qk_ld + qk_at, in.qk_ld, count, d, dp, false, tid, 256);
-        ms_load_rows(sw + stage * tile, stride, w_in + block * MS_CHUNK * d, d, MS_CHUNK, d, dp, false, tid, 256);
+        ms_load_tile<DP>(sk + stage * TILE, in.k + (size_t)first * in.qk_ld + qk_at, in.qk_ld, count, d, tid);
+        ms_load_tile<DP>(sw + stage * TILE, w_in + block * MS_CHUNK * d, d, MS_CHUNK, d, tid);
         if (tid < MS_DECAY_STRIDE / 4) ms_copy16(sd + stage * MS_DECAY_STRIDE + 4 * tid, decays + block * MS_DECAY_STRIDE + 4 * tid, true);
         ms_commit();
     };
@@ -564,8 +587,8 @@ delta_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* 
         ms_wait<0>();
         __syncthreads();                   // this chunk's tiles are here, everyone has left the chunk before
         if (stages == 2 && n + 1 < chunks) fetch(chunk + 1, stage ^ 1);
-        const float* tk = sk + stage * tile;
-        const float* tw = sw + stage * tile;
+        const float* tk = sk + stage * TILE;
+        const float* tw = sw + stage * TILE;
         const float* tail = sd + stage * MS_DECAY_STRIDE;
         float* into = chunk_state + ((size_t)chunk * n_heads + head) * d * e + col0 + 4 * gc;
 #pragma unroll
@@ -585,13 +608,15 @@ delta_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* 
             float acc[16];
 #pragma unroll
             for (int i = 0; i < 16; ++i) acc[i] = 0.f;
-#pragma unroll 2
-            for (int c = part * 4; c < dp; c += 4 * KS) {
+            const float* w_at = tw + rg * STRIDE + part * 4;
+            const float* s_at = ss + 4 * cg * STATE_STRIDE + part * 4;
+#pragma unroll 4
+            for (int c = 0; c < DP; c += 4 * KS) {
                 float4 wv[4], sv[4];
 #pragma unroll
                 for (int a = 0; a < 4; ++a) {
-                    wv[a] = *reinterpret_cast<const float4*>(tw + (rg + 16 * a) * stride + c);
-                    sv[a] = *reinterpret_cast<const float4*>(ss + (4 * cg + a) * state_stride + c);
+                    wv[a] = *reinterpret_cast<const float4*>(w_at + 16 * a * STRIDE + c);
+                    sv[a] = *reinterpret_cast<const float4*>(s_at + a * STATE_STRIDE + c);
                 }
 #pragma unroll
                 for (int a = 0; a < 4; ++a)
@@ -624,14 +649,16 @@ delta_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* 
 #pragma unroll
         for (int it = 0; it < ITEMS; ++it) {
             const int d4 = d_first + 128 * it;
-            if (d4 >= dp) break;           // dp is a multiple of 32: whole warps leave together
+            if (d4 >= DP) break;           // whole warps leave together
             float acc[16];
 #pragma unroll
             for (int i = 0; i < 16; ++i) acc[i] = 0.f;
-#pragma unroll 4
-            for (int t = ts; t < MS_CHUNK; t += TS) {
-                const float4 kv = *reinterpret_cast<const float4*>(tk + t * stride + d4);
-                const float4 yv = *reinterpret_cast<const float4*>(sy + t * COLS + 4 * gc);
+            const float* k_at = tk + ts * STRIDE + d4;
+            const float* y_at = sy + ts * COLS + 4 * gc;
+#pragma unroll 8
+            for (int t = 0; t < MS_CHUNK; t += TS) {
+                const float4 kv = *reinterpret_cast<const float4*>(k_at + t * STRIDE);
+                const float4 yv = *reinterpret_cast<const float4*>(y_at + t * COLS);
                 const float ka[4] = {kv.x, kv.y, kv.z, kv.w}, ya[4] = {yv.x, yv.y, yv.z, yv.w};
 #pragma unroll
                 for (int a = 0; a < 4; ++a)
@@ -642,7 +669,7 @@ delta_walk_kernel(StateRows in, const int* __restrict__ chunk_start, const int* 
 #pragma unroll
             for (int i = 0; i < HOLD; ++i) {
                 S[it][i] = fmaf(whole, S[it][i], acc[i]);
-                ss[(4 * gc + i % 4) * state_stride + d4 + hold_d + i / 4] = S[it][i];
+                ss[(4 * gc + i % 4) * STATE_STRIDE + d4 + hold_d + i / 4] = S[it][i];
             }
         }
         if (stages == 1) __syncthreads();  // the tiles are overwritten next
@@ -857,8 +884,9 @@ static cudaError_t ms_reserve(Kernel kernel, size_t smem) {
 extern "C" int qil_gla_carry(float* chunk_state, const float* decay_product, float* slots, const int* carry, int n_carries,
                              int n_heads, int d, int e, cudaStream_t stream);
 
+static int delta_walk_dp(int d) { return d <= 64 ? 64 : d <= 128 ? 128 : MS_MOST_D; }
 static size_t delta_walk_smem(int d, int cols, int stages) {
-    const int dp = (d + 31) / 32 * 32;
+    const int dp = delta_walk_dp(d);
     return (size_t)(stages * (2 * MS_CHUNK * (dp + 16) + MS_DECAY_STRIDE) + cols * (dp + 4 + MS_CHUNK)) * sizeof(float);
 }
 
@@ -898,13 +926,14 @@ extern "C" int qil_state_chunks(const float* q, const float* k, long long qk_ld,
     const size_t walk_smem = delta_walk_smem(d, cols, stages);
     cudaError_t err = cudaSuccess;
 #define QIL_MS(...) do { if (err == cudaSuccess) err = (__VA_ARGS__); } while (0)
-#define QIL_MS_WALK(COLS, ITEMS)                                                                                        \
+#define QIL_MS_WALK(COLS, DP)                                                                                           \
     do {                                                                                                                \
-        QIL_MS(ms_reserve(delta_walk_kernel<COLS, ITEMS>, walk_smem));                                                  \
-        QIL_MS(qil_launch_chained(delta_walk_kernel<COLS, ITEMS>, dim3(n_heads * tiles, n_carries), dim3(256), walk_smem, stream, \
-                                  in, chunk_start, chunk_len, carry, n_heads, d, e, y, (const float*)w, (const float*)decays,     \
+        QIL_MS(ms_reserve(delta_walk_kernel<COLS, DP>, walk_smem));                                                     \
+        QIL_MS(qil_launch_chained(delta_walk_kernel<COLS, DP>, dim3(n_heads * tiles, n_carries), dim3(256), walk_smem, stream,  \
+                                  in, chunk_start, chunk_len, carry, n_heads, d, e, y, (const float*)w, (const float*)decays,   \
                                   chunk_state, slots, stages));                                                         \
     } while (0)
+#define QIL_MS_COLS(DP) do { if (cols == 8) QIL_MS_WALK(8, DP); else QIL_MS_WALK(16, DP); } while (0)
 #define QIL_MS_OUTPUTS(DELTA)                                                                                           \
     do {                                                                                                                \
         QIL_MS(ms_reserve(state_outputs_kernel<T, DELTA>, out_smem));                                                   \
@@ -916,8 +945,9 @@ extern "C" int qil_state_chunks(const float* q, const float* k, long long qk_ld,
             QIL_MS(ms_reserve(delta_solve_kernel<T>, row_tile + 3 * a_tile));
             QIL_MS(qil_launch_chained(delta_solve_kernel<T>, dim3(n_heads, n_chunks), dim3(256), row_tile + 3 * a_tile, stream, in,
                                       chunk_start, chunk_len, n_heads, d, e, y, w, decays));
-            if (d <= 128) { if (cols == 8) QIL_MS_WALK(8, 1); else QIL_MS_WALK(16, 1); }
-            else { if (cols == 8) QIL_MS_WALK(8, 2); else QIL_MS_WALK(16, 2); }
+            if (delta_walk_dp(d) == 64) QIL_MS_COLS(64);
+            else if (delta_walk_dp(d) == 128) QIL_MS_COLS(128);
+            else QIL_MS_COLS(MS_MOST_D);
             QIL_MS_OUTPUTS(true);
         } else {
             QIL_MS(ms_reserve(state_own_kernel<T>, row_tile + a_tile));
@@ -931,6 +961,7 @@ extern "C" int qil_state_chunks(const float* q, const float* k, long long qk_ld,
         }
     });
 #undef QIL_MS_OUTPUTS
+#undef QIL_MS_COLS
 #undef QIL_MS_WALK
 #undef QIL_MS
     if (err != cudaSuccess) { snprintf(qil_error_text, sizeof(qil_error_text), "%s", cudaGetErrorString(err)); return (int)err; }

@@ -715,6 +715,19 @@ def test_greedy_generation_through_the_engine(folders, dtype):
             sequence.append(token)
 
 
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+def test_a_model_that_keeps_no_pages(tmp_path, dtype):
+    """Delta layers alone, one of them with a convolution of one tap: state slots and no key or value anywhere."""
+    config = cases.config(61, 48, 1e-5, 1.5, cases.delta(2, 1, 12, 16, 4, ff=40), cases.delta(3, 3, 16, 8, 1))
+    weights = cases.write_folder(config, 9, tmp_path)
+    requests = {"a": cases.random_tokens(config, 150, 1), "b": cases.random_tokens(config, 20, 2)}
+    _, cache, runner = harness.build_engine_parts(tmp_path, dtype, num_pages=4, page_size=64)
+    for schedule in (harness.whole_schedule(requests), harness.mixed_schedule(requests)):
+        got = harness.run_schedule(runner, cache, schedule)
+        judge(got, cases.plain_rows(requests, weights, config), cases.plain_rows(requests, weights, config, torch.bfloat16), dtype,
+              f"bugidra without pages {dtype}")
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_the_replay_program_runs_a_mixed_schedule(folders, truth, tmp_path, dtype):
     folder, weights, requests = folders["A"]
