@@ -16,7 +16,7 @@
 //   u_i + sum_{j < i} beta_i e^(L_i - L_j) (k_i . k_j) u_j  =  beta_i v_i - beta_i e^(L_i) S^T k_i
 //
 // so with A the strictly lower matrix of those coefficients, U = (I + A)^-1 diag(beta) V and
-// W = (I + A)^-1 diag(beta e^L) K (delta_solve, all chunks at once: forward substitution, a thread per column),
+// W = (I + A)^-1 diag(beta e^L) K (delta_solve, all chunks at once: an explicit inverse by blocks),
 //
 //   Y = U - W S            (plain: Y = V)                                    delta_walk: the chunks of a portion in order,
 //   S' = e^(L_C) S + sum_j e^(L_C - L_j) k_j y_j^T                           a block per (head, a few value columns)
